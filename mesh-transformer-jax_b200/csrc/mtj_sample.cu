@@ -39,6 +39,8 @@ namespace {
 
 constexpr int kSampThreads = 1024;
 
+// Published method: argument reduction and polynomials of the Cephes Mathematical Library (S. L. Moshier),
+// single-precision exp and log, with every operation rounded on its own.
 __device__ __forceinline__ float exp_pinned(float x) {     // x <= 0
   const float xs = fmaxf(x, -87.0f);
   const float n = rintf(__fmul_rn(xs, 1.4426950408889634f));

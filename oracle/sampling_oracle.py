@@ -93,7 +93,8 @@ def nucleaus_sample_plain(uniforms, logits, top_p=0.9, temp=1.0, top_k=None):
 
 
 # ----------------------------------------------------------------------------
-# pinned arithmetic
+# pinned arithmetic: the reductions and polynomials of the Cephes Mathematical Library (S. L. Moshier),
+# single-precision exp and log
 # ----------------------------------------------------------------------------
 _LOG2E = F32(1.4426950408889634)
 _LN2_HI = F32(0.693145751953125)          # 0x3f317200: few mantissa bits, n * LN2_HI is exact
