@@ -76,14 +76,57 @@ typedef struct mtj_config {
                                   the device error word (MTJ_ERR_TIMEOUT)        */
 } mtj_config;
 
+/* Layer-stack models (no counterpart in the reference): a list of layers, each a
+ * mixer between two RMS norms and, when ff > 0, a SwiGLU feed-forward between two
+ * more, x <- x + residual_mult * norm_after(sublayer(norm_before(x))).  Layers
+ * loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop), every
+ * pass with caches and states of its own, and every pass begins with
+ * x <- W_in [x; embedding output].
+ *   MTJ_MIXER_LATENT_ATTENTION: keys and values are linear maps of one
+ *     normalised latent of kv_rank numbers per token, plus rot_dim rotated key
+ *     dimensions shared by the heads (neighbouring dimensions are rotated together,
+ *     frequencies rot_base^(-2i/rot_dim)); position i sees j with
+ *     0 <= i - j < window; scores are multiplied by scale.
+ *   MTJ_MIXER_MAMBA1: gated causal convolution (conv taps) and selective scan
+ *     (inner channels x state), step sizes through dt_rank numbers. */
+enum { MTJ_MIXER_LATENT_ATTENTION = 0, MTJ_MIXER_MAMBA1 = 1 };
+typedef struct mtj_layer_desc {
+  int32_t mixer;
+  int32_t ff;                  /* feed-forward width, 0: no feed-forward         */
+  int32_t heads, dim, rot_dim, vdim, kv_rank, window;
+  int32_t inner, state, conv, dt_rank;
+  float scale;
+  int32_t reserved;
+  double rot_base;
+} mtj_layer_desc;
+typedef struct mtj_stack_desc {
+  const mtj_layer_desc* layers;
+  int32_t n_layers;
+  int32_t loop_start, loop_stop, loop_times;
+  float residual_mult, norm_eps;
+  int32_t act_f32;             /* 1: fp32 activations and caches throughout      */
+  int32_t tc_min_rows;         /* prompt rows from which a call takes the tensor-core
+                                  path; default 16                               */
+} mtj_stack_desc;
+
 const char* mtj_last_error(void);
-/* ABI revision: 3 (2: mtj_config with the tuning fields, mtj_generate, mtj_start_batch / mtj_admit;
- * 3: top_k in mtj_sample_top_p / mtj_nucleus_filter, mtj_set_top_k). */
+/* ABI revision: 4 (2: mtj_config with the tuning fields, mtj_generate, mtj_start_batch / mtj_admit;
+ * 3: top_k in mtj_sample_top_p / mtj_nucleus_filter, mtj_set_top_k; 4: layer-stack models, mtj_extend,
+ * mtj_release). */
 int32_t mtj_version(void);
 
 /* CausalTransformerShard.__init__ (transformer_shard.py:21-45): validates the
  * same divisibility conditions the reference asserts (layers.py:172,238-239,552). */
 int32_t mtj_create(const mtj_config* cfg, mtj_handle** out);
+/* The same for a layer-stack model.  Of cfg it reads d_model (the width), n_vocab,
+ * seq, max_batch, max_gen, max_rows and the decode fields; cores_per_replica must
+ * be 1.  seq + max_gen + 1 bounds a sequence's positions.  Tensors are loaded with
+ * mtj_load_param under their own names ("embed", "l0.mix.q", ...; a prefix up to
+ * the last '/' is dropped), linear weights [out, in].  The other calls are the
+ * same as for GPT-J, with these differences: prompts' left padding has no effect
+ * on positions, which count from 0 in each sequence; ctx_length of mtj_eval_loss
+ * and mtj_forward_logits is not used (the mixers are causal). */
+int32_t mtj_create_stack(const mtj_config* cfg, const mtj_stack_desc* stack, mtj_handle** out);
 int32_t mtj_destroy(mtj_handle* h);
 
 /* Arena sizes for this handle's config, then binding of caller memory. */
@@ -145,6 +188,17 @@ int32_t mtj_prefill(mtj_handle* h, const uint32_t* ctx_dev, const uint32_t* ctx_
  * max_gen steps in total. */
 int32_t mtj_start_batch(mtj_handle* h, int32_t batch, mtj_stream s);
 int32_t mtj_admit(mtj_handle* h, int32_t slot, const uint32_t* prompt_dev, int32_t len, mtj_stream s);
+
+/* Layer-stack models: appends len tokens to the sequence in a slot of the running
+ * batch (mtj_start_batch), at its next positions, from the cache and state that
+ * earlier calls left.  A prompt may be cut anywhere.  logits_out_dev
+ * [n_want, n_vocab] f32 receives the logits at the places want_host (indexes into
+ * the tokens, ascending order not required); n_want may be 0.  One token takes the
+ * kernels of a decode step.  mtj_admit afterwards, or mtj_release, starts the slot
+ * over: the next token is position 0. */
+int32_t mtj_extend(mtj_handle* h, int32_t slot, const uint32_t* tokens_dev, int32_t len, const int32_t* want_host,
+                   int32_t n_want, float* logits_out_dev, mtj_stream s);
+int32_t mtj_release(mtj_handle* h, int32_t slot, mtj_stream s);
 
 /* One step of the generate scan (transformer_shard.py:198-210): generate_once
  * then the sampler.  tokens_in_dev may be NULL (use the previous step's
@@ -333,6 +387,12 @@ int32_t mtj_k_prefill_attn(const void* q_bf16_dev, const void* kpool_dev, const 
                            int32_t batch, int32_t T, int32_t pos0, int32_t heads, int32_t d_head,
                            int32_t ring_pages, void* out_bf16_dev, int32_t ld_out, uint32_t* status_dev,
                            mtj_stream s);
+
+/* Layer-stack models: the residual stream after the first n_runs layer runs (a
+ * looped layer counts each time) of one fresh sequence of len tokens, put into
+ * slot 0: out_dev [len, d_model] f32.  The call ends any running batch. */
+int32_t mtj_k_stack_residual(mtj_handle* h, const uint32_t* tokens_dev, int32_t len, int32_t n_runs, float* out_dev,
+                             mtj_stream s);
 
 /* g_psum (util.py:134-136) for decode-size messages over peer memory, fused
  * with the residual add of the caller (transformer_shard.py:60,112) and the

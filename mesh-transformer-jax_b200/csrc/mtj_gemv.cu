@@ -13,6 +13,9 @@
 //             LayerNorm statistics of the finished rows computed by the last
 //             block to arrive (layers.py:285,290,313; transformer_shard.py:60)
 //   logits  : final LayerNorm prologue + bias (layers.py:561-564)
+//   SwiGLU  : LayerNorm prologue, rows in (gate, up) pairs, silu(gate) * up (layer-stack models)
+// The LayerNorm prologue with mean = 0 and a zero offset is RMSNorm; the out-proj epilogue can add the residual
+// behind a second RMSNorm (GemvArgs::post_w).
 #include "mtj_common.cuh"
 #include "mtj_kernels.h"
 
@@ -164,7 +167,7 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
     const float partner = __shfl_xor_sync(0xffffffffu, val, 1);   // the other row of the RoPE pair
     const int r = lane % RW, bt = lane / RW;
     const int n = a.n0 + row0 + r;                 // row index within the full projection
-    if (lane < RW * BT && bt < nb && row0 + r < a.N) {
+    if (lane < RW * BT && bt < nb && row0 + r < (a.n_valid > 0 ? a.n_valid : a.N)) {
       const int m = m0 + bt;
       if (EPI == kEpiInProj) {
         const int seq = a.rows.b0 + m / a.rows.Tc;
@@ -191,12 +194,15 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
           a.act2[static_cast<size_t>(m) * (a.dl + a.ffl) + a.dl + f] = gelu_tanh(val + a.b_ff[f]);
         }
       } else if (EPI == kEpiOut) {
-        float y = val + a.bias[n];
+        float y = a.bias ? val + a.bias[n] : val;
         if (a.residual) y += a.residual[static_cast<size_t>(m) * a.N + n];
         float* outp = a.out + (a.slot_sel ? static_cast<size_t>(*a.slot_sel & 1u) * a.slot_stride : 0);
-        outp[static_cast<size_t>(m) * a.N + n] = y;
+        outp[static_cast<size_t>(m) * (a.ld_out > 0 ? a.ld_out : a.N) + n] = y;
+      } else if (EPI == kEpiSwiGLU) {
+        // (gate, up) row pairs: the even row finishes the pair
+        if (!(r & 1)) a.act2[static_cast<size_t>(m) * a.ld_out + (n >> 1)] = val / (1.0f + expf(-val)) * partner;
       } else {
-        a.logits[static_cast<size_t>(m) * a.ld_logits + n] = val + a.bias[n];
+        a.logits[static_cast<size_t>(m) * a.ld_logits + n] = a.bias ? val + a.bias[n] : val;
       }
     }
   }
@@ -216,6 +222,35 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
     __syncthreads();
     if (!is_last) return;
     __threadfence();
+    if (a.post_w) {
+      // norm after the sublayer, residual add, and the root mean square of the new residual row
+      const int n_out = a.n_valid > 0 ? a.n_valid : a.N;
+      for (int bt = 0; bt < nb; ++bt) {
+        const float* row = a.out + static_cast<size_t>(m0 + bt) * (a.ld_out > 0 ? a.ld_out : a.N);
+        float* xrow = a.post_x + static_cast<size_t>(m0 + bt) * a.post_ldx;
+        float s = 0.f;
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+          const float y = __ldcg(row + i);
+          s = fmaf(y, y, s);
+        }
+        const float rs = a.post_mult / sqrtf(block_sum(s, red) / static_cast<float>(n_out) + a.post_eps);
+        float q = 0.f;
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+          const float v = fmaf(__ldcg(row + i) * rs, a.post_w[i], xrow[i]);
+          xrow[i] = v;
+          q = fmaf(v, v, q);
+        }
+        const float ms = block_sum(q, red) / static_cast<float>(n_out);
+        if (threadIdx.x == 0) {
+          a.stats_out[2 * (m0 + bt)] = 0.f;
+          a.stats_out[2 * (m0 + bt) + 1] = 1.0f / sqrtf(ms + a.post_eps);
+        }
+      }
+      if (threadIdx.x == 0) a.counters[blockIdx.y] = 0u;
+      return;
+    }
     for (int bt = 0; bt < nb; ++bt) {
       const float* row = a.out + static_cast<size_t>(m0 + bt) * a.N;
       float s = 0.f;
@@ -296,6 +331,7 @@ cudaError_t launch_gemv(GemvEpilogue epi, const GemvArgs& a, cudaStream_t s, boo
   switch (epi) {
     case kEpiInProj: return launch_epi<kEpiInProj>(a, s, pdl);
     case kEpiOut: return launch_epi<kEpiOut>(a, s, pdl);
+    case kEpiSwiGLU: return launch_epi<kEpiSwiGLU>(a, s, pdl);
     default: return launch_epi<kEpiLogits>(a, s, pdl);
   }
 }

@@ -26,8 +26,10 @@ struct KvCache {
 };
 
 enum GemvEpilogue { kEpiInProj = 0, kEpiOut = 1, kEpiLogits = 2,
-                    kEpiLogitsCE = 3 };   // logits that are never stored: per (128-entry vocabulary group, token) max and
+                    kEpiLogitsCE = 3,     // logits that are never stored: per (128-entry vocabulary group, token) max and
                                           // sum of exp instead, plus the target's logit (persistent GEMM only)
+                    kEpiPlain = 4,        // fp32 and / or bf16 result (tensor-core GEMM only)
+                    kEpiSwiGLU = 5 };     // weight rows in (gate, up) pairs: silu(gate) * up
 
 struct GemvArgs {
   // y[m, n] = sum_k W[n, k] * act(x[m, k]);  W is bf16 [N, K] (K contiguous).
@@ -63,6 +65,14 @@ struct GemvArgs {
   const uint32_t* slot_sel;    // optional: out += (*slot_sel & 1) * slot_stride (peer all-reduce slots)
   size_t slot_stride;
   int rw_override;             // 0 = default rows per warp group; 8 = eight rows (single-token launches)
+  int n_valid;                 // rows of W past this one are padding, nothing is stored for them (0 = N)
+  int ld_out;                  // row stride of `out` (0 = N); SwiGLU: of `act2`
+  // out-proj epilogue of layers with a norm after the sublayer: instead of the LayerNorm statistics of `out` the last
+  // block computes post_x += post_mult * RMSNorm(out) * post_w and, into stats_out, (0, 1 / rms) of the new post_x
+  const float* post_w;         // [n_valid] or null
+  float* post_x;               // [M, post_ldx]
+  int post_ldx;
+  float post_mult, post_eps;
 };
 
 cudaError_t launch_gemv(GemvEpilogue epi, const GemvArgs& a, cudaStream_t s, bool pdl);
@@ -74,11 +84,12 @@ struct EmbedArgs {
   RowMap rows;
   int M, d, vocab_local, vocab_start;
   const __nv_bfloat16* table;  // [vocab_local, d]
-  const float* bias;           // [d]
+  const float* bias;           // [d] or null
   float* x;                    // [M, d]
   float* stats;                // [M, 2] or null
   const uint32_t* slot_sel;    // optional: x += (*slot_sel & 1) * slot_stride (peer all-reduce slots)
   size_t slot_stride;
+  int ldx;                     // row stride of x (0 = d)
 };
 cudaError_t launch_embed(const EmbedArgs& a, cudaStream_t s, bool pdl);
 
@@ -124,9 +135,21 @@ struct PrefillAttnTcArgs {
   __nv_bfloat16* out_bf16;     // [M, ld_out]
   int ld_out;
   uint32_t* dev_err;
+  // linear keys and values (launch_prefill_attn_tc_linear): row i of sequence b of the chunk sits in matrix row
+  // b * key_rows + i and holds the key at position pos0 - hist + i
+  int window;                  // a query sees keys at most window - 1 positions back
+  int hist, key_rows;
+  int k_own;                   // 64-column blocks of a key row that belong to the head (the rest: all heads share them)
+  int v_cols;                  // value columns per head that exist (the matrix pads them to whole 64-column blocks)
+  float scale_log2;            // score scale times log2(e)
 };
 cudaError_t launch_prefill_attn_tc(const void* map_q, const void* map_k, const void* map_v,
                                    const PrefillAttnTcArgs& a, cudaStream_t s);
+// 64-column blocks of a key / value row the linear form needs, 0 = larger than its instances
+int attn_tc_key_blocks(int own_dim, int shared_dim);
+int attn_tc_value_blocks(int vdim);
+cudaError_t launch_prefill_attn_tc_linear(const void* map_q, const void* map_k, const void* map_ks, const void* map_v,
+                                          int key_blocks, int value_blocks, const PrefillAttnTcArgs& a, cudaStream_t s);
 
 // Persistent whole-step decode kernel (mtj_decode_mega.cu), one GPU, 1-4 sequences.
 struct MegaLayer {
@@ -200,7 +223,7 @@ cudaError_t launch_argmax(const ArgmaxArgs& a, cudaStream_t s, bool pdl);
 // Tensor-core GEMM (many token rows): weights bf16 [N, K], activations bf16 [*, K]
 // reached through TMA tensor maps; epilogues as in GemvArgs.
 struct GemmTcArgs {
-  int M, N, K;                 // token rows, weight rows, reduction length (multiple of 64)
+  int M, N, K;                 // token rows, weight rows, reduction length
   int x_row0;                  // first activation row (TMA row coordinate offset)
   RowMap rows;
   int dl, ffl, d_head, heads, rot;
@@ -227,6 +250,8 @@ struct GemmTcArgs {
   int ce_T, ce_vocab_start;
   int cluster_k;               // 2 or 4 (token tiles of at most 64 rows, partial == null): split K over a cluster of
                                // blocks that add their accumulators in shared memory before the fused epilogue
+  __nv_bfloat16* out_bf16;     // kEpiPlain: optional bf16 result; kEpiSwiGLU: the result (N / 2 columns)
+  int ld_bf16;
   int pair;                    // wide kernel only: 1 = clusters of 2 blocks on 256 x 256 tiles (tcgen05 cta_group::2)
   uint32_t* dev_err;
 };
@@ -238,7 +263,7 @@ int gemm_tc_decode_cluster_k(int weight_rows, int M, int K);
 cudaError_t launch_splitk_reduce(const float* partial, int ksplit, int M, int N, const float* bias,
                                  const float* residual, float* out, int ld_out, const uint32_t* slot_sel,
                                  size_t slot_stride, cudaStream_t s, bool pdl = false);
-cudaError_t make_tensor_map_bf16(void* map_out_128B, const void* base, int64_t rows, int64_t K, int box_rows);
+cudaError_t make_tensor_map_bf16(void* map_out_128B, const void* base, int64_t rows, int64_t K, int box_rows, int64_t ld = 0);   // ld: row stride in elements (0 = K)
 // map_x_lo (optional, M <= 64): a second activation view holding the bf16 rounding error of the first
 // (x = hi + lo); both are multiplied into the same accumulator.
 cudaError_t launch_gemm_tc(GemvEpilogue epi, const void* map_w, const void* map_x, const GemmTcArgs& a,

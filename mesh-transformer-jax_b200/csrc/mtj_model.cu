@@ -13,332 +13,17 @@
 #include "../../include/mtj_b200.h"
 #include "mtj_comm.h"
 #include "mtj_common.cuh"
+#include "mtj_handle.h"
 #include "mtj_kernels.h"
+#include "mtj_stack.h"
 
 namespace {
 
 thread_local std::string g_last_error;
 
-int32_t fail(int32_t code, const std::string& msg) {
-  g_last_error = msg;
-  return code;
-}
-
-#define MTJ_CUDA(expr)                                                              \
-  do {                                                                              \
-    cudaError_t _e = (expr);                                                        \
-    if (_e != cudaSuccess)                                                          \
-      return fail(MTJ_ERR_CUDA, std::string(#expr) + ": " + cudaGetErrorString(_e)); \
-  } while (0)
-
-constexpr int kTcSplitMax = 8;      // split-K factor limit of the small-M out-projection
-constexpr int kTcSplitRows = 128;
-constexpr int kHiLoRows = 64;       // decode rows that can carry hi + lo activations
-constexpr int kTpPipeMinRows = 128; // a chunk is cut in two for all-reduce overlap only if each half keeps this many rows
-
-struct alignas(64) TensorMap { unsigned char bytes[128]; };   // a CUtensorMap
-
-struct LayerWeights {
-  __nv_bfloat16* w_in = nullptr;    // [3*dl + ffl, d]  rows: Q | K | V | FF-in
-  float* b_ff = nullptr;            // [ffl]
-  __nv_bfloat16* w_out = nullptr;   // [d, dl + ffl]    cols: attn vector | gelu(ff)
-  float* b_out = nullptr;           // [d]
-  float* ln_scale = nullptr;
-  float* ln_offset = nullptr;
-  TensorMap map_in, map_out;        // TMA views of w_in / w_out for the tensor-core path
-  TensorMap map_k, map_v;           // TMA views of this layer's K / V pools as [pages*heads*64, d_head]
-};
-
-int64_t align_up(int64_t v, int64_t a) { return (v + a - 1) / a * a; }
-
-// Bump allocator over a caller-provided arena; with base == nullptr it only sizes.
-struct Carver {
-  char* base;
-  int64_t off = 0;
-  explicit Carver(void* b) : base(static_cast<char*>(b)) {}
-  template <typename T>
-  T* take(int64_t count) {
-    off = align_up(off, 256);
-    T* p = base ? reinterpret_cast<T*>(base + off) : nullptr;
-    off += count * static_cast<int64_t>(sizeof(T));
-    return p;
-  }
-};
+using namespace mtj;
 
 }  // namespace
-
-struct mtj_handle {
-  mtj_config cfg;
-  int L, d, n_heads, heads, dh, rot, V, Vl, seq, W, mp, rank, dl, ffl;
-  int max_batch, max_gen, max_rows, ring_pages, n_pages, max_pos, max_splits;
-
-  // weight arena
-  __nv_bfloat16* emb_w = nullptr;
-  float* emb_b = nullptr;
-  std::vector<LayerWeights> layers;
-  float* lnf_scale = nullptr;
-  float* lnf_offset = nullptr;
-  __nv_bfloat16* proj_w = nullptr;
-  float* proj_b = nullptr;
-  float2* sincos = nullptr;
-  std::vector<uint8_t> leaf_loaded;   // one mark per parameter leaf (embedding 2, 10 per layer, projection 4)
-  int64_t expected = 0;
-
-  // workspace
-  float* x = nullptr;
-  float* stats = nullptr;
-  float* q = nullptr;
-  float* act2 = nullptr;
-  float* part_o = nullptr;
-  float* part_ml = nullptr;
-  uint32_t* counters = nullptr;     // attention + gemv tickets (zeroed at bind)
-  uint32_t* gemv_counters = nullptr;
-  float* logits = nullptr;          // [max_batch, Vl] this shard's logits
-  float* logits_all = nullptr;      // [max_batch, V]  (== logits when mp == 1)
-  float* logits_gather = nullptr;   // [mp, max_batch, Vl] all-gather landing zone (mp > 1)
-  float* part = nullptr;            // [max_rows, d] this shard's partial sums before the all-reduce (mp > 1)
-  void* comm = nullptr;             // ncclComm_t over the "shard" axis
-  // peer-memory all-reduce for small messages (decode); buffers are cudaMalloc'ed once at set-up
-  // because they have to be exportable to the other ranks' processes
-  bool p2p_ready = false;
-  int p2p_rows = 0;                 // rows a data slot holds
-  char* p2p_local = nullptr;        // [2 slots][p2p_rows * d] floats | flags | seq | ticket
-  char* p2p_peer[mtj::kP2pMaxWorld] = {};
-  size_t p2p_flag_off = 0;
-  size_t p2p_recv_off = 0;          // push exchange of the persistent decode kernel
-  size_t p2p_push_off = 0;          // receive area of the per-layer push all-reduce [2][mp][p2p_rows][d] floats
-  size_t p2p_pflag_off = 0;         // its row flags [mp][p2p_rows]
-  size_t p2p_amax_off = 0;          // greedy-token packets [2][mp][p2p_rows][2] uint2
-  bool tp_token = true;             // decode at mp > 1: the greedy token is agreed on by pushing each rank's local
-                                    // arg-max to all ranks instead of gathering the logits (MTJ_NO_TP_TOKEN=1: off)
-  bool tp_push = false;             // batched decode at mp > 1: push all-reduce fused with the split-K reduction and
-                                    // the LayerNorm; default: from 4 shards on (MTJ_TP_PUSH=0 / 1 overrides)
-  bool xn_ready = false;            // the bf16 operand of the next projection has already been written
-  bool tc_cluster_k = true;         // batched decode: split K over block clusters when tiles are few (MTJ_NO_CLUSTER_K=1: off)
-  float* uniforms = nullptr;        // [max_batch, V] sampler inputs of the current step
-  float* top_p = nullptr;           // [max_batch]
-  float* temp = nullptr;            // [max_batch]
-  void* sample_scratch = nullptr;
-  // tensor-core path (many token rows): bf16 activation operands and their TMA views
-  bool tc_ok = false;
-  __nv_bfloat16* xn_bf16 = nullptr;   // [max_rows, d] LayerNorm output
-  __nv_bfloat16* act_bf16 = nullptr;  // [max_rows, dl + ffl] attention vector | gelu(ff)
-  TensorMap map_xn[3], map_act[3], map_proj, map_q;   // activation views with 32 / 64 / 128-row boxes
-  TensorMap map_xn_wide, map_act_wide;   // 256-row boxes for the persistent GEMM
-  __nv_bfloat16* q_bf16 = nullptr;    // [max_rows, dl] rotated queries for the tensor-core attention
-  bool attn_tc_ok = false;
-  // few-sequence decode: the bf16 rounding errors of the two activation operands (x = hi + lo), rows [0, kHiLoRows)
-  __nv_bfloat16* xn_lo = nullptr;
-  __nv_bfloat16* act_lo = nullptr;
-  TensorMap map_xn_lo[2], map_act_lo[2];   // 32 / 64-row boxes
-  bool hilo_ok = false;
-  int tc_hilo_max_b = kHiLoRows;    // up to this many sequences the activations travel as hi + lo (mtj_config.hilo_max_batch)
-  int wait_limit = 1 << 22;         // iteration limit of the bounded device-side waits (mtj_config.wait_limit)
-  bool tc_wide_ok = false;   // persistent 128 x 256 GEMM for long chunks
-  int tc_pair = 7;           // ... as block pairs on 256 x 256 tiles: bit 0 in-projection, 1 out-projection, 2 logits
-                             // (MTJ_TC_PAIR=<mask> overrides, for measurement)
-  bool mega_push = true;     // per-block push exchange inside the persistent decode kernel (MTJ_NO_MEGA_PUSH=1: slot protocol)
-  float* tc_partial = nullptr;        // [kTcSplitMax, kTcSplitRows, d] split-K partial sums of small-M out-projections
-  int eval_rows = 0;                // rows of logits materialised at a time by the loss path
-  float* eval_logits = nullptr;     // [eval_rows, Vl]
-  // loss path on the persistent GEMM: the logits are never stored, its epilogue leaves per (32-entry vocabulary
-  // group, row) the max and the sum of exp, plus the target's logit
-  int ce_groups = 0;
-  int ce_rows = 0;                  // rows per launch of that GEMM: several 256-row token tiles, so that a block's
-                                    // epilogues overlap its next tiles instead of ending the launch
-  float* ce_gmax = nullptr;         // [ce_groups, ce_rows]
-  float* ce_gsum = nullptr;
-  float* ce_tlogit = nullptr;       // [ce_rows]
-  uint8_t* ce_ghit = nullptr;       // [ce_rows]
-  bool fused_ce = true;             // MTJ_NO_FUSED_CE=1: materialise the logits slice and run ce_partial instead
-  float* ce_max = nullptr;          // [max_rows] local max, then global max
-  float* ce_lmax = nullptr;         // [max_rows] copy of the local max (mp > 1)
-  float* ce_sum = nullptr;          // [max_rows, 2]
-  uint8_t* ce_hit = nullptr;        // [max_rows]
-  uint32_t* tokens = nullptr;       // [max_batch] next decode input
-  int32_t* cur = nullptr;           // absolute position of the next decode token
-  int32_t* pad = nullptr;           // [max_batch]
-  int32_t* key_limit = nullptr;     // [max_batch]
-  int32_t* page_table = nullptr;    // [max_batch, ring_pages]
-  int32_t* row_select = nullptr;    // [max_rows]
-  uint32_t* dev_err = nullptr;
-  uint32_t* rng_seed = nullptr;     // [2] key of the device generator that draws the sampler's uniforms
-  int32_t* top_k = nullptr;         // [max_batch] the sampler's top_k, used while has_top_k
-  bool has_top_k = false;
-  __nv_bfloat16* kpool = nullptr;   // [L][n_pages][heads][kPageTokens][dh]
-  __nv_bfloat16* vpool = nullptr;
-  int64_t pool_layer_elems = 0;
-  bool bound = false;
-
-  // decode state
-  int min_pad = 0;                  // smallest first-visible position over the running sequences
-  // pages a sequence of the running batch holds at most right now (its window start to the decode position)
-  int est_pages() const {
-    const int cur = W + steps_done;
-    const int start = std::max(min_pad, cur - W + 1);
-    return cur / mtj::kPageTokens - start / mtj::kPageTokens + 1;
-  }
-  int batch = 0;
-  bool prefilled = false;
-  int steps_done = 0;
-  int64_t launches = 0;
-  bool use_pdl = true;
-  int ks_inproj = 0, ks_out = 0, ks_logits = 0;   // K-split overrides (tuning; 0 = automatic)
-  // decode of 1-4 sequences on one GPU: the whole step as one persistent kernel
-  bool use_mega = true;
-  bool mega_token = true;                  // greedy token picked inside the whole-step kernel (MTJ_NO_MEGA_TOKEN=1: separate kernel)
-  mtj::MegaLayer* mega_layers = nullptr;   // device copy of the per-layer pointers
-  uint32_t* mega_sync = nullptr;           // [5 L + 3] phase counters
-  unsigned long long* mega_amax = nullptr; // [4] running maxima of the in-kernel greedy token
-  unsigned long long* mega_trace = nullptr;  // [6 L + 3] phase time stamps (profiling read-out)
-  bool mega_trace_on = false;
-  // decode: attention runs on a side stream next to the FF half of the in-projection
-  bool fork_attn = true;
-  int mega_max_b = 1;               // sequences the whole-step decode kernel is used for (mtj_config.mega_max_batch, up to 4)
-  int tc_decode_min_b = 2;          // from this many sequences on decode takes the tensor-core GEMM path (mtj_config.tc_decode_min_batch)
-  bool tc_pdl = true;               // programmatic dependent launch on the tensor-core decode chain (MTJ_NO_TC_PDL=1: off)
-  bool fork_pdl = false;            // let the out-projection start early although it also waits on the side stream
-  cudaStream_t side_stream = nullptr;
-  // tensor-parallel prefill / eval: two row chunks are in flight, the all-reduce of one (on comm_stream)
-  // overlapping the layer of the other.  A view = one half of the row-indexed activation buffers.
-  struct ActView {
-    float *x, *stats, *part, *q;
-    __nv_bfloat16 *xn_bf16, *act_bf16, *q_bf16;
-    TensorMap map_xn[3], map_act[3], map_xn_wide, map_act_wide, map_q;
-  };
-  ActView views[2];
-  bool views_ok = false;
-  int view_rows[2] = {0, 0};
-  cudaStream_t comm_stream = nullptr;
-  cudaEvent_t ev_layer[2] = {nullptr, nullptr}, ev_reduced[2] = {nullptr, nullptr};
-  bool tp_pipe = false;             // overlap the all-reduce of one chunk with the layer of the next; default: from 4
-                                    // shards on (MTJ_TP_PIPE=0 / 1 overrides)
-  void save_view(int i) {
-    ActView& v = views[i];
-    v.x = x; v.stats = stats; v.part = part; v.q = q; v.xn_bf16 = xn_bf16; v.act_bf16 = act_bf16; v.q_bf16 = q_bf16;
-    for (int k = 0; k < 3; ++k) { v.map_xn[k] = map_xn[k]; v.map_act[k] = map_act[k]; }
-    v.map_xn_wide = map_xn_wide; v.map_act_wide = map_act_wide; v.map_q = map_q;
-  }
-  void use_view(int i) {
-    const ActView& v = views[i];
-    x = v.x; stats = v.stats; part = v.part; q = v.q; xn_bf16 = v.xn_bf16; act_bf16 = v.act_bf16; q_bf16 = v.q_bf16;
-    for (int k = 0; k < 3; ++k) { map_xn[k] = v.map_xn[k]; map_act[k] = v.map_act[k]; }
-    map_xn_wide = v.map_xn_wide; map_act_wide = v.map_act_wide; map_q = v.map_q;
-  }
-  cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
-
-  // decode step captured once per batch size and replayed (the step counter,
-  // tokens and page table live on the device, so the graph never changes)
-  bool use_graph = true;
-  cudaStream_t capture_stream = nullptr;
-  cudaGraphExec_t graph_exec = nullptr;
-  int graph_batch = 0;
-  int graph_greedy = -1;
-  int64_t graph_kernels = 0;
-
-  // optional per-family kernel timing (mtj_profile_*): events around launches
-  bool profile = false;
-  std::vector<cudaEvent_t> ev_pool;
-  size_t ev_used = 0;
-  std::vector<std::pair<int, std::pair<size_t, size_t>>> ev_spans;   // (family, (start, stop))
-
-  void prof_begin(int family, cudaStream_t s) {
-    if (!profile || ev_used + 2 > ev_pool.size()) return;
-    cudaEventRecord(ev_pool[ev_used], s);
-    ev_spans.push_back({family, {ev_used, ev_used + 1}});
-    ev_used += 2;
-  }
-  void prof_end(cudaStream_t s) {
-    if (!profile || ev_spans.empty()) return;
-    cudaEventRecord(ev_pool[ev_spans.back().second.second], s);
-  }
-
-  void carve_weights(Carver& c) {
-    emb_w = c.take<__nv_bfloat16>(static_cast<int64_t>(Vl) * d);
-    emb_b = c.take<float>(d);
-    layers.resize(L);
-    for (auto& lw : layers) {
-      lw.w_in = c.take<__nv_bfloat16>(static_cast<int64_t>(3 * dl + ffl) * d);
-      lw.b_ff = c.take<float>(ffl);
-      lw.w_out = c.take<__nv_bfloat16>(static_cast<int64_t>(d) * (dl + ffl));
-      lw.b_out = c.take<float>(d);
-      lw.ln_scale = c.take<float>(d);
-      lw.ln_offset = c.take<float>(d);
-    }
-    lnf_scale = c.take<float>(d);
-    lnf_offset = c.take<float>(d);
-    proj_w = c.take<__nv_bfloat16>(static_cast<int64_t>(Vl) * d);
-    proj_b = c.take<float>(Vl);
-    sincos = c.take<float2>(static_cast<int64_t>(max_pos) * (rot / 2));
-  }
-
-  void carve_workspace(Carver& c) {
-    const int64_t R = max_rows;
-    x = c.take<float>(R * d);
-    stats = c.take<float>(R * 2);
-    q = c.take<float>(R * dl);
-    act2 = c.take<float>(R * (dl + ffl));
-    part_o = c.take<float>(static_cast<int64_t>(max_batch) * heads * max_splits * dh);
-    part_ml = c.take<float>(static_cast<int64_t>(max_batch) * heads * max_splits * 2);
-    counters = c.take<uint32_t>(static_cast<int64_t>(max_batch) * heads);
-    gemv_counters = c.take<uint32_t>(R);
-    logits = c.take<float>(static_cast<int64_t>(std::max(max_batch, 1)) * Vl);
-    logits_all = logits;
-    if (mp > 1) {
-      logits_all = c.take<float>(static_cast<int64_t>(max_batch) * V);
-      logits_gather = c.take<float>(static_cast<int64_t>(max_batch) * V);
-      part = c.take<float>(R * d);
-    }
-    uniforms = c.take<float>(static_cast<int64_t>(max_batch) * V);
-    top_p = c.take<float>(max_batch);
-    temp = c.take<float>(max_batch);
-    sample_scratch = c.take<char>(mtj::sample_scratch_bytes(max_batch, V));
-    tc_partial = c.take<float>(static_cast<int64_t>(kTcSplitMax) * std::min<int64_t>(R, kTcSplitRows) * d);
-    q_bf16 = c.take<__nv_bfloat16>(R * dl);
-    xn_bf16 = c.take<__nv_bfloat16>(R * d);
-    act_bf16 = c.take<__nv_bfloat16>(R * (dl + ffl));
-    xn_lo = c.take<__nv_bfloat16>(std::min<int64_t>(R, kHiLoRows) * d);
-    act_lo = c.take<__nv_bfloat16>(std::min<int64_t>(R, kHiLoRows) * (dl + ffl));
-    eval_rows = static_cast<int>(std::min<int64_t>(R, 256));
-    eval_logits = c.take<float>(static_cast<int64_t>(eval_rows) * Vl);
-    ce_groups = 4 * ((Vl + 127) / 128);
-    ce_rows = static_cast<int>(std::min<int64_t>(R, 1024));
-    ce_gmax = c.take<float>(static_cast<int64_t>(ce_groups) * ce_rows);
-    ce_gsum = c.take<float>(static_cast<int64_t>(ce_groups) * ce_rows);
-    ce_tlogit = c.take<float>(ce_rows);
-    ce_ghit = c.take<uint8_t>(ce_rows);
-    ce_max = c.take<float>(R);
-    ce_lmax = c.take<float>(R);
-    ce_sum = c.take<float>(R * 2);
-    ce_hit = c.take<uint8_t>(R);
-    mega_layers = c.take<mtj::MegaLayer>(L);
-    mega_sync = c.take<uint32_t>(5 * L + 3);
-    mega_amax = c.take<unsigned long long>(4);
-    mega_trace = c.take<unsigned long long>(6 * L + 3);
-    tokens = c.take<uint32_t>(max_batch);
-    cur = c.take<int32_t>(4);
-    pad = c.take<int32_t>(max_batch);
-    key_limit = c.take<int32_t>(max_batch);
-    page_table = c.take<int32_t>(static_cast<int64_t>(max_batch) * ring_pages);
-    row_select = c.take<int32_t>(R);
-    dev_err = c.take<uint32_t>(4);
-    rng_seed = c.take<uint32_t>(4);
-    top_k = c.take<int32_t>(max_batch);
-    pool_layer_elems = static_cast<int64_t>(n_pages) * heads * mtj::kPageTokens * dh;
-    kpool = c.take<__nv_bfloat16>(pool_layer_elems * L);
-    vpool = c.take<__nv_bfloat16>(pool_layer_elems * L);
-  }
-
-  mtj::KvCache kv(int layer) const {
-    mtj::KvCache k;
-    k.kpool = kpool + pool_layer_elems * layer;
-    k.vpool = vpool + pool_layer_elems * layer;
-    k.page_table = page_table;
-    k.ring_pages = ring_pages;
-    k.pad = pad;
-    return k;
-  }
-};
 
 namespace {
 
@@ -819,6 +504,7 @@ int32_t run_embed(mtj_handle* h, const uint32_t* ids, int ids_ld, int M, const m
 // final LayerNorm + vocab-sharded logits for M output rows (layers.py:561-564)
 int32_t run_logits(mtj_handle* h, int M, const int32_t* row_select, float* out, bool decode,
                    cudaStream_t s, int row0 = 0) {
+  if (h->stack) return row_select ? h->stack->logits_select(h, row_select, M, out, s) : h->stack->logits(h, row0, M, out, decode, s);
   GemvArgs a = {};
   a.W = h->proj_w;
   a.N = h->Vl;
@@ -862,8 +548,9 @@ int32_t setup_sequences(mtj_handle* h, const std::vector<int32_t>& pad,
     for (int p = 0; p < h->ring_pages; ++p) table[static_cast<size_t>(b) * h->ring_pages + p] = b * h->ring_pages + p;
   MTJ_CUDA(cudaMemcpyAsync(h->pad, pad.data(), B * sizeof(int32_t), cudaMemcpyHostToDevice, s));
   MTJ_CUDA(cudaMemcpyAsync(h->key_limit, limit.data(), B * sizeof(int32_t), cudaMemcpyHostToDevice, s));
-  MTJ_CUDA(cudaMemcpyAsync(h->page_table, table.data(), table.size() * sizeof(int32_t),
-                           cudaMemcpyHostToDevice, s));
+  if (!table.empty())
+    MTJ_CUDA(cudaMemcpyAsync(h->page_table, table.data(), table.size() * sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  h->host_pad = pad;
   const int32_t c = cur;
   MTJ_CUDA(cudaMemcpyAsync(h->cur, &c, sizeof(int32_t), cudaMemcpyHostToDevice, s));
   // the host vectors above are pageable: the copies are staged before returning
@@ -921,8 +608,9 @@ int32_t forward_chunks(mtj_handle* h, const uint32_t* ids, int ids_ld, int batch
         const Chunk& c = chunks[i + k];
         mtj::RowMap rows = {c.b0, c.tc, c.t0, nullptr};
         const int M = c.ns * c.tc;
-        rc = run_embed(h, ids, ids_ld, M, rows, false, s);
-        for (int l = 0; l < h->L && !rc; ++l)
+        rc = h->stack ? h->stack->forward(h, ids, ids_ld, rows, M, rows, c.t0 - t_begin, false, s)
+                      : run_embed(h, ids, ids_ld, M, rows, false, s);
+        for (int l = 0; l < h->L && !rc && !h->stack; ++l)
           rc = use_tc(h, M) ? run_layer_tc(h, l, M, rows, key_limit, s) : run_layer(h, l, M, rows, false, key_limit, s);
         if (!rc) rc = after_chunk(c.b0, c.ns, c.t0, c.tc);
       }
@@ -962,13 +650,56 @@ int32_t forward_chunks(mtj_handle* h, const uint32_t* ids, int ids_ld, int batch
   return rc;
 }
 
+// the decode fields of the configuration and the environment switches
+void read_switches(mtj_handle* h, const mtj_config& c) {
+  const char* e = getenv("MTJ_NO_PDL");
+  h->use_pdl = !(e && e[0] == '1');
+  e = getenv("MTJ_NO_MEGA");
+  h->use_mega = !(e && e[0] == '1');
+  h->mega_token = !getenv("MTJ_NO_MEGA_TOKEN");
+  if (c.mega_max_batch != 0) h->mega_max_b = std::max(0, c.mega_max_batch);
+  if (c.tc_decode_min_batch > 0) h->tc_decode_min_b = c.tc_decode_min_batch;
+  if (c.hilo_max_batch != 0) h->tc_hilo_max_b = std::max(0, std::min(kHiLoRows, c.hilo_max_batch));
+  if (c.wait_limit > 0) h->wait_limit = c.wait_limit;
+  e = getenv("MTJ_NO_TC_PDL");
+  h->tc_pdl = !(e && e[0] == '1');
+  e = getenv("MTJ_NO_MEGA_PUSH");
+  h->mega_push = !(e && e[0] == '1');
+  // measured on one box: the fused push exchange loses 6 % of a 32-sequence step at 2 shards and wins 12 % at 4
+  // (the pull all-reduce reads every peer's slot, which grows with the shard count; the push does not)
+  h->tp_push = h->mp >= 4;
+  e = getenv("MTJ_TP_PUSH");
+  if (e) h->tp_push = e[0] == '1';
+  e = getenv("MTJ_NO_TP_TOKEN");
+  h->tp_token = !(e && e[0] == '1');
+  e = getenv("MTJ_NO_CLUSTER_K");
+  h->tc_cluster_k = !(e && e[0] == '1');
+  e = getenv("MTJ_NO_FUSED_CE");
+  h->fused_ce = !(e && e[0] == '1');
+  e = getenv("MTJ_NO_FORK");
+  h->fork_attn = !(e && e[0] == '1');
+  e = getenv("MTJ_FORK_PDL");
+  h->fork_pdl = e && e[0] == '1';
+  e = getenv("MTJ_KS_INPROJ");
+  if (e) h->ks_inproj = atoi(e);
+  e = getenv("MTJ_KS_OUT");
+  if (e) h->ks_out = atoi(e);
+  e = getenv("MTJ_KS_LOGITS");
+  if (e) h->ks_logits = atoi(e);
+  e = getenv("MTJ_NO_GRAPH");
+  h->use_graph = !(e && e[0] == '1');
+}
+
 }  // namespace
 
 extern "C" {
 
 const char* mtj_last_error(void) { return g_last_error.c_str(); }
-int32_t mtj_set_error(int32_t code, const char* msg) { return fail(code, msg ? msg : ""); }
-int32_t mtj_version(void) { return 3; }
+int32_t mtj_set_error(int32_t code, const char* msg) {
+  g_last_error = msg ? msg : "";
+  return code;
+}
+int32_t mtj_version(void) { return 4; }
 
 int32_t mtj_create(const mtj_config* c, mtj_handle** out) {
   if (!c || !out) return fail(MTJ_ERR_INVALID, "null argument");
@@ -1016,49 +747,43 @@ int32_t mtj_create(const mtj_config* c, mtj_handle** out) {
   h->n_pages = h->ring_pages * h->max_batch;
   h->max_splits = mtj::decode_attn_splits(h->W);
   h->expected = 2 + 10LL * h->L + 4;
-  const char* e = getenv("MTJ_NO_PDL");
-  h->use_pdl = !(e && e[0] == '1');
-  e = getenv("MTJ_NO_MEGA");
-  h->use_mega = !(e && e[0] == '1');
-  h->mega_token = !getenv("MTJ_NO_MEGA_TOKEN");
-  if (c->mega_max_batch != 0) h->mega_max_b = std::max(0, c->mega_max_batch);
-  if (c->tc_decode_min_batch > 0) h->tc_decode_min_b = c->tc_decode_min_batch;
-  if (c->hilo_max_batch != 0) h->tc_hilo_max_b = std::max(0, std::min(kHiLoRows, c->hilo_max_batch));
-  if (c->wait_limit > 0) h->wait_limit = c->wait_limit;
-  e = getenv("MTJ_NO_TC_PDL");
-  h->tc_pdl = !(e && e[0] == '1');
-  e = getenv("MTJ_NO_MEGA_PUSH");
-  h->mega_push = !(e && e[0] == '1');
-  // measured on one box: the fused push exchange loses 6 % of a 32-sequence step at 2 shards and wins 12 % at 4
-  // (the pull all-reduce reads every peer's slot, which grows with the shard count; the push does not)
-  h->tp_push = mp >= 4;
-  e = getenv("MTJ_TP_PUSH");
-  if (e) h->tp_push = e[0] == '1';
-  e = getenv("MTJ_NO_TP_TOKEN");
-  h->tp_token = !(e && e[0] == '1');
-  e = getenv("MTJ_NO_CLUSTER_K");
-  h->tc_cluster_k = !(e && e[0] == '1');
-  e = getenv("MTJ_NO_FUSED_CE");
-  h->fused_ce = !(e && e[0] == '1');
-  e = getenv("MTJ_NO_FORK");
-  h->fork_attn = !(e && e[0] == '1');
-  e = getenv("MTJ_FORK_PDL");
-  h->fork_pdl = e && e[0] == '1';
-  e = getenv("MTJ_KS_INPROJ");
-  if (e) h->ks_inproj = atoi(e);
-  e = getenv("MTJ_KS_OUT");
-  if (e) h->ks_out = atoi(e);
-  e = getenv("MTJ_KS_LOGITS");
-  if (e) h->ks_logits = atoi(e);
-  e = getenv("MTJ_NO_GRAPH");
-  h->use_graph = !(e && e[0] == '1');
+  read_switches(h, *c);
+  *out = h;
+  return MTJ_OK;
+}
 
+int32_t mtj_create_stack(const mtj_config* c, const mtj_stack_desc* desc, mtj_handle** out) {
+  if (!c || !desc || !out) return fail(MTJ_ERR_INVALID, "null argument");
+  if (c->d_model <= 0 || c->n_vocab <= 0 || c->seq < 2) return fail(MTJ_ERR_INVALID, "non-positive config value");
+  if (c->cores_per_replica != 1 || c->rank != 0)
+    return fail(MTJ_ERR_UNSUPPORTED, "layer-stack models run on one GPU (cores_per_replica 1)");
+  if (c->max_batch <= 0 || c->max_gen < 0 || c->max_rows <= 0) return fail(MTJ_ERR_INVALID, "bad capacity");
+  const int64_t max_pos = static_cast<int64_t>(c->seq) + c->max_gen + 1;
+  if (max_pos > (1 << 24)) return fail(MTJ_ERR_INVALID, "seq + max_gen is too large");
+  mtj::LayerStack* stack = nullptr;
+  const int32_t rc = mtj::LayerStack::create(*c, *desc, static_cast<int>(max_pos), &stack);
+  if (rc) return rc;
+  mtj_handle* h = new mtj_handle();
+  h->stack = stack;
+  h->cfg = *c;
+  h->L = desc->n_layers;
+  h->d = c->d_model;
+  h->V = h->Vl = c->n_vocab;
+  h->seq = c->seq;
+  h->W = c->seq - 1;
+  h->mp = 1;
+  h->max_batch = c->max_batch;
+  h->max_gen = c->max_gen;
+  h->max_rows = c->max_rows;
+  h->max_pos = static_cast<int>(max_pos);
+  read_switches(h, *c);
   *out = h;
   return MTJ_OK;
 }
 
 int32_t mtj_destroy(mtj_handle* h) {
   if (h) {
+    delete h->stack;
     for (cudaEvent_t e : h->ev_pool) cudaEventDestroy(e);
     if (h->graph_exec) cudaGraphExecDestroy(h->graph_exec);
     if (h->ev_fork) cudaEventDestroy(h->ev_fork);
@@ -1083,7 +808,8 @@ int64_t mtj_weights_bytes(const mtj_handle* h) {
   if (!h) return -1;
   mtj_handle tmp = *h;
   Carver c(nullptr);
-  tmp.carve_weights(c);
+  if (h->stack) mtj::LayerStack(*h->stack).carve_weights(c);
+  else tmp.carve_weights(c);
   return align_up(c.off, 256);
 }
 
@@ -1091,7 +817,12 @@ int64_t mtj_workspace_bytes(const mtj_handle* h) {
   if (!h) return -1;
   mtj_handle tmp = *h;
   Carver c(nullptr);
-  tmp.carve_workspace(c);
+  if (h->stack) {
+    tmp.carve_common(c);
+    mtj::LayerStack(*h->stack).carve_workspace(c);
+  } else {
+    tmp.carve_workspace(c);
+  }
   return align_up(c.off, 256);
 }
 
@@ -1104,6 +835,18 @@ int32_t mtj_bind_arenas(mtj_handle* h, void* wdev, int64_t wbytes, void* sdev, i
     return fail(MTJ_ERR_INVALID, "arena too small");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   Carver cw(wdev), cs(sdev);
+  if (h->stack) {
+    h->carve_common(cs);
+    h->stack->carve_weights(cw);
+    h->stack->carve_workspace(cs);
+    MTJ_CUDA(cudaMemsetAsync(h->dev_err, 0, sizeof(uint32_t) * 4, s));
+    MTJ_CUDA(cudaMemsetAsync(h->rng_seed, 0, sizeof(uint32_t) * 4, s));
+    const int32_t rc = h->stack->bind(h, s);
+    if (rc) return rc;
+    h->bound = true;
+    h->leaf_loaded.assign(static_cast<size_t>(h->expected), 0);
+    return MTJ_OK;
+  }
   h->carve_weights(cw);
   h->carve_workspace(cs);
   // RoPE angles in double precision like the reference's NumPy table (layers.py:128-134)
@@ -1229,6 +972,10 @@ int32_t mtj_load_param(mtj_handle* h, const char* name, const void* src, int32_t
   if (!h->bound) return fail(MTJ_ERR_STATE, "arenas not bound");
   if (dtype != MTJ_F32 && dtype != MTJ_BF16) return fail(MTJ_ERR_INVALID, "dtype");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (h->stack) {
+    const char* leaf = strrchr(name, '/');
+    return h->stack->load_param(h, leaf ? leaf + 1 : name, src, dtype, ndim, shape, s);
+  }
   // tokens of the Haiku path, "~" and the top-level module name dropped
   std::vector<std::string> tok;
   {
@@ -1473,16 +1220,107 @@ int32_t mtj_admit(mtj_handle* h, int32_t slot, const uint32_t* prompt, int32_t l
   MTJ_CUDA(cudaMemcpyAsync(h->pad + slot, &padv, sizeof(int32_t), cudaMemcpyHostToDevice, s));
   MTJ_CUDA(cudaMemcpyAsync(h->key_limit + slot, &lim, sizeof(int32_t), cudaMemcpyHostToDevice, s));
   MTJ_CUDA(cudaMemcpyAsync(h->tokens + slot, prompt + n, sizeof(uint32_t), cudaMemcpyDeviceToDevice, s));
+  h->host_pad[slot] = pos0;
   h->xn_ready = false;
   for (int t0 = 0; t0 < n && !rc; t0 += h->max_rows) {
     const int M = std::min(h->max_rows, n - t0);
     const mtj::RowMap ids_rows = {0, M, 0, nullptr};                  // the prompt is a flat id array
     const mtj::RowMap rows = {slot, M, pos0 + t0, nullptr};
+    if (h->stack) {
+      rc = h->stack->forward(h, prompt + t0, 0, ids_rows, M, rows, t0, false, s);
+      continue;
+    }
     rc = run_embed(h, prompt + t0, 0, M, ids_rows, false, s);
     for (int l = 0; l < h->L && !rc; ++l)
       rc = use_tc(h, M) ? run_layer_tc(h, l, M, rows, nullptr, s) : run_layer(h, l, M, rows, false, nullptr, s);
   }
   return rc;
+}
+
+int32_t mtj_extend(mtj_handle* h, int32_t slot, const uint32_t* tokens, int32_t len, const int32_t* want, int32_t n_want,
+                   float* logits_out, mtj_stream stream) {
+  int32_t rc = check_ready(h);
+  if (rc) return rc;
+  if (!h->stack) return fail(MTJ_ERR_UNSUPPORTED, "mtj_extend is for layer-stack models");
+  if (!h->prefilled) return fail(MTJ_ERR_STATE, "no running batch (mtj_start_batch or mtj_prefill first)");
+  if (!tokens || slot < 0 || slot >= h->batch || len < 1) return fail(MTJ_ERR_INVALID, "bad slot or tokens");
+  if (n_want < 0 || (n_want > 0 && (!want || !logits_out))) return fail(MTJ_ERR_INVALID, "bad want list");
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= len) return fail(MTJ_ERR_INVALID, "want outside the tokens");
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  // the tokens take the positions right before the batch's current one, like an admitted prompt; the sequence's start
+  // moves back by as many
+  const int cur = h->W + h->steps_done;
+  const int have = cur - h->host_pad[slot];
+  if (have + len > h->max_pos) return fail(MTJ_ERR_STATE, "the sequence has used up its positions (seq + max_gen)");
+  const int32_t padv = h->host_pad[slot] - len;
+  h->host_pad[slot] = padv;
+  MTJ_CUDA(cudaMemcpyAsync(h->pad + slot, &padv, sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  std::vector<int32_t> sel;
+  for (int t0 = 0; t0 < len; t0 += h->max_rows) {
+    const int M = std::min(h->max_rows, len - t0);
+    const mtj::RowMap ids_rows = {0, M, 0, nullptr};
+    const mtj::RowMap rows = {slot, M, cur - len + t0, nullptr};
+    rc = h->stack->forward(h, tokens + t0, 0, ids_rows, M, rows, have + t0, M == 1, s);
+    if (rc) return rc;
+    // runs of wanted places of this chunk, in the order they were asked for
+    for (int i = 0; i < n_want;) {
+      int j = i;
+      sel.clear();
+      while (j < n_want && want[j] >= t0 && want[j] < t0 + M) sel.push_back(want[j++] - t0);
+      if (j == i) {
+        ++i;
+        continue;
+      }
+      for (size_t k = 0; k < sel.size(); k += h->max_rows) {
+        const int n = static_cast<int>(std::min<size_t>(h->max_rows, sel.size() - k));
+        MTJ_CUDA(cudaMemcpyAsync(h->row_select, sel.data() + k, n * sizeof(int32_t), cudaMemcpyHostToDevice, s));
+        rc = h->stack->logits_select(h, h->row_select, n, logits_out + (static_cast<size_t>(i) + k) * h->V, s);
+        if (rc) return rc;
+      }
+      i = j;
+    }
+  }
+  return MTJ_OK;
+}
+
+int32_t mtj_release(mtj_handle* h, int32_t slot, mtj_stream stream) {
+  int32_t rc = check_ready(h);
+  if (rc) return rc;
+  if (!h->stack) return fail(MTJ_ERR_UNSUPPORTED, "mtj_release is for layer-stack models");
+  if (!h->prefilled || slot < 0 || slot >= h->batch) return fail(MTJ_ERR_INVALID, "bad slot");
+  // a sequence that starts at the current position holds nothing: caches are read from its start on and states begin
+  // at zero there
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const int32_t padv = h->W + h->steps_done, zero = 0;
+  h->host_pad[slot] = padv;
+  MTJ_CUDA(cudaMemcpyAsync(h->pad + slot, &padv, sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  MTJ_CUDA(cudaMemcpyAsync(h->tokens + slot, &zero, sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  return MTJ_OK;
+}
+
+int32_t mtj_k_stack_residual(mtj_handle* h, const uint32_t* tokens, int32_t len, int32_t n_runs, float* out,
+                             mtj_stream stream) {
+  int32_t rc = check_ready(h);
+  if (rc) return rc;
+  if (!h->stack) return fail(MTJ_ERR_UNSUPPORTED, "mtj_k_stack_residual is for layer-stack models");
+  if (!tokens || !out || len < 1 || len > h->max_rows || len > h->max_pos || n_runs < 1 || n_runs > h->stack->runs())
+    return fail(MTJ_ERR_INVALID, "bad argument");
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const std::vector<int32_t> pad(1, 0), limit(1, 0x7fffffff);
+  rc = setup_sequences(h, pad, limit, len, s);
+  if (rc) return rc;
+  h->prefilled = false;
+  const mtj::RowMap rows = {0, len, 0, nullptr};
+  h->stack->stop_after = n_runs;
+  rc = h->stack->forward(h, tokens, 0, rows, len, rows, 0, len == 1, s);
+  h->stack->stop_after = 0;
+  if (rc) return rc;
+  int ld = 0;
+  const float* x = h->stack->residual(&ld);
+  MTJ_CUDA(cudaMemcpy2DAsync(out, sizeof(float) * h->d, x, sizeof(float) * ld, sizeof(float) * h->d, len,
+                             cudaMemcpyDeviceToDevice, s));
+  return MTJ_OK;
 }
 
 int32_t mtj_decode_step(mtj_handle* h, const uint32_t* tokens_in, const float* top_p, const float* temp,
@@ -1492,6 +1330,8 @@ int32_t mtj_decode_step(mtj_handle* h, const uint32_t* tokens_in, const float* t
   if (rc) return rc;
   if (!h->prefilled) return fail(MTJ_ERR_STATE, "mtj_prefill has not run");
   if (h->steps_done >= h->max_gen) return fail(MTJ_ERR_STATE, "max_gen steps already generated");
+  if (h->stack && h->W + h->steps_done - *std::min_element(h->host_pad.begin(), h->host_pad.end()) >= h->max_pos)
+    return fail(MTJ_ERR_STATE, "a sequence has used up its positions (seq + max_gen)");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int B = h->batch;
   if (!greedy) {
@@ -1506,12 +1346,14 @@ int32_t mtj_decode_step(mtj_handle* h, const uint32_t* tokens_in, const float* t
   auto enqueue = [&](cudaStream_t st) -> int32_t {
     mtj::RowMap rows = {0, 1, 0, h->cur};
     mtj::RowMap erows = {0, 1, 0, nullptr};
-    const bool mega = h->use_mega && (h->mp == 1 || use_p2p(h, B)) && B <= h->mega_max_b && !h->profile && (h->d % 256) == 0;
+    const bool mega = h->use_mega && !h->stack && (h->mp == 1 || use_p2p(h, B)) && B <= h->mega_max_b && !h->profile && (h->d % 256) == 0;
     const bool tc = use_tc_decode(h, B);
     h->xn_ready = false;
     // one GPU, greedy: the persistent kernel also picks the token and advances the position
     const bool mega_token = mega && greedy && h->mp == 1 && h->mega_token;
-    int32_t r = mega ? MTJ_OK : run_embed(h, h->tokens, 1, B, erows, true, st, tc);
+    int32_t r = MTJ_OK;
+    if (h->stack) r = h->stack->forward(h, h->tokens, 1, erows, B, rows, 0, true, st);
+    else if (!mega) r = run_embed(h, h->tokens, 1, B, erows, true, st, tc);
     if (r) return r;
     if (mega) {
       mtj::MegaArgs ma = {};
@@ -1551,7 +1393,7 @@ int32_t mtj_decode_step(mtj_handle* h, const uint32_t* tokens_in, const float* t
       MTJ_CUDA(mtj::launch_decode_mega(ma, st, nullptr));
       h->launches++;
     }
-    for (int l = 0; !mega && l < h->L; ++l) {
+    for (int l = 0; !mega && !h->stack && l < h->L; ++l) {
       r = tc ? run_layer_tc(h, l, B, rows, nullptr, st, nullptr, true) : run_layer(h, l, B, rows, true, nullptr, st);
       if (r) return r;
     }
@@ -1664,7 +1506,7 @@ int32_t mtj_forward_logits(mtj_handle* h, const uint32_t* obs, const uint32_t* c
   if (rc) return rc;
   if (h->mp > 1 && !h->comm) return fail(MTJ_ERR_STATE, "cores_per_replica > 1 needs mtj_comm_init first");
   if (!obs || !logits_out || batch <= 0 || batch > h->max_batch) return fail(MTJ_ERR_INVALID, "bad batch");
-  if (T <= 0 || T > h->ring_pages * mtj::kPageTokens || T > h->max_pos)
+  if (T <= 0 || (!h->stack && T > h->ring_pages * mtj::kPageTokens) || T > h->max_pos)
     return fail(MTJ_ERR_INVALID, "T exceeds the KV capacity");
   if (n_last <= 0 || n_last > T) return fail(MTJ_ERR_INVALID, "bad n_last");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -1708,7 +1550,7 @@ int32_t mtj_eval_loss(mtj_handle* h, const uint32_t* obs, const uint32_t* target
   if (h->mp > 1 && !h->comm) return fail(MTJ_ERR_STATE, "cores_per_replica > 1 needs mtj_comm_init first");
   if (!obs || !target || !all_loss || !correct || batch <= 0 || batch > h->max_batch)
     return fail(MTJ_ERR_INVALID, "bad argument");
-  if (T <= 0 || T > h->ring_pages * mtj::kPageTokens || T > h->max_pos)
+  if (T <= 0 || (!h->stack && T > h->ring_pages * mtj::kPageTokens) || T > h->max_pos)
     return fail(MTJ_ERR_INVALID, "T exceeds the KV capacity");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   std::vector<int32_t> pad(batch, 0), limit(batch);
@@ -1828,7 +1670,7 @@ int32_t mtj_sample_top_p(const float* logits, const float* uniforms, const float
 }
 
 int32_t mtj_mega_trace(mtj_handle* h, int32_t enable, uint64_t* out, int32_t n, mtj_stream stream) {
-  if (!h || !h->bound) return fail(MTJ_ERR_STATE, "not bound");
+  if (!h || !h->bound || h->stack) return fail(MTJ_ERR_STATE, "not bound");
   if (out) {
     if (n > 6 * h->L + 3) n = 6 * h->L + 3;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -1850,7 +1692,7 @@ int64_t mtj_launch_count(const mtj_handle* h) { return h ? h->launches : -1; }
 int32_t mtj_profile_enable(mtj_handle* h, int32_t on) {
   if (!h) return fail(MTJ_ERR_INVALID, "null handle");
   if (on && h->ev_pool.empty()) {
-    h->ev_pool.resize(2 * (4 * static_cast<size_t>(h->L) + 2) * 64);
+    h->ev_pool.resize(2 * (5 * static_cast<size_t>(h->stack ? h->stack->runs() : h->L) + 2) * 64);
     for (auto& e : h->ev_pool) MTJ_CUDA(cudaEventCreate(&e));
   }
   h->profile = on != 0;
@@ -1896,6 +1738,7 @@ int32_t mtj_k_layer(mtj_handle* h, int32_t layer, const float* x_in, int32_t bat
                     mtj_stream stream) {
   int32_t rc = check_ready(h);
   if (rc) return rc;
+  if (h->stack) return fail(MTJ_ERR_UNSUPPORTED, "this unit entry point is for GPT-J handles");
   if (h->mp > 1 && !h->comm) return fail(MTJ_ERR_STATE, "cores_per_replica > 1 needs mtj_comm_init first");
   if (!x_in || !out || layer < 0 || layer >= h->L || batch <= 0 || batch > h->max_batch || T <= 0)
     return fail(MTJ_ERR_INVALID, "bad argument");
@@ -1925,6 +1768,7 @@ int32_t mtj_k_layer(mtj_handle* h, int32_t layer, const float* x_in, int32_t bat
 int32_t mtj_k_projection(mtj_handle* h, const float* x_in, int32_t rows, float* logits_out, mtj_stream stream) {
   int32_t rc = check_ready(h);
   if (rc) return rc;
+  if (h->stack) return fail(MTJ_ERR_UNSUPPORTED, "this unit entry point is for GPT-J handles");
   if (!x_in || !logits_out || rows <= 0 || rows > h->max_rows) return fail(MTJ_ERR_INVALID, "bad argument");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   MTJ_CUDA(mtj::launch_residual_stats(h->x, x_in, h->stats, rows, h->d, false, s, false));
@@ -1937,6 +1781,7 @@ int32_t mtj_k_projection_loss(mtj_handle* h, const float* x_in, const uint32_t* 
                               float* loss_out, uint8_t* correct_out, mtj_stream stream) {
   int32_t rc = check_ready(h);
   if (rc) return rc;
+  if (h->stack) return fail(MTJ_ERR_UNSUPPORTED, "this unit entry point is for GPT-J handles");
   if (h->mp > 1 && !h->comm) return fail(MTJ_ERR_STATE, "cores_per_replica > 1 needs mtj_comm_init first");
   if (!x_in || !targets || !loss_out || !correct_out || rows <= 0 || rows > h->max_rows)
     return fail(MTJ_ERR_INVALID, "bad argument");
@@ -1986,6 +1831,7 @@ int32_t mtj_k_embed(mtj_handle* h, const uint32_t* ids, int32_t rows, float* x_o
                     mtj_stream stream) {
   int32_t rc = check_ready(h);
   if (rc) return rc;
+  if (h->stack) return fail(MTJ_ERR_UNSUPPORTED, "this unit entry point is for GPT-J handles");
   if (!ids || !x_out || rows <= 0) return fail(MTJ_ERR_INVALID, "bad argument");
   mtj::EmbedArgs e = {};
   e.ids = ids;

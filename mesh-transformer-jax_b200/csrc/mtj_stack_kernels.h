@@ -1,0 +1,140 @@
+// Launchers of the layer-stack kernels: row norms, latent attention, selective scan (internal to libmtj_b200).
+//
+// Positions.  A row m of a call sits at frame position rows.pos0 + m % Tc of sequence rows.b0 + m / Tc (RowMap); the
+// position inside its own sequence, which these kernels use, is that minus pad[sequence].  Rows before the
+// sequence's start (left padding of a batched prompt) have a negative own position: they store nothing in caches and
+// states and give finite values.
+#pragma once
+#include "mtj_kernels.h"
+
+namespace mtj {
+
+template <typename K, typename... A>
+cudaError_t launch_pdl(K kernel, dim3 grid, dim3 block, size_t smem, cudaStream_t s, bool pdl, A... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl ? 1 : 0;
+  return cudaLaunchKernelEx(&cfg, kernel, args...);
+}
+
+// ---- mtj_stack_kernels.cu
+// One row per block:  y = sum of the planes;  x += mult * RMSNorm(y) * w_post (y may be null);  then, of the new x:
+// stats = (0, 1 / rms), xn = RMSNorm(x) * w_next in bf16, and cat = [x | x0] for the projection at the start of a pass.
+struct ResidualNormArgs {
+  float* x;                    // [M, ld]; columns d .. ld - 1 of every buffer here are zero
+  int M, d, ld;
+  const float* y;              // [planes, M, ld] or null
+  int planes;
+  const float* w_post;         // [ld]
+  float mult, eps;
+  float* stats;                // [M, 2] or null
+  const float* w_next;         // [ld], with xn
+  __nv_bfloat16* xn;           // [M, ld] or null
+  const float* x0;             // [M, ld], with cat_*
+  float* cat_f32;              // [M, 2 ld] or null
+  __nv_bfloat16* cat_bf16;     // [M, 2 ld] or null
+};
+cudaError_t launch_residual_norm(const ResidualNormArgs& a, cudaStream_t s, bool pdl);
+cudaError_t launch_gather_rows_bf16(const __nv_bfloat16* src, int ld, const int32_t* rows, int n, __nv_bfloat16* dst,
+                                    cudaStream_t s);
+// src [N, K] (bf16 or fp32) -> bf16 dst[(r0 + n / gin * gout + n % gin) * ld + (k < csplit ? k : k + cshift)]
+cudaError_t launch_pack_rows(const void* src, int src_is_bf16, int N, int K, __nv_bfloat16* dst, int ld, int r0, int gin,
+                             int gout, int csplit, int cshift, cudaStream_t s);
+// fp32 dst[i] = -exp(src[i])
+cudaError_t launch_neg_exp(const void* src, int src_is_bf16, int64_t n, float* dst, cudaStream_t s);
+// src [N, K] -> fp32 dst [K, ld]
+cudaError_t launch_transpose_f32(const void* src, int src_is_bf16, int N, int K, float* dst, int ld, cudaStream_t s);
+// y[m] (+)= x[m] elementwise copies of fp32 rows
+cudaError_t launch_copy_rows(const float* src, float* dst, int64_t n, cudaStream_t s, bool pdl);
+
+// ---- mtj_latent_attn.cu: attention over a cached latent (and one rotated key part) shared by all heads
+struct LatentCache {
+  void* pool;                  // [pages][kPageTokens][row_ld] bf16 or fp32: latent (kv_ld columns) | rotated part
+  int f32;                     // element type of the pool
+  const int32_t* page_table;   // [sequences][ring_pages]; ring slot of own position p: (p / kPageTokens) % ring_pages
+  int ring_pages, row_ld, kv_ld;
+};
+struct LatentArgs {
+  int M, heads, dim, rot, vdim, rank, window;
+  float scale, eps;
+  RowMap rows;
+  const int32_t* pad;
+  LatentCache cache;
+  const float2* sincos;        // [positions][rot / 2] = (sin, cos)
+  const float* p1;             // [M, ld_p1] fp32: q head by head [dim | rot], then latent | rotated part
+  int ld_p1;
+  const float* kv_norm;        // [rank]
+  const __nv_bfloat16* w_uk;   // [heads * dim, kv_ld]
+  const __nv_bfloat16* w_uv;   // [heads * vdim, kv_ld]
+  // absorbed form (few rows, fp32 runs): q' = W_uk^T q, scores against the latent itself
+  float* q_abs;                // [M, heads, row_ld], scaled
+  int splits;                  // key ranges per row
+  float* part_o;               // [M, heads, splits, kv_ld]
+  float* part_ml;              // [M, heads, splits, 2]
+  float* out;                  // [M, ld_out] or null
+  __nv_bfloat16* out_bf16;     // [M, ld_out] or null
+  int ld_out;
+  // expanded form (many rows): operands of the tensor-core attention
+  __nv_bfloat16* q_pack;       // [M, heads * 64 * key_blocks]
+  int key_blocks, k_own;
+  __nv_bfloat16* c_lin;        // [sequences * key_rows, kv_ld] latents of the history and the chunk
+  __nv_bfloat16* kr_lin;       // [sequences * key_rows, kr_ld] their rotated parts, zero-padded
+  int kr_ld, hist, key_rows, nseq;
+};
+// normalises and caches the latent, rotates and caches the key part, rotates and absorbs the queries
+cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl);
+cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl);
+// merges the key ranges and applies W_uv
+cudaError_t launch_latent_out(const LatentArgs& a, cudaStream_t s, bool pdl);
+// the same caching, with the queries packed for the tensor-core attention and the latents copied to c_lin / kr_lin;
+// the second fills the history rows from the cache
+cudaError_t launch_latent_pack(const LatentArgs& a, cudaStream_t s);
+cudaError_t launch_latent_history(const LatentArgs& a, cudaStream_t s);
+constexpr int kLatentMaxRank = 1024;
+int latent_attn_splits(int window);
+
+// ---- mtj_ssm.cu: causal convolution and selective scan with carried state
+struct SsmArgs {
+  int M, inner, state, taps, dt_rank;
+  RowMap rows;
+  int nseq;                    // sequences in the call
+  const int32_t* pad;
+  const void* xz;              // [M, ld_xz] x | z (z at column z0), fp32 or bf16
+  int xz_bf16, ld_xz, z0;
+  const float* conv_w;         // [taps, ld_u]
+  const float* conv_b;         // [ld_u]
+  float* conv_state;           // [slots][taps - 1][inner]
+  float* u;                    // [M, ld_u] or null
+  __nv_bfloat16* u_bf16;       // [M, ld_u] or null
+  int ld_u;
+  const float* xp;             // [M, ld_xp] dt | B | C
+  int ld_xp;
+  __nv_bfloat16* dtr_bf16;     // [M, ld_dtr] bf16 copy of the dt part (launch_ssm_split), or null
+  int ld_dtr;
+  const float* dt_raw;         // [M, ld_u] W_dt dt, before the bias (scan)
+  const __nv_bfloat16* w_dt;   // [inner, ld_wdt] (step)
+  int ld_wdt;
+  const float* dt_b;
+  const float* A;              // [inner, state], negative
+  const float* D;
+  float* ssm_state;            // [slots][inner][state]
+  float* out;                  // [M, ld_u] or null
+  __nv_bfloat16* out_bf16;     // [M, ld_u] or null
+};
+// u = silu(conv(x) + b) for all rows, then the taps - 1 last inputs of every sequence into conv_state
+cudaError_t launch_ssm_conv(const SsmArgs& a, cudaStream_t s, bool pdl);
+cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s);
+// the recurrence over the rows of every sequence, from and to ssm_state, with the gate
+cudaError_t launch_ssm_scan(const SsmArgs& a, cudaStream_t s);
+// one row per sequence: step size, recurrence and gate in one kernel
+cudaError_t launch_ssm_step(const SsmArgs& a, cudaStream_t s, bool pdl);
+constexpr int kSsmMaxState = 256;
+
+}  // namespace mtj

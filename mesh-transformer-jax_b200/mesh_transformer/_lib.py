@@ -9,7 +9,10 @@ import ctypes
 import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
-LIB_PATH = os.path.join(os.path.dirname(_HERE), "libmtj_b200.so")
+# the whole library, or a build of one model family's units (build.py --family), which lacks the other families'
+# entry points
+_CANDIDATES = [os.path.join(os.path.dirname(_HERE), n) for n in ("libmtj_b200.so", "libmtj_b200_stack.so")]
+LIB_PATH = os.environ.get("MTJ_LIBRARY") or next((p for p in _CANDIDATES if os.path.exists(p)), _CANDIDATES[0])
 
 MTJ_F32, MTJ_BF16 = 0, 1
 
@@ -27,6 +30,19 @@ class MtjConfig(ctypes.Structure):
         "hilo_max_batch", "mega_max_batch", "tc_decode_min_batch", "wait_limit")]
 
 
+class MtjLayerDesc(ctypes.Structure):
+    _fields_ = ([(n, ctypes.c_int32) for n in (
+        "mixer", "ff", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "inner", "state", "conv", "dt_rank")]
+        + [("scale", ctypes.c_float), ("reserved", ctypes.c_int32), ("rot_base", ctypes.c_double)])
+
+
+class MtjStackDesc(ctypes.Structure):
+    _fields_ = ([("layers", ctypes.POINTER(MtjLayerDesc))]
+                + [(n, ctypes.c_int32) for n in ("n_layers", "loop_start", "loop_stop", "loop_times")]
+                + [("residual_mult", ctypes.c_float), ("norm_eps", ctypes.c_float), ("act_f32", ctypes.c_int32),
+                   ("tc_min_rows", ctypes.c_int32)])
+
+
 def _load():
     if not os.path.exists(LIB_PATH):
         raise ImportError(
@@ -38,6 +54,10 @@ def _load():
         "mtj_last_error": (ctypes.c_char_p, []),
         "mtj_version": (i32, []),
         "mtj_create": (i32, [ctypes.POINTER(MtjConfig), ctypes.POINTER(vp)]),
+        "mtj_create_stack": (i32, [ctypes.POINTER(MtjConfig), ctypes.POINTER(MtjStackDesc), ctypes.POINTER(vp)]),
+        "mtj_extend": (i32, [vp, i32, vp, i32, ctypes.POINTER(i32), i32, vp, vp]),
+        "mtj_release": (i32, [vp, i32, vp]),
+        "mtj_k_stack_residual": (i32, [vp, vp, i32, i32, vp, vp]),
         "mtj_destroy": (i32, [vp]),
         "mtj_weights_bytes": (i64, [vp]),
         "mtj_workspace_bytes": (i64, [vp]),
@@ -78,7 +98,10 @@ def _load():
         "mtj_k_all_reduce": (i32, [vp, ctypes.POINTER(vp), i32, i32, i32, i32, vp, vp, vp, i32, vp]),
         "mtj_k_decode_attn": (i32, [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, i64, vp, i32, vp]),
     }
+    partial = not LIB_PATH.endswith("libmtj_b200.so")
     for name, (res, args) in sig.items():
+        if partial and not hasattr(lib, name):
+            continue                    # a unit entry point of another family
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args

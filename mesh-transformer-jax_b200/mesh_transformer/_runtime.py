@@ -10,13 +10,23 @@ import sys
 import numpy as np
 import torch
 
-from . import _lib
+from . import _lib, registry
 from ._lib import MtjConfig, check, lib
 
 PREFIX = "causal_transformer_shard/~/"
 
 
 def validate_config(config: dict) -> None:
+    """Raises unless the configuration is one its model family can run."""
+    registry.family(config).validate(config)
+
+
+def param_shapes(config: dict) -> dict:
+    """{module: {leaf: per-shard shape}} of a configuration."""
+    return registry.family(config).param_shapes(config)
+
+
+def _validate_gptj(config: dict) -> None:
     """The assertions / errors of the reference constructors
     (layers.py:77,172,179,238-239,552; transformer_shard.py:42)."""
     if config.get("norm", "layernorm") != "layernorm":
@@ -29,7 +39,7 @@ def validate_config(config: dict) -> None:
     assert config["n_heads"] % mp == 0
 
 
-def param_shapes(config: dict) -> dict:
+def _param_shapes_gptj(config: dict) -> dict:
     """Per-shard leaf shapes of the Haiku tree (layers.py:185,235-258,550-559)."""
     mp = config["cores_per_replica"]
     d, V, L = config["d_model"], config["n_vocab"], config["layers"]
@@ -47,6 +57,63 @@ def param_shapes(config: dict) -> dict:
     s[PREFIX + "projection_shard/~/replicated_layer_norm"] = {"scale": (d,), "offset": (d,)}
     s[PREFIX + "projection_shard/~/linear"] = {"w": (d, Vl), "b": (Vl,)}
     return s
+
+
+@registry.register("gptj")
+class GptJ:
+    """The reference's model: the family of a configuration without an ``architecture`` key."""
+    validate = staticmethod(_validate_gptj)
+    param_shapes = staticmethod(_param_shapes_gptj)
+
+    @staticmethod
+    def prepare(config):
+        return config
+
+    @staticmethod
+    def create(config, caps, handle) -> int:
+        """``caps``: the capacity and decode fields of mtj_config."""
+        d_head = config["d_model"] // config["n_heads"]
+        cfg = MtjConfig(layers=config["layers"], d_model=config["d_model"], n_heads=config["n_heads"],
+                        n_vocab=config["n_vocab"], pe_rotary_dims=config.get("pe_rotary_dims", d_head),
+                        seq=config["seq"], cores_per_replica=config["cores_per_replica"], **caps)
+        return lib.mtj_create(ctypes.byref(cfg), handle)
+
+    @staticmethod
+    def init_state(config, rank, device, seed):
+        """Random initialisation with the reference's scales (layers.py:185,
+        253-258; transformer_shard.py:35): truncated normal, std 1/sqrt(fan_in)
+        for plain Linears, 1/sqrt(n_vocab) for the table, (2/layers)/sqrt(d)
+        for the two output projections; LN scale 1, everything else 0.  Leaves
+        carry a leading axis holding this process's shard."""
+        cfg = config
+        gen = torch.Generator(device=device)
+        gen.manual_seed(seed + 1000 * rank)
+        dtype = torch.bfloat16 if "early_cast" in cfg else torch.float32
+        d, L = cfg["d_model"], cfg["layers"]
+
+        def tn(shape, std):
+            t = torch.empty((1,) + tuple(shape), dtype=torch.float32, device=device)
+            torch.nn.init.trunc_normal_(t, mean=0.0, std=std, a=-2 * std, b=2 * std, generator=gen)
+            return t.to(dtype)
+
+        params = {}
+        for mod, leaves in param_shapes(cfg).items():
+            out = {}
+            for leaf, shape in leaves.items():
+                if leaf == "scale":
+                    out[leaf] = torch.ones((1,) + shape, dtype=dtype, device=device)
+                elif leaf in ("offset", "b"):
+                    out[leaf] = torch.zeros((1,) + shape, dtype=dtype, device=device)
+                elif "embedding_shard" in mod:
+                    out[leaf] = tn(shape, 1.0 / np.sqrt(cfg["n_vocab"]))
+                elif mod.endswith("linear_3") or mod.endswith("linear_5"):
+                    out[leaf] = tn(shape, (2.0 / L) / np.sqrt(d))
+                elif mod.endswith("linear_5") or mod.endswith("linear_4") or "projection_shard" in mod \
+                        or mod.endswith("linear") or mod.endswith("linear_1") or mod.endswith("linear_2"):
+                    fan_in = shape[0] if not mod.endswith("linear_5") else shape[0] * cfg["cores_per_replica"]
+                    out[leaf] = tn(shape, 1.0 / np.sqrt(fan_in))
+            params[mod] = out
+        return {"params": params, "step": np.array(0), "opt_state": None}
 
 
 def gather_vocab_shards(local: torch.Tensor) -> torch.Tensor:
@@ -69,6 +136,7 @@ class ShardRuntime:
 
     def __init__(self, config: dict, rank: int = 0, device=None, max_batch: int = 1,
                  max_gen: int = 256, max_rows: int | None = None, **tuning):
+        config = registry.prepare(config)
         validate_config(config)
         if not torch.cuda.is_available():
             raise RuntimeError("libmtj_b200 needs a CUDA device; there is no CPU path")
@@ -77,7 +145,6 @@ class ShardRuntime:
         self.rank = rank
         self.mp = config["cores_per_replica"]
         seq = config["seq"]
-        d_head = config["d_model"] // config["n_heads"]
         if max_rows is None:
             max_rows = min(max(seq, max_batch), 4096)
         unknown = set(tuning) - set(self.TUNING)
@@ -94,12 +161,10 @@ class ShardRuntime:
                     v = -1                         # the variable's 0 has always meant "never"
             tune.append(int(v) if v is not None else 0)
         self.tuning = dict(zip(self.TUNING, tune))
-        cfg = MtjConfig(config["layers"], config["d_model"], config["n_heads"], config["n_vocab"],
-                        config.get("pe_rotary_dims", d_head), seq, self.mp, rank,
-                        max_batch, max_gen, max_rows, *tune)
+        caps = dict(self.tuning, rank=rank, max_batch=max_batch, max_gen=max_gen, max_rows=max_rows)
         self.max_batch, self.max_gen, self.max_rows = max_batch, max_gen, max_rows
         self._h = ctypes.c_void_p()
-        check(lib.mtj_create(ctypes.byref(cfg), ctypes.byref(self._h)))
+        check(registry.family(config).create(config, caps, ctypes.byref(self._h)))
         with torch.cuda.device(self.device):
             wb, sb = lib.mtj_weights_bytes(self._h), lib.mtj_workspace_bytes(self._h)
             self.weights_arena = torch.empty(wb + 256, dtype=torch.uint8, device=self.device)
@@ -199,6 +264,29 @@ class ShardRuntime:
         prompt_dev = prompt_dev.contiguous()
         check(lib.mtj_admit(self._h, slot, prompt_dev.data_ptr(), prompt_dev.numel(), self.stream))
         torch.cuda.current_stream(self.device).synchronize()       # the caller may drop ``prompt_dev``
+
+    def extend(self, slot: int, tokens_dev: torch.Tensor, want=()) -> torch.Tensor:
+        """Appends tokens ([len] int32 on the device) to the sequence in a slot of the running batch (layer-stack
+        models); returns the logits [len(want), n_vocab] at the places ``want``."""
+        tokens_dev = tokens_dev.contiguous()
+        want = [int(w) for w in want]
+        out = torch.empty((len(want), self.vocab_local), dtype=torch.float32, device=self.device)
+        arr = (ctypes.c_int32 * len(want))(*want) if want else None
+        check(lib.mtj_extend(self._h, slot, tokens_dev.data_ptr(), tokens_dev.numel(), arr, len(want),
+                             out.data_ptr() if want else None, self.stream))
+        torch.cuda.current_stream(self.device).synchronize()       # the caller may drop ``tokens_dev``
+        return out
+
+    def release(self, slot: int) -> None:
+        """Gives back what the sequence in a slot holds; the slot's next token is position 0."""
+        check(lib.mtj_release(self._h, slot, self.stream))
+
+    def stack_residual(self, tokens_dev: torch.Tensor, n_runs: int) -> torch.Tensor:
+        """Residual stream [len, width] after the first ``n_runs`` layer runs of a fresh sequence."""
+        out = torch.empty((tokens_dev.numel(), self.config["d_model"]), dtype=torch.float32, device=self.device)
+        check(lib.mtj_k_stack_residual(self._h, tokens_dev.data_ptr(), tokens_dev.numel(), n_runs, out.data_ptr(),
+                                       self.stream))
+        return out
 
     def decode_step(self, tokens_in=None, tokens_out=None, logits_out=None, greedy=True,
                     top_p=None, temp=None, uniforms=None) -> None:

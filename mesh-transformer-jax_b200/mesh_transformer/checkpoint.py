@@ -241,3 +241,49 @@ def read_ckpt(pytree, dir, shards_in, shards_out=None, load_opt=True, by_role=Fa
     if isinstance(loaded, dict) and (not load_opt or "opt_state" not in loaded):
         loaded["opt_state"] = original_opt_state
     return loaded
+
+
+# ------------------------------------------------------------- safetensors ----
+_ST_DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "F64": torch.float64,
+              "I32": torch.int32, "I64": torch.int64, "U8": torch.uint8, "I8": torch.int8}
+
+
+def read_safetensors(path: str) -> dict:
+    """{name: CPU tensor} of a safetensors file: an 8-byte little-endian header length, the JSON header (name ->
+    dtype, shape, data_offsets) and the data."""
+    import json
+    with open(path, "rb") as f:
+        head = f.read(8)
+        if len(head) != 8:
+            raise ValueError(f"{path}: not a safetensors file")
+        n = int.from_bytes(head, "little")
+        header = json.loads(f.read(n))
+        data = np.fromfile(f, dtype=np.uint8)
+    out = {}
+    for name, t in header.items():
+        if name == "__metadata__":
+            continue
+        lo, hi = t["data_offsets"]
+        dtype = _ST_DTYPES[t["dtype"]]
+        size = int(np.prod(t["shape"], dtype=np.int64)) * torch.empty((), dtype=dtype).element_size()
+        if hi - lo != size or hi > data.size:
+            raise ValueError(f"{path}: {name} has {hi - lo} bytes where its shape needs {size}")
+        out[name] = torch.from_numpy(data[lo:hi].copy()).view(dtype).reshape(t["shape"])
+    return out
+
+
+def write_safetensors(path: str, tensors: dict) -> None:
+    """The inverse of ``read_safetensors``."""
+    import json
+    names = {v: k for k, v in _ST_DTYPES.items()}
+    header, blobs, at = {}, [], 0
+    for name, t in tensors.items():
+        t = torch.as_tensor(t).detach().cpu().contiguous()
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes()
+        header[name] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
+        blobs.append(raw)
+        at += len(raw)
+    head = json.dumps(header).encode()
+    head += b" " * (-len(head) % 8)
+    with open(path, "wb") as f:
+        f.write(len(head).to_bytes(8, "little") + head + b"".join(blobs))

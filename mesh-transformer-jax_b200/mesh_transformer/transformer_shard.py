@@ -15,6 +15,7 @@ import time
 import numpy as np
 import torch
 
+from . import registry
 from ._runtime import PREFIX, ShardRuntime, param_shapes, validate_config
 from .util import head_print, to_bf16
 
@@ -32,8 +33,9 @@ class CausalTransformerShard:
     def __init__(self, config, runtime: ShardRuntime | None = None, **runtime_kw):
         validate_config(config)
         self.config = config
-        self.heads = config["n_heads"]
-        self.heads_per_shard = config["n_heads"] // config["cores_per_replica"]
+        if "n_heads" in config:                    # layer-stack models give head counts per layer
+            self.heads = config["n_heads"]
+            self.heads_per_shard = config["n_heads"] // config["cores_per_replica"]
         self.runtime = runtime if runtime is not None else ShardRuntime(config, **runtime_kw)
 
     def generate_initial(self, context_dev: torch.Tensor, length):
@@ -56,6 +58,7 @@ class CausalTransformerShard:
 
 class CausalTransformer:
     def __init__(self, config, device=None, init_weights: bool = True):
+        config = registry.prepare(config)
         self.config = config
         validate_config(config)
         rank, world = _world()
@@ -95,40 +98,8 @@ class CausalTransformer:
         self._dirty = True
 
     def _init_state(self, seed: int):
-        """Random initialisation with the reference's scales (layers.py:185,
-        253-258; transformer_shard.py:35): truncated normal, std 1/sqrt(fan_in)
-        for plain Linears, 1/sqrt(n_vocab) for the table, (2/layers)/sqrt(d)
-        for the two output projections; LN scale 1, everything else 0.  Leaves
-        carry a leading axis holding this process's shard."""
-        cfg = self.config
-        gen = torch.Generator(device=self.device)
-        gen.manual_seed(seed + 1000 * self.rank)
-        dtype = torch.bfloat16 if "early_cast" in cfg else torch.float32
-        d, L = cfg["d_model"], cfg["layers"]
-
-        def tn(shape, std):
-            t = torch.empty((1,) + tuple(shape), dtype=torch.float32, device=self.device)
-            torch.nn.init.trunc_normal_(t, mean=0.0, std=std, a=-2 * std, b=2 * std, generator=gen)
-            return t.to(dtype)
-
-        params = {}
-        for mod, leaves in param_shapes(cfg).items():
-            out = {}
-            for leaf, shape in leaves.items():
-                if leaf == "scale":
-                    out[leaf] = torch.ones((1,) + shape, dtype=dtype, device=self.device)
-                elif leaf in ("offset", "b"):
-                    out[leaf] = torch.zeros((1,) + shape, dtype=dtype, device=self.device)
-                elif "embedding_shard" in mod:
-                    out[leaf] = tn(shape, 1.0 / np.sqrt(cfg["n_vocab"]))
-                elif mod.endswith("linear_3") or mod.endswith("linear_5"):
-                    out[leaf] = tn(shape, (2.0 / L) / np.sqrt(d))
-                elif mod.endswith("linear_5") or mod.endswith("linear_4") or "projection_shard" in mod \
-                        or mod.endswith("linear") or mod.endswith("linear_1") or mod.endswith("linear_2"):
-                    fan_in = shape[0] if not mod.endswith("linear_5") else shape[0] * cfg["cores_per_replica"]
-                    out[leaf] = tn(shape, 1.0 / np.sqrt(fan_in))
-            params[mod] = out
-        return {"params": params, "step": np.array(0), "opt_state": None}
+        """Random initialisation of the configuration's model family."""
+        return registry.family(self.config).init_state(self.config, self.rank, self.device, seed)
 
     def move_xmap(self, state, _):
         """to_bf16 over the state (transformer_shard.py:250-253)."""
