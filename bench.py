@@ -611,6 +611,138 @@ def run_mtj(args):
     print(json.dumps(line), flush=True)
 
 
+# ------------------------------------------------------- layer-stack models ----
+def stack_model(d):
+    """A Keselix model with layers of a real model's proportions at width d: a state-space layer and a latent-attention
+    layer in turn, the middle two run twice."""
+    attn = {"type": "latent_attention",
+            "mixer": {"heads": d // 128, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+                      "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": 64}},
+            "mlp": {"kind": "dense", "ff": d * 11 // 4}}
+    ssm = {"type": "mamba1", "mixer": {"inner": 2 * d, "state": 16, "conv": 4, "dt_rank": d // 16}, "mlp": None}
+    return {"architecture": "Keselix", "vocab": 32768, "width": d, "layers": [ssm, attn, ssm, attn],
+            "loop": {"start": 1, "stop": 3, "times": 2}, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "seq": 2048}
+
+
+def stack_work(cfg, runs, T, window):
+    """(weight elements a decode step reads, flops of a T-token prompt without the logits) over the layer runs."""
+    from mesh_transformer.layer_stack import tensor_shapes
+    import math
+    shapes = tensor_shapes(cfg)
+    weights = sum(math.prod(v) for i in runs for k, v in shapes.items() if k.startswith(f"l{i}.") and len(v) > 1)
+    weights += cfg["loop"]["times"] * math.prod(shapes["loop.in"])
+    pairs = sum(min(t + 1, window) for t in range(T))
+    attn = sum(2 * pairs * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
+               for m in (cfg["layers"][i]["mixer"] for i in runs if cfg["layers"][i]["type"] == "latent_attention"))
+    return weights, 2 * weights * T + attn
+
+
+def run_stack(args):
+    """Keselix beside GPT-J (the closest model) at equal width and number of layer runs, one GPU, random weights:
+    prefill of one 2048-token prompt, decode of 1, 8 and 32 sequences behind such prompts, kernel families."""
+    import torch
+    import __graft_entry__ as ge
+    if args.gpus != 1:
+        raise SystemExit("--workload stack runs on one GPU")
+    ge.build()
+    from mesh_transformer._runtime import ShardRuntime
+    from mesh_transformer.transformer_shard import CausalTransformer
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    try:
+        peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+    except Exception:
+        peaks = {}
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+
+    def timed(fn):
+        torch.cuda.synchronize()
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1)
+
+    def median(xs):
+        return sorted(xs)[len(xs) // 2]
+
+    sampler = ClockSampler(0)
+    sampler.start()
+    t_wall0 = time.time()
+    T, K, W = 2048, args.steps, args.warmup
+    sizes, launches = {}, 0
+    for d in [int(v) for v in args.stack_widths.split(",")]:
+        kes = stack_model(d)
+        runs = [0, 1, 2, 1, 2, 3]
+        window = kes["layers"][1]["mixer"]["mask"]["size"]
+        gptj = dict(GPTJ_6B, layers=len(runs), d_model=d, n_heads=d // 256, n_vocab=kes["vocab"], early_cast=True)
+        row = {}
+        for name, cfg in (("keselix", kes), ("gptj", gptj)):
+            net = CausalTransformer(dict(cfg), device=device)
+            V = cfg.get("n_vocab", kes["vocab"])
+            if name == "keselix":
+                weights, flops = stack_work(cfg, runs, T - 1, window)
+                m = kes["layers"][1]["mixer"]
+                cache = 3 * window * (m["kv_rank"] + m["rot_dim"]) * 2          # three attention runs
+                cache += 3 * 2 * (2 * d * 16 * 4 + 2 * d * 3 * 4)                # three states, read and written
+            else:
+                weights = 12 * d * d * len(runs)
+                flops = 2 * weights * (T - 1) + len(runs) * 2 * d * (T - 1) * T
+                cache = len(runs) * (T - 1) * 2 * d * 2
+            weights += V * d
+            out = {"weights_read_per_step_mb": weights * 2 / 1e6}
+            for B in (1, 8, 32):
+                # every prompt twice, warm-up and K timed steps, the blocks, a profiled pass
+                rt = ShardRuntime(net.config, device=device, max_batch=B, max_gen=W + 6 * K + 64, max_rows=4096)
+                rt.load_params(net.state["params"])
+                ctx = torch.randint(0, V, (B, T), dtype=torch.int32, device=device)
+                rt.prefill(ctx, [T] * B)
+                if B == 1:
+                    rt.prefill(ctx, [T])
+                    ms = median([timed(lambda: rt.prefill(ctx, [T])) for _ in range(7)])
+                    rt.profile_enable(True)
+                    rt.prefill(ctx, [T])
+                    fam = {k: v[0] for k, v in rt.profile_read().items() if v[1]}
+                    rt.profile_enable(False)
+                    out["prefill_2048"] = {"ms": ms, "tokens_per_s": (T - 1) / ms * 1e3, "tflops": flops / ms / 1e9,
+                                           "frac_of_bf16_peak": flops / ms / 1e9 / tc, "family_ms": fam}
+                tok = torch.empty((B,), dtype=torch.int32, device=device)
+                for _ in range(max(W, 3)):
+                    rt.decode_step(None, tok)
+                n0 = rt.launch_count()
+                ms = median([timed(lambda: [rt.decode_step(None, tok) for _ in range(K)]) for _ in range(5)]) / K
+                launches += (rt.launch_count() - n0) // 5
+                rt.profile_enable(True)
+                for _ in range(8):
+                    rt.decode_step(None, tok)
+                fam = {k: v[0] / 8 for k, v in rt.profile_read().items() if v[1]}
+                rt.profile_enable(False)
+                rt.check_device_status()
+                nbytes = weights * 2 + B * cache
+                out[f"decode_b{B}"] = {"ms_per_step": ms, "tokens_per_s": B / ms * 1e3, "gbs": nbytes / ms / 1e6,
+                                       "frac_of_hbm_peak": nbytes / ms / 1e6 / hbm, "family_ms": fam,
+                                       "launches_per_step": (rt.launch_count() - n0) / (5 * K + 8)}
+                rt.close()
+                del rt
+            net.state = None
+            torch.cuda.empty_cache()
+            row[name] = out
+        sizes[str(d)] = row
+    sampler.stop()
+    top = sizes[str(args.stack_widths.split(",")[-1])]["keselix"]
+    print(json.dumps({
+        "metric": "keselix_decode_tokens_per_s", "value": top["decode_b1"]["tokens_per_s"], "unit": UNIT, "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": top["decode_b1"]["ms_per_step"], "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "gpu_launches": launches,
+        "clocks": sampler.summary(t_wall0, time.time()),
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tc, "source": "measured" if peaks else "fallback"},
+        "config": {"workload": "layer-stack model (state-space and latent-attention layers) beside GPT-J at equal width and "
+                               "number of layer runs; random weights; one 2048-token prompt, greedy decode",
+                   "l2": "every step reads more weights than L2 holds (looped layers twice)", "parallelism": "mp1"},
+        "sizes": sizes}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -620,8 +752,10 @@ def main():
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--model", default="6b", choices=["6b", "22b"],
                     help="6b: GPT-J-6B (the headline); 22b: the L48 d6144 h24 scale-up (fits 8 GPUs)")
-    ap.add_argument("--workload", default="headline", choices=["headline", "serving"],
-                    help="headline: full-window greedy decode; serving: 1024-token prompts + nucleus sampling")
+    ap.add_argument("--workload", default="headline", choices=["headline", "serving", "stack"],
+                    help="headline: full-window greedy decode; serving: 1024-token prompts + nucleus sampling; stack: a "
+                         "layer-stack model (Keselix) beside GPT-J at equal widths")
+    ap.add_argument("--stack-widths", default="2048,4096", help="widths of --workload stack")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--headline-only", action="store_true",
                     help="skip the eval 8 x 2048, serving batch-32 and (8 GPUs) 22B blocks of the JSON line")
@@ -631,6 +765,8 @@ def main():
     args = ap.parse_args()
     if args.impl == "reference":
         run_reference(args)
+    elif args.workload == "stack":
+        run_stack(args)
     else:
         run_mtj(args)
 

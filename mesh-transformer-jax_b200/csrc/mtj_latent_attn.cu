@@ -24,6 +24,14 @@ namespace {
 constexpr int kThreads = 256;
 constexpr int kHG = 8;            // heads per block (= warps)
 constexpr int kTK = 32;           // keys per tile (= lanes)
+constexpr int kAbsorbCols = 128;  // latent columns per block of the absorb kernel
+
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 __device__ __forceinline__ float la_block_sum(float v, float* red) {
   v = warp_sum(v);
@@ -59,10 +67,19 @@ template <typename T, int RT>
 __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArgs a) {
   extern __shared__ float ab_smem[];
   __shared__ float red[kThreads / 32];
+  // a thread owns 8 latent columns of the block's chunk and every dsplit-th query dimension
+  const int k0 = blockIdx.z * kAbsorbCols, cols = min(kAbsorbCols, a.cache.kv_ld - k0);
+  const int groups = cols >> 3, dsplit = kThreads / groups;
+  const int g = threadIdx.x % groups, ds = threadIdx.x / groups;
+  const __nv_bfloat16* w =
+      a.w_uk + static_cast<size_t>(blockIdx.y < a.heads ? blockIdx.y : 0) * a.dim * a.cache.kv_ld + k0 + g * 8;
+  if (blockIdx.y < a.heads && ds < dsplit)
+    for (int j = ds; j < a.dim; j += dsplit) prefetch_l2(w + static_cast<size_t>(j) * a.cache.kv_ld);
   pdl_wait();
   pdl_launch_dependents();
   const int m0 = blockIdx.x * RT, nr = min(RT, a.M - m0);
   if (blockIdx.y == a.heads) {
+    if (blockIdx.z) return;
     for (int r = 0; r < nr; ++r) {
       int seq;
       const int p = own_pos(a.rows, a.pad, m0 + r, &seq);
@@ -85,7 +102,7 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
     const int m = m0 + min(r, nr - 1);
     const float* q = a.p1 + static_cast<size_t>(m) * a.ld_p1 + h * hd;
     for (int j = threadIdx.x; j < a.dim; j += kThreads) qs[r * a.dim + j] = q[j] * a.scale;
-    if (r < nr) {
+    if (r < nr && blockIdx.z == 0) {
       int seq;
       const int p = max(own_pos(a.rows, a.pad, m, &seq), 0);
       const float2* sc = a.sincos + static_cast<size_t>(p) * (a.rot >> 1);
@@ -95,13 +112,9 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
     }
   }
   __syncthreads();
-  // a thread owns 8 latent columns and every dsplit-th query dimension
-  const int groups = a.cache.kv_ld >> 3, dsplit = kThreads / groups;
-  const int g = threadIdx.x % groups, ds = threadIdx.x / groups;
   if (ds < dsplit) {
     float acc[RT][8] = {};
-    const __nv_bfloat16* w = a.w_uk + static_cast<size_t>(h) * a.dim * a.cache.kv_ld + g * 8;
-#pragma unroll 4
+#pragma unroll 8
     for (int j = ds; j < a.dim; j += dsplit) {
       float w8[8];
       unpack8(ld_stream16(w + static_cast<size_t>(j) * a.cache.kv_ld), w8);
@@ -115,14 +128,14 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
 #pragma unroll
     for (int r = 0; r < RT; ++r)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) part[(ds * RT + r) * a.cache.kv_ld + g * 8 + e] = acc[r][e];
+      for (int e = 0; e < 8; ++e) part[(ds * RT + r) * cols + g * 8 + e] = acc[r][e];
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < nr * a.cache.kv_ld; i += kThreads) {
-    const int r = i / a.cache.kv_ld, k = i % a.cache.kv_ld;
+  for (int i = threadIdx.x; i < nr * cols; i += kThreads) {
+    const int r = i / cols, k = i % cols;
     float v = 0.f;
-    for (int d = 0; d < dsplit; ++d) v += part[(d * RT + r) * a.cache.kv_ld + k];
-    a.q_abs[(static_cast<size_t>(m0 + r) * a.heads + h) * a.cache.row_ld + k] = v;
+    for (int d = 0; d < dsplit; ++d) v += part[(d * RT + r) * cols + k];
+    a.q_abs[(static_cast<size_t>(m0 + r) * a.heads + h) * a.cache.row_ld + k0 + k] = v;
   }
 }
 
@@ -177,13 +190,17 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
   const int nv = ld / kVec;
   for (int kt = k0; kt < k1; kt += kTK) {
     __syncthreads();                                                // the tile and the weights of the last round are read
-    for (int i = threadIdx.x; i < kTK * nv; i += kThreads) {
-      const int key = i / nv, c = i % nv;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (kt + key < k1)
-        v = *reinterpret_cast<const uint4*>(static_cast<const T*>(a.cache.pool) + cache_row(a.cache, seq, kt + key) + c * kVec);
-      *reinterpret_cast<uint4*>(cs + key * tld + c * kVec) = v;
+    for (int key = warp; key < kTK; key += kThreads / 32) {           // a warp per row, all copies in flight at once
+      T* dst = cs + key * tld;
+      if (kt + key < k1) {
+        const T* src = static_cast<const T*>(a.cache.pool) + cache_row(a.cache, seq, kt + key);
+        for (int c = lane; c < nv; c += 32) cp16(smem_u32(dst + c * kVec), src + c * kVec);
+      } else {
+        for (int c = lane; c < nv; c += 32) *reinterpret_cast<uint4*>(dst + c * kVec) = make_uint4(0u, 0u, 0u, 0u);
+      }
     }
+    cp_commit();
+    cp_wait<0>();
     __syncthreads();
     float s = 0.f, s2 = 0.f;
     {
@@ -247,17 +264,215 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
   }
 }
 
+// The same for several rows at a time with bf16 caches, on the tensor cores: one block = (row, 16 MT heads, key range).
+// The heads are the M dimension of mma.m16n8k16: S[heads, 32 keys] = Q' . C^T, fp32 online softmax, O[heads, latent] +=
+// P . C from the same tile, so a cached byte is read once per 32 heads.  A warp owns NT 8-column blocks of O.  Tiles
+// come by cp.async, one ahead.  (M is the number of heads, far below the 128 rows of a tcgen05 tile, and the bound is
+// the cache traffic.)
+__device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm2(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma16816(float* d, const uint32_t* a, const uint32_t* b) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+
+template <int MT>
+constexpr size_t mma_smem_bytes(int row_ld) {
+  const size_t row = (row_ld + 15) / 16 * 16 + 8;       // an odd number of 16-byte units: conflict-free ldmatrix
+  return 2 * row * (16 * MT + 2 * kTK) + 2 * 16 * MT * 40 + 4 * (3 - MT) * 16 * MT * (kTK + 1) + 4 * 16 * MT;
+}
+
+template <int MT, int NT>
+__global__ void __launch_bounds__(kThreads) latent_attn_mma_kernel(const LatentArgs a) {
+  constexpr int HM = 16 * MT, KH = 3 - MT;               // MT == 1: two warps share a score tile, half of K each
+  constexpr int kPld = 40, kSld = kTK + 1;
+  extern __shared__ __align__(16) unsigned char lm_smem[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int ld = a.cache.row_ld, kv_ld = a.cache.kv_ld, kd = (ld + 15) & ~15, sld = kd + 8;
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(lm_smem);            // [HM][sld]
+  __nv_bfloat16* cs = qs + HM * sld;                                        // [2][kTK][sld]
+  __nv_bfloat16* ps = cs + 2 * kTK * sld;                                   // [HM][kPld]
+  float* ss = reinterpret_cast<float*>(ps + HM * kPld);                     // [KH][HM][kSld]
+  float* corr_s = ss + KH * HM * kSld;                                      // [HM]
+  const int m = blockIdx.z, h0 = blockIdx.y * HM, split = blockIdx.x;
+  pdl_wait();
+  pdl_launch_dependents();
+  int seq;
+  const int p = own_pos(a.rows, a.pad, m, &seq);
+  const int lo = max(0, p - a.window + 1), n = p - lo + 1;
+  const int per = (((max(n, 0) + a.splits - 1) / a.splits) + kTK - 1) / kTK * kTK;
+  const int k0 = lo + split * per, k1 = min(k0 + per, p + 1);
+  const int nv = ld >> 3;
+  auto fetch = [&](int kt, int b) {
+    for (int key = warp; key < kTK; key += kThreads / 32) {
+      __nv_bfloat16* dst = cs + (b * kTK + key) * sld;
+      if (kt + key < k1) {
+        const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.cache.pool) + cache_row(a.cache, seq, kt + key);
+        for (int c = lane; c < nv; c += 32) cp16(smem_u32(dst + c * 8), src + c * 8);
+      } else {
+        for (int c = lane; c < nv; c += 32) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+    cp_commit();
+  };
+  if (k0 < k1) fetch(k0, 0);
+  for (int i = threadIdx.x; i < HM * (kd >> 3); i += kThreads) {
+    const int h = i / (kd >> 3), c = i % (kd >> 3) * 8;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (h0 + h < a.heads && c < ld) {
+      const float4* q = reinterpret_cast<const float4*>(a.q_abs + (static_cast<size_t>(m) * a.heads + h0 + h) * ld + c);
+      const float4 x = q[0], y = q[1];
+      v = make_uint4(pack_bf16x2(x.x, x.y), pack_bf16x2(x.z, x.w), pack_bf16x2(y.x, y.y), pack_bf16x2(y.z, y.w));
+    }
+    *reinterpret_cast<uint4*>(qs + h * sld + c) = v;
+  }
+  if (kd > ld)                                           // the last half block of K in the key tiles
+    for (int i = threadIdx.x; i < 2 * kTK; i += kThreads) *reinterpret_cast<uint4*>(cs + i * sld + ld) = make_uint4(0u, 0u, 0u, 0u);
+
+  float acc[MT][NT][4] = {};
+  float mx[2 * MT], l[2 * MT];                           // of rows warp, warp + 8, ...
+#pragma unroll
+  for (int i = 0; i < 2 * MT; ++i) {
+    mx[i] = -INFINITY;
+    l[i] = 0.f;
+  }
+  const uint32_t q_base = smem_u32(qs), p_base = smem_u32(ps);
+  for (int kt = k0, it = 0; kt < k1; kt += kTK, ++it) {
+    const int b = it & 1;
+    const uint32_t c_base = smem_u32(cs + b * kTK * sld);
+    if (kt + kTK < k1) {
+      fetch(kt + kTK, b ^ 1);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    {
+      const int mt = MT == 2 ? warp >> 2 : 0, kh = MT == 2 ? 0 : warp >> 2, nt = warp & 3;
+      const int ks = kd >> 4, s0 = KH == 2 ? kh * (ks >> 1) : 0, s1 = KH == 2 && kh == 0 ? ks >> 1 : ks;
+      float s4[2][4] = {};
+      const uint32_t qa = q_base + 2u * ((mt * 16 + (lane & 15)) * sld + (lane >> 4) * 8);
+      const uint32_t ca = c_base + 2u * ((nt * 8 + (lane & 7)) * sld + ((lane >> 3) & 1) * 8);
+#pragma unroll 2
+      for (int k = s0; k < s1; k += 2) {                   // two chains
+        uint32_t af[4], bf[2];
+        ldsm4(af, qa + 32u * k);
+        ldsm2(bf, ca + 32u * k);
+        mma16816(s4[0], af, bf);
+        if (k + 1 < s1) {
+          ldsm4(af, qa + 32u * k + 32u);
+          ldsm2(bf, ca + 32u * k + 32u);
+          mma16816(s4[1], af, bf);
+        }
+      }
+      float* sp = ss + (kh * HM + mt * 16 + (lane >> 2)) * kSld + nt * 8 + (lane & 3) * 2;
+      sp[0] = s4[0][0] + s4[1][0];
+      sp[1] = s4[0][1] + s4[1][1];
+      sp[8 * kSld] = s4[0][2] + s4[1][2];
+      sp[8 * kSld + 1] = s4[0][3] + s4[1][3];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2 * MT; ++i) {
+      const int r = warp + 8 * i;
+      float s = ss[r * kSld + lane];
+      if (KH == 2) s += ss[(HM + r) * kSld + lane];
+      if (kt + lane >= k1) s = -INFINITY;
+      const float m_new = fmaxf(mx[i], warp_max(s));
+      const float corr = __expf(mx[i] - m_new), w = __expf(s - m_new);
+      l[i] = l[i] * corr + warp_sum(w);
+      mx[i] = m_new;
+      ps[r * kPld + lane] = __float2bfloat16_rn(w);
+      if (lane == 0) corr_s[r] = corr;
+    }
+    __syncthreads();
+    uint32_t pf[MT][2][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const float c0 = corr_s[mt * 16 + (lane >> 2)], c1 = corr_s[mt * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        acc[mt][j][0] *= c0;
+        acc[mt][j][1] *= c0;
+        acc[mt][j][2] *= c1;
+        acc[mt][j][3] *= c1;
+      }
+#pragma unroll
+      for (int k = 0; k < 2; ++k) ldsm4(pf[mt][k], p_base + 2u * ((mt * 16 + (lane & 15)) * kPld + k * 16 + (lane >> 4) * 8));
+    }
+#pragma unroll
+    for (int j = 0; j < NT; j += 2) {
+      const int col = (warp * NT + j) * 8;
+      if (col < kv_ld) {
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          uint32_t bf[4];
+          ldsm4t(bf, c_base + 2u * ((k * 16 + (lane & 15)) * sld + col + (lane >> 4) * 8));
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma16816(acc[mt][j], pf[mt][k], bf);
+            mma16816(acc[mt][j + 1], pf[mt][k], bf + 2);
+          }
+        }
+      }
+    }
+    __syncthreads();                                     // the tile may be fetched over
+  }
+  const size_t base = (static_cast<size_t>(m) * a.heads + h0) * a.splits + split;
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int col = (warp * NT + j) * 8 + (lane & 3) * 2, h = mt * 16 + (lane >> 2);
+      if (col < kv_ld) {
+        if (h0 + h < a.heads)
+          *reinterpret_cast<float2*>(a.part_o + (base + static_cast<size_t>(h) * a.splits) * kv_ld + col) = make_float2(acc[mt][j][0], acc[mt][j][1]);
+        if (h0 + h + 8 < a.heads)
+          *reinterpret_cast<float2*>(a.part_o + (base + static_cast<size_t>(h + 8) * a.splits) * kv_ld + col) = make_float2(acc[mt][j][2], acc[mt][j][3]);
+      }
+    }
+#pragma unroll
+  for (int i = 0; i < 2 * MT; ++i) {
+    const int r = warp + 8 * i;
+    if (lane == 0 && h0 + r < a.heads) {
+      float* ml = a.part_ml + 2 * (base + static_cast<size_t>(r) * a.splits);
+      ml[0] = mx[i];
+      ml[1] = l[i];
+    }
+  }
+}
+
 constexpr int kMaxSplits = 64;
+constexpr int kMmaRows = 5;       // rows from which the tensor-core form is used
 constexpr int kVC = 32;           // value rows per block
 
-template <int RT>
+// KC = 256-column chunks of a latent row; a warp owns four value rows, whose weights it has loaded before the
+// predecessor kernel is done.
+template <int RT, int KC>
 __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a) {
   extern __shared__ float lo_smem[];                     // [RT][kv_ld]
   __shared__ float ws[RT][kMaxSplits];
-  pdl_wait();
-  pdl_launch_dependents();
+  constexpr int kVW = kVC / (kThreads / 32);             // value rows per warp
   const int h = blockIdx.x, v0 = blockIdx.y * kVC, m0 = blockIdx.z * RT, nr = min(RT, a.M - m0);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, kv_ld = a.cache.kv_ld;
+  uint4 w[kVW][KC];
+#pragma unroll
+  for (int i = 0; i < kVW; ++i)
+#pragma unroll
+    for (int c = 0; c < KC; ++c) {
+      const int v = v0 + warp * kVW + i, k = c * 256 + lane * 8;
+      w[i][c] = v < a.vdim && k < kv_ld ? ld_stream16(a.w_uv + (static_cast<size_t>(h) * a.vdim + v) * kv_ld + k) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  pdl_wait();
+  pdl_launch_dependents();
   if (warp < nr) {
     const float* ml = a.part_ml + 2 * (static_cast<size_t>(m0 + warp) * a.heads + h) * a.splits;
     float mx = -INFINITY;
@@ -265,45 +480,57 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
     mx = warp_max(mx);
     float l = 0.f;
     for (int s = lane; s < a.splits; s += 32) {
-      const float w = ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - mx);
-      ws[warp][s] = w;
-      l = fmaf(w, ml[2 * s + 1], l);
+      const float e = ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - mx);
+      ws[warp][s] = e;
+      l = fmaf(e, ml[2 * s + 1], l);
     }
     l = warp_sum(l);
     const float inv = l > 0.f ? 1.0f / l : 0.f;
     for (int s = lane; s < a.splits; s += 32) ws[warp][s] *= inv;
   }
   __syncthreads();
-  for (int r = 0; r < RT; ++r) {
-    const float* po = a.part_o + (static_cast<size_t>(m0 + min(r, nr - 1)) * a.heads + h) * a.splits * kv_ld;
-    for (int k = threadIdx.x; k < kv_ld; k += kThreads) {
-      float v = 0.f;
-      for (int s = 0; s < a.splits; ++s) v = fmaf(ws[min(r, nr - 1)][s], po[static_cast<size_t>(s) * kv_ld + k], v);
-      lo_smem[r * kv_ld + k] = v;
+  const int k4 = kv_ld >> 2;
+  for (int i = threadIdx.x; i < RT * k4; i += kThreads) {
+    const int r = min(i / k4, nr - 1), k = i % k4;
+    const float4* po = reinterpret_cast<const float4*>(a.part_o + (static_cast<size_t>(m0 + r) * a.heads + h) * a.splits * kv_ld) + k;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < a.splits; ++s) {
+      const float4 p = po[static_cast<size_t>(s) * k4];
+      const float e = ws[r][s];
+      v.x = fmaf(e, p.x, v.x); v.y = fmaf(e, p.y, v.y); v.z = fmaf(e, p.z, v.z); v.w = fmaf(e, p.w, v.w);
     }
+    reinterpret_cast<float4*>(lo_smem)[i] = v;
   }
   __syncthreads();
-  for (int v = v0 + warp; v < min(v0 + kVC, a.vdim); v += kThreads / 32) {
-    const __nv_bfloat16* w = a.w_uv + (static_cast<size_t>(h) * a.vdim + v) * kv_ld;
-    float acc[RT] = {};
-    for (int k = lane * 8; k < kv_ld; k += 256) {
-      float w8[8];
-      unpack8(ld_stream16(w + k), w8);
+  for (int r = 0; r < nr; ++r) {
+    float acc[kVW] = {};
 #pragma unroll
-      for (int r = 0; r < RT; ++r) {
-        const float* o = lo_smem + r * kv_ld + k;
+    for (int c = 0; c < KC; ++c) {
+      const int k = c * 256 + lane * 8;
+      if (k < kv_ld) {
+        const float4 o0 = *reinterpret_cast<const float4*>(lo_smem + r * kv_ld + k), o1 = *reinterpret_cast<const float4*>(lo_smem + r * kv_ld + k + 4);
+        const float o[8] = {o0.x, o0.y, o0.z, o0.w, o1.x, o1.y, o1.z, o1.w};
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[r] = fmaf(w8[e], o[e], acc[r]);
+        for (int i = 0; i < kVW; ++i) {
+          float w8[8];
+          unpack8(w[i][c], w8);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[i] = fmaf(w8[e], o[e], acc[i]);
+        }
       }
     }
+    float y = 0.f;
 #pragma unroll
-    for (int r = 0; r < RT; ++r) {
-      const float y = warp_sum(acc[r]);
-      if (lane == 0 && r < nr) {
-        const size_t o = static_cast<size_t>(m0 + r) * a.ld_out + h * a.vdim + v;
-        if (a.out) a.out[o] = y;
-        if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
-      }
+    for (int i = 0; i < kVW; ++i) {
+      const float t = warp_sum(acc[i]);
+      if (lane == i) y = t;
+    }
+    const int v = v0 + warp * kVW + lane;
+    if (lane < kVW && v < a.vdim) {
+      const size_t o = static_cast<size_t>(m0 + r) * a.ld_out + h * a.vdim + v;
+      if (a.out) a.out[o] = y;
+      if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
     }
   }
 }
@@ -337,8 +564,22 @@ __global__ void __launch_bounds__(kThreads) latent_pack_kernel(const LatentArgs 
   for (int h = warp; h < a.heads; h += kThreads / 32) {
     const float* q = row + h * hd;
     __nv_bfloat16* o = a.q_pack + (static_cast<size_t>(m) * a.heads + h) * (64 * a.key_blocks);
-    for (int j = lane; j < a.dim; j += 32) o[j] = __float2bfloat16_rn(q[j]);
-    for (int j = lane; j < a.rot; j += 32) o[64 * a.k_own + j] = __float2bfloat16_rn(rotated(q + a.dim, j, sc));
+    if (((a.dim | a.rot | a.ld_p1) & 3) == 0) {
+      for (int j = 4 * lane; j < a.dim; j += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(q + j);
+        *reinterpret_cast<uint2*>(o + j) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+      }
+      for (int j = 4 * lane; j < a.rot; j += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(q + a.dim + j);
+        const float2 s0 = sc[j >> 1], s1 = sc[(j >> 1) + 1];
+        *reinterpret_cast<uint2*>(o + 64 * a.k_own + j) =
+            make_uint2(pack_bf16x2(v.x * s0.y - v.y * s0.x, v.y * s0.y + v.x * s0.x),
+                       pack_bf16x2(v.z * s1.y - v.w * s1.x, v.w * s1.y + v.z * s1.x));
+      }
+    } else {
+      for (int j = lane; j < a.dim; j += 32) o[j] = __float2bfloat16_rn(q[j]);
+      for (int j = lane; j < a.rot; j += 32) o[64 * a.k_own + j] = __float2bfloat16_rn(rotated(q + a.dim, j, sc));
+    }
   }
 }
 
@@ -372,7 +613,7 @@ cudaError_t absorb(const LatentArgs& a, cudaStream_t s, bool pdl) {
   cudaError_t e = allow_smem(once, latent_absorb_kernel<T, RT>, 160 * 1024);
   if (e != cudaSuccess) return e;
   if (smem > 160 * 1024) return cudaErrorInvalidValue;
-  return launch_pdl(latent_absorb_kernel<T, RT>, dim3((a.M + RT - 1) / RT, a.heads + 1), dim3(kThreads), smem, s, pdl, a);
+  return launch_pdl(latent_absorb_kernel<T, RT>, dim3((a.M + RT - 1) / RT, a.heads + 1, (a.cache.kv_ld + kAbsorbCols - 1) / kAbsorbCols), dim3(kThreads), smem, s, pdl, a);
 }
 
 template <typename T, int NC>
@@ -385,9 +626,29 @@ cudaError_t attend(const LatentArgs& a, cudaStream_t s, bool pdl) {
   return launch_pdl(latent_attn_kernel<T, NC>, dim3(a.splits, (a.heads + kHG - 1) / kHG, a.M), dim3(kThreads), smem, s, pdl, a);
 }
 
+template <int MT, int NT>
+cudaError_t attend_mma(const LatentArgs& a, cudaStream_t s, bool pdl) {
+  static DeviceOnce once;
+  cudaError_t e = allow_smem(once, latent_attn_mma_kernel<MT, NT>, 220 * 1024);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(latent_attn_mma_kernel<MT, NT>, dim3(a.splits, (a.heads + 16 * MT - 1) / (16 * MT), a.M), dim3(kThreads),
+                    mma_smem_bytes<MT>(a.cache.row_ld), s, pdl, a);
+}
+
+// head tiles of the tensor-core form (0: this call takes the CUDA-core form)
+int mma_head_tiles(int M, int heads, int row_ld, int kv_ld, int tensor_cores) {
+  if (!tensor_cores || M < kMmaRows || mma_smem_bytes<1>(row_ld) > 220 * 1024) return 0;
+  return heads > 16 && kv_ld <= 512 && mma_smem_bytes<2>(row_ld) <= 220 * 1024 ? 2 : 1;
+}
+
 }  // namespace
 
-int latent_attn_splits(int window) { return std::max(1, std::min(kMaxSplits, (window + 63) / 64)); }
+int latent_attn_splits(int M, int heads, int row_ld, int kv_ld, int tensor_cores, int window) {
+  const int mt = mma_head_tiles(M, heads, row_ld, kv_ld, tensor_cores);
+  const int groups = M * (mt ? (heads + 16 * mt - 1) / (16 * mt) : (heads + kHG - 1) / kHG);
+  // one wave of blocks for the tensor-core form (one per SM), four per SM for the other
+  return std::max(1, std::min({kMaxSplits, (window + kTK - 1) / kTK, (mt ? 148 : kLatentBlocks) / groups}));
+}
 
 cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a)) return cudaErrorInvalidValue;
@@ -397,6 +658,12 @@ cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl) 
 
 cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a) || a.splits < 1 || a.splits > kMaxSplits) return cudaErrorInvalidValue;
+  const int mt = mma_head_tiles(a.M, a.heads, a.cache.row_ld, a.cache.kv_ld, a.tensor_cores && !a.cache.f32);
+  if (mt) {
+    const int nt = (a.cache.kv_ld + 63) / 64;             // 8-column blocks per warp
+    if (mt == 2) return nt <= 2 ? attend_mma<2, 2>(a, s, pdl) : nt <= 4 ? attend_mma<2, 4>(a, s, pdl) : attend_mma<2, 8>(a, s, pdl);
+    return nt <= 2 ? attend_mma<1, 2>(a, s, pdl) : nt <= 4 ? attend_mma<1, 4>(a, s, pdl) : nt <= 8 ? attend_mma<1, 8>(a, s, pdl) : attend_mma<1, 16>(a, s, pdl);
+  }
   const bool two = a.cache.kv_ld > 2 * kThreads;
   if (a.cache.f32) return two ? attend<float, 2>(a, s, pdl) : attend<float, 1>(a, s, pdl);
   return two ? attend<__nv_bfloat16, 2>(a, s, pdl) : attend<__nv_bfloat16, 1>(a, s, pdl);
@@ -404,11 +671,12 @@ cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl) {
 
 cudaError_t launch_latent_out(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a) || a.splits < 1 || a.splits > kMaxSplits) return cudaErrorInvalidValue;
-  const int chunks = (a.vdim + kVC - 1) / kVC;
-  if (a.M == 1)
-    return launch_pdl(latent_out_kernel<1>, dim3(a.heads, chunks, 1), dim3(kThreads), sizeof(float) * a.cache.kv_ld, s, pdl, a);
-  return launch_pdl(latent_out_kernel<4>, dim3(a.heads, chunks, (a.M + 3) / 4), dim3(kThreads),
-                    sizeof(float) * 4 * a.cache.kv_ld, s, pdl, a);
+  const int chunks = (a.vdim + kVC - 1) / kVC, kc = (a.cache.kv_ld + 255) / 256;
+  auto go = [&](auto kernel, int rt) {
+    return launch_pdl(kernel, dim3(a.heads, chunks, (a.M + rt - 1) / rt), dim3(kThreads), sizeof(float) * rt * a.cache.kv_ld, s, pdl, a);
+  };
+  if (a.M == 1) return kc == 1 ? go(latent_out_kernel<1, 1>, 1) : kc == 2 ? go(latent_out_kernel<1, 2>, 1) : go(latent_out_kernel<1, 4>, 1);
+  return kc == 1 ? go(latent_out_kernel<8, 1>, 8) : kc == 2 ? go(latent_out_kernel<8, 2>, 8) : go(latent_out_kernel<8, 4>, 8);
 }
 
 cudaError_t launch_latent_pack(const LatentArgs& a, cudaStream_t s) {

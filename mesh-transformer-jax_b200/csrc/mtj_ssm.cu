@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
   if (c >= a.inner) return;
   const SeqSpan sp = seq_span(a, blockIdx.z);
   const T* x = static_cast<const T*>(a.xz);
-  const float* old = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.inner + c;
+  const float* old = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.ld_u + c;
   const float bias = a.conv_b[c];
   const int t0 = blockIdx.y * kConvRows, base = blockIdx.z * a.rows.Tc;
   for (int t = t0; t < min(t0 + kConvRows, a.rows.Tc); ++t) {
@@ -53,7 +53,7 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
         const int back = a.taps - 1 - j;                  // rows back from the current one
         float xv;
         if (rel >= back) xv = ld(x, static_cast<size_t>(row - back) * a.ld_xz + c);
-        else if (sp.start + rel >= back) xv = old[static_cast<size_t>(a.taps - 1 + rel - back) * a.inner];
+        else if (sp.start + rel >= back) xv = old[static_cast<size_t>(a.taps - 1 + rel - back) * a.ld_u];
         else continue;                                    // before the sequence: zero
         v = fmaf(a.conv_w[static_cast<size_t>(j) * a.ld_u + c], xv, v);
       }
@@ -62,6 +62,74 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
     const size_t o = static_cast<size_t>(row) * a.ld_u + c;
     if (a.u) a.u[o] = v;
     if (a.u_bf16) a.u_bf16[o] = __float2bfloat16_rn(v);
+  }
+}
+
+// The same for at most four taps, a thread owning eight neighbouring channels: it walks kVecRows rows with the last
+// TAPS - 1 inputs in registers, one 16-byte load per row.  Columns between inner and the row stride hold zeros.
+constexpr int kVecRows = 16;
+
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float* f) { unpack8(*reinterpret_cast<const uint4*>(p), f); }
+__device__ __forceinline__ void ld8(const float* p, float* f) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) ssm_conv_vec_kernel(const SsmArgs a) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (c >= a.ld_u) return;
+  const SeqSpan sp = seq_span(a, blockIdx.z);
+  const T* x = static_cast<const T*>(a.xz) + c;
+  const float* old = a.conv_state + static_cast<size_t>(sp.seq) * (TAPS - 1) * a.ld_u + c;
+  float w[TAPS][8], bias[8], hist[TAPS > 1 ? TAPS - 1 : 1][8];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) ld8(a.conv_w + static_cast<size_t>(j) * a.ld_u + c, w[j]);
+  ld8(a.conv_b + c, bias);
+  const int t0 = blockIdx.y * kVecRows, base = blockIdx.z * a.rows.Tc, t1 = min(t0 + kVecRows, a.rows.Tc);
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {                   // the inputs in front of row t0
+    const int rel = base + t0 - sp.row0 - (TAPS - 1) + j;
+    if (rel >= 0) ld8(x + static_cast<size_t>(sp.row0 + rel) * a.ld_xz, hist[j]);
+    else if (sp.start + rel >= 0 && rel >= -(TAPS - 1)) ld8(old + static_cast<size_t>(TAPS - 1 + rel) * a.ld_u, hist[j]);
+    else
+#pragma unroll
+      for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
+  }
+#pragma unroll 4
+  for (int t = t0; t < t1; ++t) {
+    const int row = base + t;
+    const bool real = row >= sp.row0;
+    float xv[8], v[8];
+    ld8(x + static_cast<size_t>(row) * a.ld_xz, xv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float y = bias[e];
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) y = fmaf(w[j][e], hist[j][e], y);
+      y = fmaf(w[TAPS - 1][e], xv[e], y);
+      v[e] = real ? silu(y) : 0.f;
+    }
+    if (real) {
+      if constexpr (TAPS > 1) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) hist[j][e] = hist[j + 1][e];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) hist[TAPS - 2][e] = xv[e];
+      }
+    }
+    const size_t o = static_cast<size_t>(row) * a.ld_u + c;
+    if (a.u) {
+      reinterpret_cast<float4*>(a.u + o)[0] = make_float4(v[0], v[1], v[2], v[3]);
+      reinterpret_cast<float4*>(a.u + o)[1] = make_float4(v[4], v[5], v[6], v[7]);
+    } else {
+      *reinterpret_cast<uint4*>(a.u_bf16 + o) =
+          make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+    }
   }
 }
 
@@ -76,13 +144,13 @@ __global__ void __launch_bounds__(256) ssm_conv_state_kernel(const SsmArgs a) {
   const SeqSpan sp = seq_span(a, blockIdx.y);
   if (sp.n <= 0) return;
   const T* x = static_cast<const T*>(a.xz);
-  float* st = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.inner + c;
+  float* st = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.ld_u + c;
   for (int j = 0; j < a.taps - 1; ++j) {
     const int rel = sp.n - (a.taps - 1) + j;
     float v = 0.f;
     if (rel >= 0) v = ld(x, static_cast<size_t>(sp.row0 + rel) * a.ld_xz + c);
-    else if (sp.start + rel >= 0) v = st[static_cast<size_t>(a.taps - 1 + rel) * a.inner];
-    st[static_cast<size_t>(j) * a.inner] = v;
+    else if (sp.start + rel >= 0) v = st[static_cast<size_t>(a.taps - 1 + rel) * a.ld_u];
+    st[static_cast<size_t>(j) * a.ld_u] = v;
   }
 }
 
@@ -94,55 +162,126 @@ __global__ void __launch_bounds__(256) ssm_conv_step_kernel(const SsmArgs a) {
   const int c = blockIdx.x * 256 + threadIdx.x, m = blockIdx.y;
   if (c >= a.inner) return;
   const SeqSpan sp = seq_span(a, m);
-  float* st = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.inner + c;
+  float* st = a.conv_state + static_cast<size_t>(sp.seq) * (a.taps - 1) * a.ld_u + c;
   const float x = ld(static_cast<const T*>(a.xz), static_cast<size_t>(m) * a.ld_xz + c);
   float v = fmaf(a.conv_w[static_cast<size_t>(a.taps - 1) * a.ld_u + c], x, a.conv_b[c]);
   for (int j = 0; j < a.taps - 1; ++j) {
-    const float xv = sp.start >= a.taps - 1 - j ? st[static_cast<size_t>(j) * a.inner] : 0.f;
+    const float xv = sp.start >= a.taps - 1 - j ? st[static_cast<size_t>(j) * a.ld_u] : 0.f;
     v = fmaf(a.conv_w[static_cast<size_t>(j) * a.ld_u + c], xv, v);
-    if (j > 0) st[static_cast<size_t>(j - 1) * a.inner] = xv;
+    if (j > 0) st[static_cast<size_t>(j - 1) * a.ld_u] = xv;
   }
-  if (a.taps > 1) st[static_cast<size_t>(a.taps - 2) * a.inner] = x;
+  if (a.taps > 1) st[static_cast<size_t>(a.taps - 2) * a.ld_u] = x;
   v = silu(v);
   const size_t o = static_cast<size_t>(m) * a.ld_u + c;
   if (a.u) a.u[o] = v;
   if (a.u_bf16) a.u_bf16[o] = __float2bfloat16_rn(v);
 }
 
-__global__ void ssm_split_kernel(const SsmArgs a) {
+// xp = sum of the split-K planes of the projection; its dt part once more in bf16, the operand of the next one.
+__global__ void __launch_bounds__(128) ssm_split_kernel(const SsmArgs a) {
+  pdl_wait();
+  pdl_launch_dependents();
   const size_t m = blockIdx.x;
-  for (int i = threadIdx.x; i < a.dt_rank; i += blockDim.x)
-    a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(a.xp[m * a.ld_xp + i]);
+  const int n = a.dt_rank + 2 * a.state;
+  const float* src = a.xp_planes + m * n;
+  for (int i = threadIdx.x; i < n; i += 128) {
+    float v = src[i];
+#pragma unroll 8
+    for (int p = 1; p < a.planes; ++p) v += src[static_cast<size_t>(p) * a.M * n + i];
+    a.xp_out[m * a.ld_xp + i] = v;
+    if (i < a.dt_rank) a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(v);
+  }
 }
 
 // The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states; a block covers
-// 128 / G channels and stages kTT rows of dt, u, z (per channel) and B, C (shared) in shared memory.
+// CH = 128 / G channels.  Tiles of kTT rows of dt, u, z (per channel) and B, C (shared) come into shared memory by
+// cp.async, one tile ahead of the recurrence.  The work is bound by the exponentials (one per row, channel and state).
 constexpr int kScanThreads = 128;
 constexpr int kTT = 32;
 
+__device__ __forceinline__ void cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp4(void* dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// fp32 runs take the accurate exponential, serving runs the hardware's base-2 one (A is scaled by log2 e for it)
+template <typename T>
+struct Decay;
+template <>
+struct Decay<float> {
+  static constexpr float kScale = 1.0f;
+  __device__ static __forceinline__ float f(float x) { return expf(x); }
+};
+template <>
+struct Decay<__nv_bfloat16> {
+  static constexpr float kScale = 1.4426950408889634f;
+  __device__ static __forceinline__ float f(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+  }
+};
+
+template <typename T, int G, int NS>
+struct ScanTile {
+  static constexpr int CH = kScanThreads / G, NSP = G * NS;
+  float B[kTT][NSP], C[kTT][NSP];
+  float dt[kTT][CH];
+  T u[kTT][CH], z[kTT][CH];
+};
+
 template <typename T, int G, int NS>
 __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const SsmArgs a) {
-  constexpr int CH = kScanThreads / G;
-  extern __shared__ float sc_smem[];
-  const int nsp = G * NS;                                // states, padded
-  float* sB = sc_smem;                                   // [kTT][nsp]
-  float* sC = sB + kTT * nsp;
-  float* sDt = sC + kTT * nsp;                           // [kTT][CH]
-  float* sU = sDt + kTT * CH;
-  float* sY = sU + kTT * CH;
+  using Tile = ScanTile<T, G, NS>;
+  constexpr int CH = Tile::CH, NSP = Tile::NSP, kVec = 16 / static_cast<int>(sizeof(T));
+  extern __shared__ __align__(16) unsigned char sc_smem[];
+  Tile* tiles = reinterpret_cast<Tile*>(sc_smem);
+  float(*sY)[CH] = reinterpret_cast<float(*)[CH]>(sc_smem + 2 * sizeof(Tile));
   const SeqSpan sp = seq_span(a, blockIdx.y);
   const int ch = threadIdx.x / G, g = threadIdx.x % G;
   const int c0 = blockIdx.x * CH, c = c0 + ch;
   const bool c_ok = c < a.inner;
   const T* u = a.u ? reinterpret_cast<const T*>(a.u) : reinterpret_cast<const T*>(a.u_bf16);
-  const T* xz = static_cast<const T*>(a.xz);
+  const T* z = static_cast<const T*>(a.xz) + a.z0;
+  auto fetch = [&](int t0, Tile& d) {
+    const int nt = min(kTT, sp.n - t0);
+    for (int i = threadIdx.x; i < nt * (CH / 4); i += kScanThreads) {
+      const int t = i / (CH / 4), q = i % (CH / 4) * 4;
+      if (c0 + q < a.ld_u) cp16(&d.dt[t][q], a.dt_raw + static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + q);
+    }
+    constexpr int kRow = CH / kVec > 0 ? CH / kVec : 1;
+    static_assert(CH % kVec == 0, "whole 16-byte groups of channels");
+    for (int i = threadIdx.x; i < nt * kRow; i += kScanThreads) {
+      const int t = i / kRow, q = i % kRow * kVec;
+      if (c0 + q >= a.ld_u) continue;
+      const size_t m = static_cast<size_t>(sp.row0 + t0 + t);
+      cp16(&d.u[t][q], u + m * a.ld_u + c0 + q);
+      cp16(&d.z[t][q], z + m * a.ld_xz + c0 + q);
+    }
+    for (int i = threadIdx.x; i < nt * NSP; i += kScanThreads) {
+      const int t = i / NSP, n = i % NSP;
+      if (n >= a.state) continue;                        // stays zero
+      const float* row = a.xp + static_cast<size_t>(sp.row0 + t0 + t) * a.ld_xp + a.dt_rank + n;
+      cp4(&d.B[t][n], row);
+      cp4(&d.C[t][n], row + a.state);
+    }
+    cp_commit();
+  };
+  for (int i = threadIdx.x; i < static_cast<int>(2 * sizeof(Tile) / 4); i += kScanThreads) reinterpret_cast<float*>(tiles)[i] = 0.f;
+  __syncthreads();
+  if (sp.n > 0) fetch(0, tiles[0]);
   float S[NS], A[NS];
   float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + (c_ok ? c : 0)) * a.state;
 #pragma unroll
   for (int i = 0; i < NS; ++i) {
     const int n = g * NS + i;
     const bool ok = c_ok && n < a.state;
-    A[i] = ok ? a.A[static_cast<size_t>(c) * a.state + n] : 0.f;
+    A[i] = ok ? a.A[static_cast<size_t>(c) * a.state + n] * Decay<T>::kScale : 0.f;
     S[i] = (ok && sp.start > 0 && sp.n > 0) ? state[n] : 0.f;
   }
   // rows in front of the sequence's start give zeros
@@ -154,45 +293,43 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const SsmArgs a)
       if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(0.f);
     }
   }
-  for (int t0 = 0; t0 < sp.n; t0 += kTT) {
+  // the channel a thread finishes (softplus, gate) is the same in every round: CH divides the block
+  const int fc = threadIdx.x % CH, f_ok = c0 + fc < a.inner;
+  const float dt_b = f_ok ? a.dt_b[c0 + fc] : 0.f, D = f_ok ? a.D[c0 + fc] : 0.f;
+  for (int t0 = 0, k = 0; t0 < sp.n; t0 += kTT, ++k) {
+    Tile& d = tiles[k & 1];
     const int nt = min(kTT, sp.n - t0);
+    if (t0 + kTT < sp.n) {
+      fetch(t0 + kTT, tiles[(k + 1) & 1]);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
     __syncthreads();
-    for (int i = threadIdx.x; i < nt * nsp; i += kScanThreads) {
-      const int t = i / nsp, n = i % nsp;
-      const float* row = a.xp + static_cast<size_t>(sp.row0 + t0 + t) * a.ld_xp + a.dt_rank;
-      sB[i] = n < a.state ? row[n] : 0.f;
-      sC[i] = n < a.state ? row[a.state + n] : 0.f;
-    }
-    for (int i = threadIdx.x; i < nt * CH; i += kScanThreads) {
-      const int t = i / CH, cc = c0 + i % CH;
-      const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + cc;
-      const bool ok = cc < a.inner;
-      sDt[i] = ok ? softplus(a.dt_raw[o] + a.dt_b[cc]) : 0.f;
-      sU[i] = ok ? ld(u, o) : 0.f;
-    }
+    for (int t = threadIdx.x / CH; t < nt; t += G) d.dt[t][fc] = f_ok ? softplus(d.dt[t][fc] + dt_b) : 0.f;
     __syncthreads();
 #pragma unroll 4
     for (int t = 0; t < nt; ++t) {
-      const float dt = sDt[t * CH + ch], du = dt * sU[t * CH + ch];
+      const float dt = d.dt[t][ch], du = dt * ld(&d.u[t][ch], 0);
       float y = 0.f;
 #pragma unroll
       for (int i = 0; i < NS; ++i) {
-        S[i] = fmaf(expf(dt * A[i]), S[i], du * sB[t * nsp + g * NS + i]);
-        y = fmaf(S[i], sC[t * nsp + g * NS + i], y);
+        S[i] = fmaf(Decay<T>::f(dt * A[i]), S[i], du * d.B[t][g * NS + i]);
+        y = fmaf(S[i], d.C[t][g * NS + i], y);
       }
 #pragma unroll
       for (int o = G / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (g == 0) sY[t * CH + ch] = y;
+      if (g == 0) sY[t][ch] = y;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < nt * CH; i += kScanThreads) {
-      const int t = i / CH, cc = c0 + i % CH;
-      if (cc >= a.inner) continue;
-      const size_t m = static_cast<size_t>(sp.row0 + t0 + t), o = m * a.ld_u + cc;
-      const float y = fmaf(a.D[cc], sU[i], sY[i]) * silu(ld(xz, m * a.ld_xz + a.z0 + cc));
+    for (int t = threadIdx.x / CH; t < nt; t += G) {
+      if (!f_ok) break;
+      const float y = fmaf(D, ld(&d.u[t][fc], 0), sY[t][fc]) * silu(ld(&d.z[t][fc], 0));
+      const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + fc;
       if (a.out) a.out[o] = y;
       if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
     }
+    __syncthreads();                                     // the tile may be fetched over, sY written again
   }
   if (c_ok && sp.n > 0) {
 #pragma unroll
@@ -201,42 +338,68 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const SsmArgs a)
   }
 }
 
-// Decode: G lanes per channel do the step-size projection, the state update and the output of one row.
-template <typename T, int G>
+// Decode, one row per sequence: G lanes per channel do the step size (its projection too, unless dt_raw holds it),
+// the state update and the output.  VEC: the state count is a multiple of four and every lane owns four
+// neighbouring states (state <= 4 G), so a warp reads and writes whole lines of the state.
+template <typename T, int G, bool VEC>
 __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
   extern __shared__ float st_smem[];                     // dt | B | C of the row
+  const int m = blockIdx.y, g = threadIdx.x % G, c = blockIdx.x * (256 / G) + threadIdx.x / G;
+  const bool ok = c < a.inner;
+  const int cc = ok ? c : 0;
+  float4 A4 = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (VEC && 4 * g < a.state) A4 = *reinterpret_cast<const float4*>(a.A + static_cast<size_t>(cc) * a.state + 4 * g);
+  if (!a.dt_raw)
+    for (int k = g * 8; k < a.ld_wdt; k += G * 8) prefetch_l2(a.w_dt + static_cast<size_t>(cc) * a.ld_wdt + k);
   pdl_wait();
   pdl_launch_dependents();
-  const int m = blockIdx.y, g = threadIdx.x % G, c = blockIdx.x * (256 / G) + threadIdx.x / G;
   const SeqSpan sp = seq_span(a, m);
+  float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + cc) * a.state;
+  float4 s4 = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (VEC && 4 * g < a.state && sp.start > 0) s4 = *reinterpret_cast<const float4*>(state + 4 * g);
   const int np = a.ld_wdt + 2 * a.state;                  // the dt part padded with zeros to the weight's row length
   for (int i = threadIdx.x; i < np; i += 256) {
     const float* row = a.xp + static_cast<size_t>(m) * a.ld_xp;
     st_smem[i] = i < a.dt_rank ? row[i] : i < a.ld_wdt ? 0.f : row[a.dt_rank + i - a.ld_wdt];
   }
   __syncthreads();
-  const bool ok = c < a.inner;
-  const int cc = ok ? c : 0;
   float dt = 0.f;
-  for (int k = g * 8; k < a.ld_wdt; k += G * 8) {
-    float w8[8];
-    unpack8(ld_stream16(a.w_dt + static_cast<size_t>(cc) * a.ld_wdt + k), w8);
+  if (a.dt_raw) {
+    dt = a.dt_raw[static_cast<size_t>(m) * a.ld_u + cc];
+  } else {
+#pragma unroll 4
+    for (int k = g * 8; k < a.ld_wdt; k += G * 8) {
+      float w8[8];
+      unpack8(ld_stream16(a.w_dt + static_cast<size_t>(cc) * a.ld_wdt + k), w8);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) dt = fmaf(w8[e], st_smem[k + e], dt);
+      for (int e = 0; e < 8; ++e) dt = fmaf(w8[e], st_smem[k + e], dt);
+    }
+#pragma unroll
+    for (int o = G / 2; o > 0; o >>= 1) dt += __shfl_xor_sync(0xffffffffu, dt, o);
   }
-#pragma unroll
-  for (int o = G / 2; o > 0; o >>= 1) dt += __shfl_xor_sync(0xffffffffu, dt, o);
   dt = softplus(dt + a.dt_b[cc]);
   const float u = a.u ? a.u[static_cast<size_t>(m) * a.ld_u + cc] : __bfloat162float(a.u_bf16[static_cast<size_t>(m) * a.ld_u + cc]);
   const float du = dt * u;
   const float* B = st_smem + a.ld_wdt;
-  float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + cc) * a.state;
+  const float* C = B + a.state;
   float y = 0.f;
-  for (int n = g; n < a.state; n += G) {
-    const float old = sp.start > 0 ? state[n] : 0.f;
-    const float s = fmaf(expf(dt * a.A[static_cast<size_t>(cc) * a.state + n]), old, du * B[n]);
-    if (ok) state[n] = s;
-    y = fmaf(s, B[a.state + n], y);
+  if (VEC) {
+    if (4 * g < a.state) {
+      const int n = 4 * g;
+      s4.x = fmaf(expf(dt * A4.x), s4.x, du * B[n]);
+      s4.y = fmaf(expf(dt * A4.y), s4.y, du * B[n + 1]);
+      s4.z = fmaf(expf(dt * A4.z), s4.z, du * B[n + 2]);
+      s4.w = fmaf(expf(dt * A4.w), s4.w, du * B[n + 3]);
+      if (ok) *reinterpret_cast<float4*>(state + n) = s4;
+      y = s4.x * C[n] + s4.y * C[n + 1] + s4.z * C[n + 2] + s4.w * C[n + 3];
+    }
+  } else {
+    for (int n = g; n < a.state; n += G) {
+      const float old = sp.start > 0 ? state[n] : 0.f;
+      const float s = fmaf(expf(dt * a.A[static_cast<size_t>(cc) * a.state + n]), old, du * B[n]);
+      if (ok) state[n] = s;
+      y = fmaf(s, C[n], y);
+    }
   }
 #pragma unroll
   for (int o = G / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
@@ -251,40 +414,62 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
 
 bool ssm_ok(const SsmArgs& a) {
   return a.M > 0 && a.inner > 0 && a.state > 0 && a.state <= kSsmMaxState && a.taps >= 1 && a.nseq > 0 && a.rows.Tc > 0 &&
-         a.M == a.nseq * a.rows.Tc && a.ld_u >= a.inner && (a.u != nullptr) != (a.u_bf16 != nullptr) &&
+         a.M == a.nseq * a.rows.Tc && a.ld_u >= a.inner && (a.ld_u & 7) == 0 && (a.ld_xz & 7) == 0 && (a.u != nullptr) != (a.u_bf16 != nullptr) &&
          (a.u != nullptr) == !a.xz_bf16;
 }
 
 template <typename T, int G, int NS>
 cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
-  constexpr int CH = kScanThreads / G;
-  const size_t smem = sizeof(float) * kTT * (2 * G * NS + 3 * CH);
+  using Tile = ScanTile<T, G, NS>;
+  constexpr int smem = static_cast<int>(2 * sizeof(Tile) + sizeof(float) * kTT * Tile::CH);
   static DeviceOnce once;
   cudaError_t e = once.run([&] {
-    return cudaFuncSetAttribute(ssm_scan_kernel<T, G, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    return cudaFuncSetAttribute(ssm_scan_kernel<T, G, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   });
   if (e != cudaSuccess) return e;
-  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CH - 1) / CH, a.nseq), kScanThreads, smem, s>>>(a);
+  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + Tile::CH - 1) / Tile::CH, a.nseq), kScanThreads, smem, s>>>(a);
   return cudaGetLastError();
 }
 
 template <typename T>
 cudaError_t scan_states(const SsmArgs& a, cudaStream_t s) {
+  // few channels: more lanes per channel, so that every scheduler has a few warps
+  const bool few = static_cast<int64_t>(a.inner) * a.nseq < 148 * 2 * 32;
   if (a.state <= 8) return scan<T, 4, 2>(a, s);
-  if (a.state <= 16) return scan<T, 4, 4>(a, s);
+  if (a.state <= 16) return few ? scan<T, 8, 2>(a, s) : scan<T, 4, 4>(a, s);
   if (a.state <= 32) return scan<T, 8, 4>(a, s);
   if (a.state <= 64) return scan<T, 16, 4>(a, s);
-  if (a.state <= 128) return scan<T, 32, 4>(a, s);
-  return scan<T, 32, 8>(a, s);
+  if (a.state <= 128) return scan<T, 16, 8>(a, s);
+  return scan<T, 16, 16>(a, s);
+}
+
+template <typename T, int G, bool VEC>
+cudaError_t step(const SsmArgs& a, size_t smem, cudaStream_t s, bool pdl) {
+  constexpr int CH = 256 / G;
+  return launch_pdl(ssm_step_kernel<T, G, VEC>, dim3((a.inner + CH - 1) / CH, a.M), dim3(256), smem, s, pdl, a);
 }
 
 template <typename T>
 cudaError_t step_states(const SsmArgs& a, cudaStream_t s, bool pdl) {
   const size_t smem = sizeof(float) * (a.ld_wdt + 2 * static_cast<size_t>(a.state));
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
-  if (a.state <= 8) return launch_pdl(ssm_step_kernel<T, 8>, dim3((a.inner + 31) / 32, a.M), dim3(256), smem, s, pdl, a);
-  if (a.state <= 16) return launch_pdl(ssm_step_kernel<T, 16>, dim3((a.inner + 15) / 16, a.M), dim3(256), smem, s, pdl, a);
-  return launch_pdl(ssm_step_kernel<T, 32>, dim3((a.inner + 7) / 8, a.M), dim3(256), smem, s, pdl, a);
+  if ((a.state & 3) == 0 && a.state <= 128) {
+    if (a.state <= 16) return step<T, 4, true>(a, smem, s, pdl);
+    if (a.state <= 32) return step<T, 8, true>(a, smem, s, pdl);
+    return step<T, 32, true>(a, smem, s, pdl);
+  }
+  return a.state <= 8 ? step<T, 8, false>(a, smem, s, pdl) : step<T, 32, false>(a, smem, s, pdl);
+}
+
+template <typename T>
+cudaError_t conv_vec(const SsmArgs& a, cudaStream_t s, bool pdl) {
+  const dim3 grid((a.ld_u / 8 + 127) / 128, (a.rows.Tc + kVecRows - 1) / kVecRows, a.nseq);
+  switch (a.taps) {
+    case 1: return launch_pdl(ssm_conv_vec_kernel<T, 1>, grid, dim3(128), 0, s, pdl, a);
+    case 2: return launch_pdl(ssm_conv_vec_kernel<T, 2>, grid, dim3(128), 0, s, pdl, a);
+    case 3: return launch_pdl(ssm_conv_vec_kernel<T, 3>, grid, dim3(128), 0, s, pdl, a);
+    default: return launch_pdl(ssm_conv_vec_kernel<T, 4>, grid, dim3(128), 0, s, pdl, a);
+  }
 }
 
 }  // namespace
@@ -296,21 +481,21 @@ cudaError_t launch_ssm_conv(const SsmArgs& a, cudaStream_t s, bool pdl) {
     return a.xz_bf16 ? launch_pdl(ssm_conv_step_kernel<__nv_bfloat16>, dim3(cb, a.M), dim3(256), 0, s, pdl, a)
                      : launch_pdl(ssm_conv_step_kernel<float>, dim3(cb, a.M), dim3(256), 0, s, pdl, a);
   const dim3 grid(cb, (a.rows.Tc + kConvRows - 1) / kConvRows, a.nseq);
-  cudaError_t e = a.xz_bf16 ? launch_pdl(ssm_conv_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, a)
-                            : launch_pdl(ssm_conv_kernel<float>, grid, dim3(256), 0, s, pdl, a);
+  cudaError_t e = a.taps <= 4 ? (a.xz_bf16 ? conv_vec<__nv_bfloat16>(a, s, pdl) : conv_vec<float>(a, s, pdl))
+                  : a.xz_bf16 ? launch_pdl(ssm_conv_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, a)
+                              : launch_pdl(ssm_conv_kernel<float>, grid, dim3(256), 0, s, pdl, a);
   if (e != cudaSuccess || a.taps == 1) return e;
   return a.xz_bf16 ? launch_pdl(ssm_conv_state_kernel<__nv_bfloat16>, dim3(cb, a.nseq), dim3(256), 0, s, pdl, a)
                    : launch_pdl(ssm_conv_state_kernel<float>, dim3(cb, a.nseq), dim3(256), 0, s, pdl, a);
 }
 
-cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s) {
-  if (!ssm_ok(a) || !a.dtr_bf16) return cudaErrorInvalidValue;
-  ssm_split_kernel<<<a.M, 64, 0, s>>>(a);
-  return cudaGetLastError();
+cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s, bool pdl) {
+  if (!ssm_ok(a) || !a.dtr_bf16 || !a.xp_planes || !a.xp_out || a.planes < 1) return cudaErrorInvalidValue;
+  return launch_pdl(ssm_split_kernel, dim3(a.M), dim3(128), 0, s, pdl, a);
 }
 
 cudaError_t launch_ssm_scan(const SsmArgs& a, cudaStream_t s) {
-  if (!ssm_ok(a) || !a.dt_raw) return cudaErrorInvalidValue;
+  if (!ssm_ok(a) || !a.dt_raw || (a.ld_u & 7) || (a.ld_xz & 7) || (a.z0 & 7)) return cudaErrorInvalidValue;
   return a.xz_bf16 ? scan_states<__nv_bfloat16>(a, s) : scan_states<float>(a, s);
 }
 

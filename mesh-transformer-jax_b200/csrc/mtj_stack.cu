@@ -18,7 +18,6 @@ namespace {
 int up8(int64_t v) { return static_cast<int>(align_up(v, 8)); }
 int up4(int v) { return (v + 3) & ~3; }
 constexpr int kAbsorbRows = 256;       // rows of the absorbed attention's scratch
-constexpr int kAbsorbBlocks = 592;     // blocks its decode form aims at (148 SMs x 4)
 constexpr int kSelectGemvRows = 4;
 }  // namespace
 
@@ -72,7 +71,7 @@ int32_t LayerStack::create(const mtj_config& cfg, const mtj_stack_desc& desc, in
       if (m.inner <= 0 || m.state <= 0 || m.conv <= 0 || m.dt_rank <= 0) return fail(MTJ_ERR_INVALID, at + "state-space sizes");
       if (m.state > kSsmMaxState || m.conv > 64 || m.dt_rank > 8192)
         return fail(MTJ_ERR_UNSUPPORTED, at + "state-space mixers take state up to 256, conv up to 64, dt_rank up to 8192");
-      l.in.shape(2 * m.inner, st.d_);
+      l.in.shape(up8(m.inner) + m.inner, st.d_);      // x rows, zero rows up to a multiple of 8, z rows
       l.out.shape(st.d_, m.inner);
       l.x.shape(m.dt_rank + 2 * m.state, m.inner);
       l.dt.shape(m.inner, m.dt_rank);
@@ -149,11 +148,6 @@ void LayerStack::carve_weights(Carver& c) {
   w_end_ = c.base ? c.base + c.off : nullptr;
 }
 
-int LayerStack::decode_splits(int M, const Layer& l) const {
-  const int groups = M * ((l.d.heads + 7) / 8);
-  return std::max(1, std::min(latent_attn_splits(std::min(l.d.window, max_pos_)), kAbsorbBlocks / groups));
-}
-
 void LayerStack::carve_workspace(Carver& c) {
   const int64_t R = R_;
   s_begin_ = c.base ? c.base + c.off : nullptr;
@@ -193,8 +187,8 @@ void LayerStack::carve_workspace(Carver& c) {
   xp_ = c.take<float>(R * xp);
   dt_raw_ = c.take<float>(R * u);
   q_abs_ = c.take<float>(rows_a_ * qabs);
-  part_o_ = c.take<float>((rows_a_ + kAbsorbBlocks) * po);
-  part_ml_ = c.take<float>((rows_a_ + kAbsorbBlocks) * ml * 2);
+  part_o_ = c.take<float>((rows_a_ + kLatentBlocks) * po);
+  part_ml_ = c.take<float>((rows_a_ + kLatentBlocks) * ml * 2);
   counters_ = c.take<uint32_t>(R);
   if (loop_times_ > 0) {
     x0_ = c.take<float>(R * ld_);
@@ -207,6 +201,8 @@ void LayerStack::carve_workspace(Carver& c) {
     xz_bf_ = c.take<__nv_bfloat16>(R * xz);
     u_bf_ = c.take<__nv_bfloat16>(R * u);
     dtr_bf_ = c.take<__nv_bfloat16>(R * dtr);
+    xp_planes_elems_ = xp * std::max<int64_t>(4 * R, 32 * std::min<int64_t>(R, 128));
+    xp_planes_ = c.take<float>(xp_planes_elems_);
     act_bf_ = c.take<__nv_bfloat16>(R * act);
     q_pack_ = c.take<__nv_bfloat16>(R * qp);
     c_lin_ = c.take<__nv_bfloat16>(lin_rows_ * cl);
@@ -221,7 +217,7 @@ void LayerStack::carve_workspace(Carver& c) {
       const int64_t elems = static_cast<int64_t>(max_batch_) * l.ring_pages * kPageTokens * l.row_ld;
       r.cache = f32_ ? static_cast<void*>(c.take<float>(elems)) : static_cast<void*>(c.take<__nv_bfloat16>(elems));
     } else {
-      r.conv_state = c.take<float>(static_cast<int64_t>(max_batch_) * (l.d.conv - 1) * l.d.inner);
+      r.conv_state = c.take<float>(static_cast<int64_t>(max_batch_) * (l.d.conv - 1) * l.ld_u);
       r.ssm_state = c.take<float>(static_cast<int64_t>(max_batch_) * l.d.inner * l.d.state);
     }
   }
@@ -325,7 +321,7 @@ int32_t LayerStack::bind(mtj_handle* h, cudaStream_t s) {
         v.dst2 = l.up.w; v.ld2 = l.up.ld; v.r02 = m.heads * 64 * l.k_own; v.gin2 = m.vdim; v.gout2 = 64 * l.value_blocks;
       }
     } else {
-      rows(p + "mix.in", l.in.N, l.in.K, l.in.w, l.in.ld);
+      rows(p + "mix.in", 2 * m.inner, d_, l.in.w, l.in.ld, 0, m.inner, up8(m.inner));
       rows(p + "mix.x", l.x.N, l.x.K, l.x.w, l.x.ld);
       rows(p + "mix.dt", l.dt.N, l.dt.K, l.dt.w, l.dt.ld);
       vec(p + "mix.conv.b", m.inner, l.conv_b);
@@ -418,6 +414,27 @@ int32_t LayerStack::gemm(mtj_handle* h, GemvEpilogue epi, const Linear& l, const
   return MTJ_OK;
 }
 
+// A projection with few weight rows: K split over blocks, the partial sums [planes, M, N] left for the consumer to add.
+int32_t LayerStack::gemm_planes(mtj_handle* h, const Linear& l, const __nv_bfloat16* x, int M, int* planes, bool decode,
+                                cudaStream_t s) {
+  const int bn = gemm_tc_token_tile_for(M);
+  const auto key = xmap(x, l.K, l.ld, std::min(M, 128));
+  if (!key) return fail(MTJ_ERR_CUDA, "cuTensorMapEncodeTiled failed");
+  const int tiles = ((l.N + 127) / 128) * ((M + bn - 1) / bn);
+  const int64_t fit = xp_planes_elems_ / (static_cast<int64_t>(M) * l.N);
+  GemmTcArgs a = {};
+  a.M = M;
+  a.N = l.N;
+  a.K = l.K;
+  a.partial = xp_planes_;
+  a.ksplit = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({fit, 296 / tiles, (l.K + 127) / 128, 32})));
+  a.dev_err = h->dev_err;
+  MTJ_CUDA(launch_gemm_tc(kEpiPlain, &l.map, key, a, s, decode && h->use_pdl && h->tc_pdl));
+  h->launches++;
+  *planes = a.ksplit;
+  return MTJ_OK;
+}
+
 int32_t LayerStack::gemv(mtj_handle* h, GemvEpilogue epi, const Linear& l, const float* x, int ldx, int M, const float* norm,
                          float* out, int ld_out, const float* post_w, bool pdl, cudaStream_t s, const int32_t* select,
                          const float* stats) {
@@ -474,14 +491,13 @@ int32_t LayerStack::mamba(mtj_handle* h, const Run& r, int M, const RowMap& rows
   a.nseq = M / rows.Tc;
   a.pad = h->pad;
   a.ld_xz = up8(l.in.N);
-  a.z0 = m.inner;
+  a.z0 = l.ld_u;
   a.conv_w = l.conv_w;
   a.conv_b = l.conv_b;
   a.conv_state = r.conv_state;
   a.ld_u = l.ld_u;
   a.xp = xp_;
   a.ld_xp = l.ld_xp;
-  a.dt_raw = dt_raw_;
   a.w_dt = l.dt.w;
   a.ld_wdt = l.dt.ld;
   a.dt_b = l.dt_b;
@@ -494,6 +510,8 @@ int32_t LayerStack::mamba(mtj_handle* h, const Run& r, int M, const RowMap& rows
     a.xz_bf16 = 1;
     a.u_bf16 = u_bf_;
     a.out_bf16 = act_bf_;
+    a.xp_planes = xp_planes_;
+    a.xp_out = xp_;
     a.dtr_bf16 = dtr_bf_;
     a.ld_dtr = l.dt.ld;
     MTJ_DO(gemm(h, kEpiPlain, l.in, xn_bf_, M, nullptr, 0, xz_bf_, a.ld_xz, decode, s));
@@ -507,22 +525,22 @@ int32_t LayerStack::mamba(mtj_handle* h, const Run& r, int M, const RowMap& rows
   h->prof_begin(MTJ_FAMILY_ATTN, s);
   MTJ_CUDA(launch_ssm_conv(a, s, pdl));
   h->launches += (rows.Tc == 1 || m.conv == 1) ? 1 : 2;
-  if (tc) MTJ_DO(gemm(h, kEpiPlain, l.x, u_bf_, M, xp_, l.ld_xp, nullptr, 0, decode, s));
-  else MTJ_DO(gemv(h, kEpiOut, l.x, u_, l.ld_u, M, nullptr, xp_, l.ld_xp, nullptr, pdl, s));
-  if (rows.Tc == 1) {
-    MTJ_CUDA(launch_ssm_step(a, s, pdl));
+  if (tc) {
+    MTJ_DO(gemm_planes(h, l.x, u_bf_, M, &a.planes, decode, s));
+    MTJ_CUDA(launch_ssm_split(a, s, pdl));
     h->launches++;
+    MTJ_DO(gemm(h, kEpiPlain, l.dt, dtr_bf_, M, dt_raw_, l.ld_u, nullptr, 0, decode, s));
+    a.dt_raw = dt_raw_;
   } else {
-    if (tc) {
-      MTJ_CUDA(launch_ssm_split(a, s));
-      h->launches++;
-      MTJ_DO(gemm(h, kEpiPlain, l.dt, dtr_bf_, M, dt_raw_, l.ld_u, nullptr, 0, decode, s));
-    } else {
+    MTJ_DO(gemv(h, kEpiOut, l.x, u_, l.ld_u, M, nullptr, xp_, l.ld_xp, nullptr, pdl, s));
+    if (rows.Tc > 1) {
       MTJ_DO(gemv(h, kEpiOut, l.dt, xp_, l.ld_xp, M, nullptr, dt_raw_, l.ld_u, nullptr, pdl, s));
+      a.dt_raw = dt_raw_;
     }
-    MTJ_CUDA(launch_ssm_scan(a, s));
-    h->launches++;
   }
+  if (rows.Tc == 1) MTJ_CUDA(launch_ssm_step(a, s, pdl));
+  else MTJ_CUDA(launch_ssm_scan(a, s));
+  h->launches++;
   h->prof_end(s);
   h->prof_begin(MTJ_FAMILY_OUTPROJ, s);
   if (tc) MTJ_DO(gemm(h, kEpiPlain, l.out, act_bf_, M, y_, ld_, nullptr, 0, decode, s));
@@ -599,10 +617,11 @@ int32_t LayerStack::latent(mtj_handle* h, const Run& r, int M, const RowMap& row
       for (int t0 = 0; t0 < per; t0 += rows_a_) {
         LatentArgs b = a;
         b.M = std::min(rows_a_, per - t0);
+        b.tensor_cores = tc ? 1 : 0;
         b.rows = rows.Tc == 1 ? RowMap{rows.b0 + t0, 1, rows.pos0_host, rows.pos0_dev}
                               : RowMap{rows.b0 + m0 / per, b.M, rows.pos0_host + t0, rows.pos0_dev};
         b.p1 = p1_ + static_cast<size_t>(m0 + t0) * a.ld_p1;
-        b.splits = decode_splits(b.M, l);
+        b.splits = latent_attn_splits(b.M, m.heads, l.row_ld, l.kv_ld, tc ? 1 : 0, std::min(m.window, max_pos_));
         if (tc) b.out_bf16 = act_bf_ + static_cast<size_t>(m0 + t0) * a.ld_out;
         else b.out = act_ + static_cast<size_t>(m0 + t0) * a.ld_out;
         MTJ_CUDA(launch_latent_absorb(b, s, pdl));

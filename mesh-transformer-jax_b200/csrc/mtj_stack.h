@@ -82,13 +82,13 @@ class LayerStack {
   const TensorMap* xmap(const __nv_bfloat16* buf, int K, int ld, int M);
   int32_t gemm(mtj_handle* h, GemvEpilogue epi, const Linear& l, const __nv_bfloat16* x, int M, float* out, int ld_out,
                __nv_bfloat16* out_bf16, int ld_bf16, bool decode, cudaStream_t s, int x_row0 = 0, int rows_x = 0);
+  int32_t gemm_planes(mtj_handle* h, const Linear& l, const __nv_bfloat16* x, int M, int* planes, bool decode, cudaStream_t s);
   int32_t gemv(mtj_handle* h, GemvEpilogue epi, const Linear& l, const float* x, int ldx, int M, const float* norm, float* out,
                int ld_out, const float* post_w, bool pdl, cudaStream_t s, const int32_t* select = nullptr,
                const float* stats = nullptr);
   int32_t mamba(mtj_handle* h, const Run& r, int M, const RowMap& rows, bool tc, bool decode, cudaStream_t s);
   int32_t latent(mtj_handle* h, const Run& r, int M, const RowMap& rows, int hist, bool tc, bool decode, cudaStream_t s);
   int32_t add_leaf(const std::string& name, Leaf leaf);
-  int decode_splits(int M, const Layer& l) const;
 
   int d_ = 0, V_ = 0, ld_ = 0, R_ = 0, max_batch_ = 0, max_pos_ = 0;
   int loop_start_ = 0, loop_stop_ = 0, loop_times_ = 0;
@@ -107,9 +107,10 @@ class LayerStack {
 
   // workspace, sized for the widest layer
   int rows_a_ = 0, lin_rows_ = 0, ld_p1_ = 0, ld_act_ = 0;
+  int64_t xp_planes_elems_ = 0;
   bool last_tc_ = false;
   float *x_ = nullptr, *x0_ = nullptr, *stats_ = nullptr, *cat_ = nullptr, *y_ = nullptr, *p1_ = nullptr, *u_ = nullptr, *xp_ = nullptr,
-        *dt_raw_ = nullptr, *act_ = nullptr, *q_abs_ = nullptr, *part_o_ = nullptr, *part_ml_ = nullptr;
+        *dt_raw_ = nullptr, *act_ = nullptr, *xp_planes_ = nullptr, *q_abs_ = nullptr, *part_o_ = nullptr, *part_ml_ = nullptr;
   __nv_bfloat16 *xn_bf_ = nullptr, *cat_bf_ = nullptr, *xz_bf_ = nullptr, *u_bf_ = nullptr, *dtr_bf_ = nullptr, *act_bf_ = nullptr,
                 *sel_bf_ = nullptr, *q_pack_ = nullptr, *c_lin_ = nullptr, *kr_lin_ = nullptr, *kv_lin_ = nullptr;
   uint32_t* counters_ = nullptr;

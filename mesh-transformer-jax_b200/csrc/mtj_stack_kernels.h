@@ -75,6 +75,7 @@ struct LatentArgs {
   const __nv_bfloat16* w_uv;   // [heads * vdim, kv_ld]
   // absorbed form (few rows, fp32 runs): q' = W_uk^T q, scores against the latent itself
   float* q_abs;                // [M, heads, row_ld], scaled
+  int tensor_cores;            // bf16 queries and weights on the tensor cores are allowed
   int splits;                  // key ranges per row
   float* part_o;               // [M, heads, splits, kv_ld]
   float* part_ml;              // [M, heads, splits, 2]
@@ -98,7 +99,8 @@ cudaError_t launch_latent_out(const LatentArgs& a, cudaStream_t s, bool pdl);
 cudaError_t launch_latent_pack(const LatentArgs& a, cudaStream_t s);
 cudaError_t launch_latent_history(const LatentArgs& a, cudaStream_t s);
 constexpr int kLatentMaxRank = 1024;
-int latent_attn_splits(int window);
+constexpr int kLatentBlocks = 592;       // most (rows x splits x head groups) a call spreads over beyond one per row
+int latent_attn_splits(int M, int heads, int row_ld, int kv_ld, int tensor_cores, int window);
 
 // ---- mtj_ssm.cu: causal convolution and selective scan with carried state
 struct SsmArgs {
@@ -110,15 +112,19 @@ struct SsmArgs {
   int xz_bf16, ld_xz, z0;
   const float* conv_w;         // [taps, ld_u]
   const float* conv_b;         // [ld_u]
-  float* conv_state;           // [slots][taps - 1][inner]
+  float* conv_state;           // [slots][taps - 1][ld_u]
   float* u;                    // [M, ld_u] or null
   __nv_bfloat16* u_bf16;       // [M, ld_u] or null
   int ld_u;
   const float* xp;             // [M, ld_xp] dt | B | C
   int ld_xp;
-  __nv_bfloat16* dtr_bf16;     // [M, ld_dtr] bf16 copy of the dt part (launch_ssm_split), or null
+  // launch_ssm_split: xp_out (= xp) and dtr_bf16 [M, ld_dtr], its dt part, from [planes, M, dt_rank + 2 state]
+  const float* xp_planes;
+  int planes;
+  float* xp_out;
+  __nv_bfloat16* dtr_bf16;
   int ld_dtr;
-  const float* dt_raw;         // [M, ld_u] W_dt dt, before the bias (scan)
+  const float* dt_raw;         // [M, ld_u] W_dt dt, before the bias; null in a step: the step projects itself
   const __nv_bfloat16* w_dt;   // [inner, ld_wdt] (step)
   int ld_wdt;
   const float* dt_b;
@@ -130,7 +136,7 @@ struct SsmArgs {
 };
 // u = silu(conv(x) + b) for all rows, then the taps - 1 last inputs of every sequence into conv_state
 cudaError_t launch_ssm_conv(const SsmArgs& a, cudaStream_t s, bool pdl);
-cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s);
+cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s, bool pdl);
 // the recurrence over the rows of every sequence, from and to ssm_state, with the gate
 cudaError_t launch_ssm_scan(const SsmArgs& a, cudaStream_t s);
 // one row per sequence: step size, recurrence and gate in one kernel
