@@ -473,29 +473,31 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
     }
   pdl_wait();
   pdl_launch_dependents();
-  if (warp < nr) {
-    const float* ml = a.part_ml + 2 * (static_cast<size_t>(m0 + warp) * a.heads + h) * a.splits;
+  for (int r = warp; r < nr; r += kThreads / 32) {
+    const float* ml = a.part_ml + 2 * (static_cast<size_t>(m0 + r) * a.heads + h) * a.splits;
     float mx = -INFINITY;
     for (int s = lane; s < a.splits; s += 32) mx = fmaxf(mx, ml[2 * s]);
     mx = warp_max(mx);
     float l = 0.f;
     for (int s = lane; s < a.splits; s += 32) {
       const float e = ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - mx);
-      ws[warp][s] = e;
+      ws[r][s] = e;
       l = fmaf(e, ml[2 * s + 1], l);
     }
     l = warp_sum(l);
     const float inv = l > 0.f ? 1.0f / l : 0.f;
-    for (int s = lane; s < a.splits; s += 32) ws[warp][s] *= inv;
+    for (int s = lane; s < a.splits; s += 32) ws[r][s] *= inv;
   }
   __syncthreads();
+  // RT == 1: two threads share a column group, each adding half of the ranges
+  constexpr int kParts = RT == 1 ? 2 : 1;
   const int k4 = kv_ld >> 2;
-  for (int i = threadIdx.x; i < RT * k4; i += kThreads) {
-    const int r = min(i / k4, nr - 1), k = i % k4;
+  for (int i = threadIdx.x; i < kParts * nr * k4; i += kThreads) {
+    const int part = i / (nr * k4), j = i % (nr * k4), r = j / k4, k = j % k4;
     const float4* po = reinterpret_cast<const float4*>(a.part_o + (static_cast<size_t>(m0 + r) * a.heads + h) * a.splits * kv_ld) + k;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-    for (int s = 0; s < a.splits; ++s) {
+#pragma unroll 16
+    for (int s = part; s < a.splits; s += kParts) {
       const float4 p = po[static_cast<size_t>(s) * k4];
       const float e = ws[r][s];
       v.x = fmaf(e, p.x, v.x); v.y = fmaf(e, p.y, v.y); v.z = fmaf(e, p.z, v.z); v.w = fmaf(e, p.w, v.w);
@@ -503,6 +505,10 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
     reinterpret_cast<float4*>(lo_smem)[i] = v;
   }
   __syncthreads();
+  if (kParts == 2) {
+    for (int i = threadIdx.x; i < kv_ld; i += kThreads) lo_smem[i] += lo_smem[kv_ld + i];
+    __syncthreads();
+  }
   for (int r = 0; r < nr; ++r) {
     float acc[kVW] = {};
 #pragma unroll
@@ -638,7 +644,7 @@ cudaError_t attend_mma(const LatentArgs& a, cudaStream_t s, bool pdl) {
 // head tiles of the tensor-core form (0: this call takes the CUDA-core form)
 int mma_head_tiles(int M, int heads, int row_ld, int kv_ld, int tensor_cores) {
   if (!tensor_cores || M < kMmaRows || mma_smem_bytes<1>(row_ld) > 220 * 1024) return 0;
-  return heads > 16 && kv_ld <= 512 && mma_smem_bytes<2>(row_ld) <= 220 * 1024 ? 2 : 1;
+  return 1;
 }
 
 }  // namespace
@@ -646,14 +652,14 @@ int mma_head_tiles(int M, int heads, int row_ld, int kv_ld, int tensor_cores) {
 int latent_attn_splits(int M, int heads, int row_ld, int kv_ld, int tensor_cores, int window) {
   const int mt = mma_head_tiles(M, heads, row_ld, kv_ld, tensor_cores);
   const int groups = M * (mt ? (heads + 16 * mt - 1) / (16 * mt) : (heads + kHG - 1) / kHG);
-  // one wave of blocks for the tensor-core form (one per SM), four per SM for the other
-  return std::max(1, std::min({kMaxSplits, (window + kTK - 1) / kTK, (mt ? 148 : kLatentBlocks) / groups}));
+  // one wave of blocks: two per SM for the tensor-core form, four for the other
+  return std::max(1, std::min({kMaxSplits, (window + kTK - 1) / kTK, (mt ? 296 : kLatentBlocks) / groups}));
 }
 
 cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a)) return cudaErrorInvalidValue;
-  if (a.cache.f32) return a.M == 1 ? absorb<float, 1>(a, s, pdl) : absorb<float, 4>(a, s, pdl);
-  return a.M == 1 ? absorb<__nv_bfloat16, 1>(a, s, pdl) : absorb<__nv_bfloat16, 4>(a, s, pdl);
+  if (a.cache.f32) return a.M == 1 ? absorb<float, 1>(a, s, pdl) : absorb<float, 8>(a, s, pdl);
+  return a.M == 1 ? absorb<__nv_bfloat16, 1>(a, s, pdl) : absorb<__nv_bfloat16, 8>(a, s, pdl);
 }
 
 cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl) {
@@ -661,7 +667,6 @@ cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl) {
   const int mt = mma_head_tiles(a.M, a.heads, a.cache.row_ld, a.cache.kv_ld, a.tensor_cores && !a.cache.f32);
   if (mt) {
     const int nt = (a.cache.kv_ld + 63) / 64;             // 8-column blocks per warp
-    if (mt == 2) return nt <= 2 ? attend_mma<2, 2>(a, s, pdl) : nt <= 4 ? attend_mma<2, 4>(a, s, pdl) : attend_mma<2, 8>(a, s, pdl);
     return nt <= 2 ? attend_mma<1, 2>(a, s, pdl) : nt <= 4 ? attend_mma<1, 4>(a, s, pdl) : nt <= 8 ? attend_mma<1, 8>(a, s, pdl) : attend_mma<1, 16>(a, s, pdl);
   }
   const bool two = a.cache.kv_ld > 2 * kThreads;
@@ -673,10 +678,11 @@ cudaError_t launch_latent_out(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a) || a.splits < 1 || a.splits > kMaxSplits) return cudaErrorInvalidValue;
   const int chunks = (a.vdim + kVC - 1) / kVC, kc = (a.cache.kv_ld + 255) / 256;
   auto go = [&](auto kernel, int rt) {
-    return launch_pdl(kernel, dim3(a.heads, chunks, (a.M + rt - 1) / rt), dim3(kThreads), sizeof(float) * rt * a.cache.kv_ld, s, pdl, a);
+    return launch_pdl(kernel, dim3(a.heads, chunks, (a.M + rt - 1) / rt), dim3(kThreads), sizeof(float) * std::max(rt, 2) * a.cache.kv_ld, s, pdl, a);
   };
   if (a.M == 1) return kc == 1 ? go(latent_out_kernel<1, 1>, 1) : kc == 2 ? go(latent_out_kernel<1, 2>, 1) : go(latent_out_kernel<1, 4>, 1);
-  return kc == 1 ? go(latent_out_kernel<8, 1>, 8) : kc == 2 ? go(latent_out_kernel<8, 2>, 8) : go(latent_out_kernel<8, 4>, 8);
+  if (a.M <= 8 || kc > 2) return kc == 1 ? go(latent_out_kernel<8, 1>, 8) : kc == 2 ? go(latent_out_kernel<8, 2>, 8) : go(latent_out_kernel<8, 4>, 8);
+  return kc == 1 ? go(latent_out_kernel<16, 1>, 16) : go(latent_out_kernel<16, 2>, 16);
 }
 
 cudaError_t launch_latent_pack(const LatentArgs& a, cudaStream_t s) {

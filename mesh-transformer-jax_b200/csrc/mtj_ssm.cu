@@ -67,13 +67,32 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
 
 // The same for at most four taps, a thread owning eight neighbouring channels: it walks kVecRows rows with the last
 // TAPS - 1 inputs in registers, one 16-byte load per row.  Columns between inner and the row stride hold zeros.
-constexpr int kVecRows = 16;
+constexpr int kVecRows = 8;
 
 __device__ __forceinline__ void ld8(const __nv_bfloat16* p, float* f) { unpack8(*reinterpret_cast<const uint4*>(p), f); }
 __device__ __forceinline__ void ld8(const float* p, float* f) {
   const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
   f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
 }
+
+template <typename T>
+struct Raw8;                       // eight elements as loaded
+template <>
+struct Raw8<__nv_bfloat16> {
+  using V = uint4;
+  __device__ static __forceinline__ V load(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+  __device__ static __forceinline__ void get(const V& v, float* f) { unpack8(v, f); }
+};
+template <>
+struct Raw8<float> {
+  struct V { float4 a, b; };
+  __device__ static __forceinline__ V load(const float* p) {
+    return {reinterpret_cast<const float4*>(p)[0], reinterpret_cast<const float4*>(p)[1]};
+  }
+  __device__ static __forceinline__ void get(const V& v, float* f) {
+    f[0] = v.a.x; f[1] = v.a.y; f[2] = v.a.z; f[3] = v.a.w; f[4] = v.b.x; f[5] = v.b.y; f[6] = v.b.z; f[7] = v.b.w;
+  }
+};
 
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) ssm_conv_vec_kernel(const SsmArgs a) {
@@ -98,12 +117,16 @@ __global__ void __launch_bounds__(128) ssm_conv_vec_kernel(const SsmArgs a) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
   }
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-    const int row = base + t;
+  typename Raw8<T>::V raw[kVecRows];                      // all rows in flight at once
+#pragma unroll
+  for (int i = 0; i < kVecRows; ++i) raw[i] = Raw8<T>::load(x + static_cast<size_t>(base + min(t0 + i, t1 - 1)) * a.ld_xz);
+#pragma unroll
+  for (int i = 0; i < kVecRows; ++i) {
+    if (t0 + i >= t1) break;
+    const int row = base + t0 + i;
     const bool real = row >= sp.row0;
     float xv[8], v[8];
-    ld8(x + static_cast<size_t>(row) * a.ld_xz, xv);
+    Raw8<T>::get(raw[i], xv);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       float y = bias[e];
@@ -178,36 +201,49 @@ __global__ void __launch_bounds__(256) ssm_conv_step_kernel(const SsmArgs a) {
 }
 
 // xp = sum of the split-K planes of the projection; its dt part once more in bf16, the operand of the next one.
-__global__ void __launch_bounds__(128) ssm_split_kernel(const SsmArgs a) {
+__global__ void __launch_bounds__(64) ssm_split_kernel(const SsmArgs a) {
   pdl_wait();
   pdl_launch_dependents();
   const size_t m = blockIdx.x;
-  const int n = a.dt_rank + 2 * a.state;
-  const float* src = a.xp_planes + m * n;
-  for (int i = threadIdx.x; i < n; i += 128) {
-    float v = src[i];
-#pragma unroll 8
-    for (int p = 1; p < a.planes; ++p) v += src[static_cast<size_t>(p) * a.M * n + i];
-    a.xp_out[m * a.ld_xp + i] = v;
-    if (i < a.dt_rank) a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(v);
-  }
+  const int n = a.dt_rank + 2 * a.state, i = blockIdx.y * 64 + threadIdx.x;
+  if (i >= n) return;
+  const float* src = a.xp_planes + m * n + i;
+  const size_t plane = static_cast<size_t>(a.M) * n;
+  float v = src[0];
+#pragma unroll 16
+  for (int p = 1; p < a.planes; ++p) v += src[p * plane];
+  a.xp_out[m * a.ld_xp + i] = v;
+  if (i < a.dt_rank) a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(v);
 }
 
-// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states; a block covers
-// CH = 128 / G channels.  Tiles of kTT rows of dt, u, z (per channel) and B, C (shared) come into shared memory by
-// cp.async, one tile ahead of the recurrence.  The work is bound by the exponentials (one per row, channel and state).
-constexpr int kScanThreads = 128;
-constexpr int kTT = 32;
+// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states; a warp works on its
+// CW = 32 / G channels alone (no block barriers, so the warps of an SM are in different phases): tiles of 8 to 32 rows of
+// dt, u, z (per channel) and B, C (shared) come into its shared memory by cp.async, one tile ahead; step sizes are
+// finished for the whole tile, the recurrence leaves per-lane partial outputs, and the last phase adds them, applies D
+// and the gate.  The bound is the exponentials: one per row, channel and state.
+constexpr int kScanWarps = 4;
 
-__device__ __forceinline__ void cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+template <int BYTES>
+__device__ __forceinline__ void cp_async(void* dst, const void* src) {
+  if constexpr (BYTES == 16)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  else
+    asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// nt rows of CW neighbouring elements -> dst [nt][CW], by one warp
+template <typename T, int CW>
+__device__ __forceinline__ void tile_rows(T* dst, const T* src, size_t ld_src, int nt, int lane) {
+  constexpr int kRow = CW * static_cast<int>(sizeof(T)), kPiece = kRow < 16 ? kRow : 16, kPer = kRow / kPiece, kElems = kPiece / static_cast<int>(sizeof(T));
+  for (int i = lane; i < nt * kPer; i += 32) {
+    const int t = i / kPer, q = i % kPer * kElems;
+    if constexpr (kPiece >= 4) cp_async<kPiece>(dst + t * CW + q, src + t * ld_src + q);
+    else dst[t * CW + q] = src[t * ld_src + q];
+  }
+}
 
 // fp32 runs take the accurate exponential, serving runs the hardware's base-2 one (A is scaled by log2 e for it)
 template <typename T>
@@ -229,52 +265,52 @@ struct Decay<__nv_bfloat16> {
 
 template <typename T, int G, int NS>
 struct ScanTile {
-  static constexpr int CH = kScanThreads / G, NSP = G * NS;
+  static constexpr int CW = 32 / G, NSP = G * NS;
+  static constexpr int kTT = NSP <= 64 ? 32 : NSP <= 128 ? 16 : 8;      // rows
   float B[kTT][NSP], C[kTT][NSP];
-  float dt[kTT][CH];
-  T u[kTT][CH], z[kTT][CH];
+  float dt[kTT][CW];
+  T u[kTT][CW], z[kTT][CW];
+};
+template <typename T, int G, int NS>
+struct ScanSmem {
+  static constexpr int kTT = ScanTile<T, G, NS>::kTT;
+  ScanTile<T, G, NS> tile[2];
+  float2 step[kTT][32 / G];        // (dt, dt u)
+  float y[kTT][32];                // per lane
 };
 
 template <typename T, int G, int NS>
-__global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const SsmArgs a) {
+__global__ void __launch_bounds__(32 * kScanWarps) ssm_scan_kernel(const SsmArgs a) {
   using Tile = ScanTile<T, G, NS>;
-  constexpr int CH = Tile::CH, NSP = Tile::NSP, kVec = 16 / static_cast<int>(sizeof(T));
+  constexpr int CW = Tile::CW, NSP = Tile::NSP, kTT = Tile::kTT;
   extern __shared__ __align__(16) unsigned char sc_smem[];
-  Tile* tiles = reinterpret_cast<Tile*>(sc_smem);
-  float(*sY)[CH] = reinterpret_cast<float(*)[CH]>(sc_smem + 2 * sizeof(Tile));
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  auto& sm = reinterpret_cast<ScanSmem<T, G, NS>*>(sc_smem)[warp];
   const SeqSpan sp = seq_span(a, blockIdx.y);
-  const int ch = threadIdx.x / G, g = threadIdx.x % G;
-  const int c0 = blockIdx.x * CH, c = c0 + ch;
+  const int ch = lane / G, g = lane % G;
+  const int c0 = (blockIdx.x * kScanWarps + warp) * CW, c = c0 + ch;
+  if (c0 >= a.inner) return;                             // whole warps only: nothing below synchronises the block
   const bool c_ok = c < a.inner;
-  const T* u = a.u ? reinterpret_cast<const T*>(a.u) : reinterpret_cast<const T*>(a.u_bf16);
-  const T* z = static_cast<const T*>(a.xz) + a.z0;
+  const T* u = (a.u ? reinterpret_cast<const T*>(a.u) : reinterpret_cast<const T*>(a.u_bf16)) + static_cast<size_t>(sp.row0) * a.ld_u + c0;
+  const T* z = static_cast<const T*>(a.xz) + static_cast<size_t>(sp.row0) * a.ld_xz + a.z0 + c0;
+  const float* dtp = a.dt_raw + static_cast<size_t>(sp.row0) * a.ld_u + c0;
+  const float* xp = a.xp + static_cast<size_t>(sp.row0) * a.ld_xp + a.dt_rank;
   auto fetch = [&](int t0, Tile& d) {
     const int nt = min(kTT, sp.n - t0);
-    for (int i = threadIdx.x; i < nt * (CH / 4); i += kScanThreads) {
-      const int t = i / (CH / 4), q = i % (CH / 4) * 4;
-      if (c0 + q < a.ld_u) cp16(&d.dt[t][q], a.dt_raw + static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + q);
-    }
-    constexpr int kRow = CH / kVec > 0 ? CH / kVec : 1;
-    static_assert(CH % kVec == 0, "whole 16-byte groups of channels");
-    for (int i = threadIdx.x; i < nt * kRow; i += kScanThreads) {
-      const int t = i / kRow, q = i % kRow * kVec;
-      if (c0 + q >= a.ld_u) continue;
-      const size_t m = static_cast<size_t>(sp.row0 + t0 + t);
-      cp16(&d.u[t][q], u + m * a.ld_u + c0 + q);
-      cp16(&d.z[t][q], z + m * a.ld_xz + c0 + q);
-    }
-    for (int i = threadIdx.x; i < nt * NSP; i += kScanThreads) {
-      const int t = i / NSP, n = i % NSP;
-      if (n >= a.state) continue;                        // stays zero
-      const float* row = a.xp + static_cast<size_t>(sp.row0 + t0 + t) * a.ld_xp + a.dt_rank + n;
-      cp4(&d.B[t][n], row);
-      cp4(&d.C[t][n], row + a.state);
+    tile_rows<float, CW>(&d.dt[0][0], dtp + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
+    tile_rows<T, CW>(&d.u[0][0], u + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
+    tile_rows<T, CW>(&d.z[0][0], z + static_cast<size_t>(t0) * a.ld_xz, a.ld_xz, nt, lane);
+    for (int n = lane; n < 2 * a.state; n += 32) {       // B then C: neighbours in the row
+      float* dst = n < a.state ? &d.B[0][n] : &d.C[0][n - a.state];
+      const float* src = xp + static_cast<size_t>(t0) * a.ld_xp + n;
+#pragma unroll 8
+      for (int t = 0; t < nt; ++t) cp_async<4>(dst + t * NSP, src + static_cast<size_t>(t) * a.ld_xp);
     }
     cp_commit();
   };
-  for (int i = threadIdx.x; i < static_cast<int>(2 * sizeof(Tile) / 4); i += kScanThreads) reinterpret_cast<float*>(tiles)[i] = 0.f;
-  __syncthreads();
-  if (sp.n > 0) fetch(0, tiles[0]);
+  for (int i = lane; i < static_cast<int>(2 * sizeof(Tile) / 4); i += 32) reinterpret_cast<float*>(sm.tile)[i] = 0.f;   // padded states stay zero
+  __syncwarp();
+  if (sp.n > 0) fetch(0, sm.tile[0]);
   float S[NS], A[NS];
   float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + (c_ok ? c : 0)) * a.state;
 #pragma unroll
@@ -284,52 +320,56 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const SsmArgs a)
     A[i] = ok ? a.A[static_cast<size_t>(c) * a.state + n] * Decay<T>::kScale : 0.f;
     S[i] = (ok && sp.start > 0 && sp.n > 0) ? state[n] : 0.f;
   }
-  // rows in front of the sequence's start give zeros
-  for (int i = threadIdx.x; i < (a.rows.Tc - sp.n) * CH; i += kScanThreads) {
-    const int t = i / CH, cc = c0 + i % CH;
-    if (cc < a.inner) {
-      const size_t o = (static_cast<size_t>(blockIdx.y) * a.rows.Tc + t) * a.ld_u + cc;
-      if (a.out) a.out[o] = 0.f;
-      if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(0.f);
-    }
-  }
-  // the channel a thread finishes (softplus, gate) is the same in every round: CH divides the block
-  const int fc = threadIdx.x % CH, f_ok = c0 + fc < a.inner;
+  // phases over (row, channel) pairs: lane -> channel fc, rows t = ft, ft + G, ...
+  const int fc = lane % CW, ft = lane / CW;
+  const bool f_ok = c0 + fc < a.inner;
   const float dt_b = f_ok ? a.dt_b[c0 + fc] : 0.f, D = f_ok ? a.D[c0 + fc] : 0.f;
+  // rows in front of the sequence's start give zeros
+  for (int t = ft; t < a.rows.Tc - sp.n; t += G) {
+    const size_t o = (static_cast<size_t>(blockIdx.y) * a.rows.Tc + t) * a.ld_u + c0 + fc;
+    if (f_ok && a.out) a.out[o] = 0.f;
+    if (f_ok && a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(0.f);
+  }
   for (int t0 = 0, k = 0; t0 < sp.n; t0 += kTT, ++k) {
-    Tile& d = tiles[k & 1];
+    Tile& d = sm.tile[k & 1];
     const int nt = min(kTT, sp.n - t0);
     if (t0 + kTT < sp.n) {
-      fetch(t0 + kTT, tiles[(k + 1) & 1]);
+      fetch(t0 + kTT, sm.tile[(k + 1) & 1]);
       cp_wait<1>();
     } else {
       cp_wait<0>();
     }
-    __syncthreads();
-    for (int t = threadIdx.x / CH; t < nt; t += G) d.dt[t][fc] = f_ok ? softplus(d.dt[t][fc] + dt_b) : 0.f;
-    __syncthreads();
+    __syncwarp();
 #pragma unroll 4
+    for (int t = ft; t < nt; t += G) {
+      const float dt = f_ok ? softplus(d.dt[t][fc] + dt_b) : 0.f;
+      sm.step[t][fc] = make_float2(dt, dt * ld(&d.u[t][fc], 0));
+    }
+    __syncwarp();
+#pragma unroll 8
     for (int t = 0; t < nt; ++t) {
-      const float dt = d.dt[t][ch], du = dt * ld(&d.u[t][ch], 0);
+      const float2 st = sm.step[t][ch];
       float y = 0.f;
 #pragma unroll
       for (int i = 0; i < NS; ++i) {
-        S[i] = fmaf(Decay<T>::f(dt * A[i]), S[i], du * d.B[t][g * NS + i]);
+        S[i] = fmaf(Decay<T>::f(st.x * A[i]), S[i], st.y * d.B[t][g * NS + i]);
         y = fmaf(S[i], d.C[t][g * NS + i], y);
       }
-#pragma unroll
-      for (int o = G / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (g == 0) sY[t][ch] = y;
+      sm.y[t][lane] = y;
     }
-    __syncthreads();
-    for (int t = threadIdx.x / CH; t < nt; t += G) {
+    __syncwarp();
+#pragma unroll 4
+    for (int t = ft; t < nt; t += G) {
       if (!f_ok) break;
-      const float y = fmaf(D, ld(&d.u[t][fc], 0), sY[t][fc]) * silu(ld(&d.z[t][fc], 0));
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < G; ++i) y += sm.y[t][fc * G + i];
+      y = fmaf(D, ld(&d.u[t][fc], 0), y) * silu(ld(&d.z[t][fc], 0));
       const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + fc;
       if (a.out) a.out[o] = y;
       if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
     }
-    __syncthreads();                                     // the tile may be fetched over, sY written again
+    __syncwarp();                                        // the tile may be fetched over, y written again
   }
   if (c_ok && sp.n > 0) {
 #pragma unroll
@@ -358,7 +398,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
   float4 s4 = make_float4(0.f, 0.f, 0.f, 0.f);
   if (VEC && 4 * g < a.state && sp.start > 0) s4 = *reinterpret_cast<const float4*>(state + 4 * g);
   const int np = a.ld_wdt + 2 * a.state;                  // the dt part padded with zeros to the weight's row length
-  for (int i = threadIdx.x; i < np; i += 256) {
+  for (int i = (a.dt_raw ? a.ld_wdt : 0) + threadIdx.x; i < np; i += 256) {
     const float* row = a.xp + static_cast<size_t>(m) * a.ld_xp;
     st_smem[i] = i < a.dt_rank ? row[i] : i < a.ld_wdt ? 0.f : row[a.dt_rank + i - a.ld_wdt];
   }
@@ -420,27 +460,24 @@ bool ssm_ok(const SsmArgs& a) {
 
 template <typename T, int G, int NS>
 cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
-  using Tile = ScanTile<T, G, NS>;
-  constexpr int smem = static_cast<int>(2 * sizeof(Tile) + sizeof(float) * kTT * Tile::CH);
+  constexpr int smem = static_cast<int>(kScanWarps * sizeof(ScanSmem<T, G, NS>)), CH = kScanWarps * 32 / G;
+  static_assert(smem <= 220 * 1024, "shared memory");
   static DeviceOnce once;
   cudaError_t e = once.run([&] {
     return cudaFuncSetAttribute(ssm_scan_kernel<T, G, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   });
   if (e != cudaSuccess) return e;
-  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + Tile::CH - 1) / Tile::CH, a.nseq), kScanThreads, smem, s>>>(a);
+  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CH - 1) / CH, a.nseq), 32 * kScanWarps, smem, s>>>(a);
   return cudaGetLastError();
 }
 
 template <typename T>
 cudaError_t scan_states(const SsmArgs& a, cudaStream_t s) {
-  // few channels: more lanes per channel, so that every scheduler has a few warps
-  const bool few = static_cast<int64_t>(a.inner) * a.nseq < 148 * 2 * 32;
-  if (a.state <= 8) return scan<T, 4, 2>(a, s);
-  if (a.state <= 16) return few ? scan<T, 8, 2>(a, s) : scan<T, 4, 4>(a, s);
+  if (a.state <= 16) return scan<T, 4, 4>(a, s);
   if (a.state <= 32) return scan<T, 8, 4>(a, s);
   if (a.state <= 64) return scan<T, 16, 4>(a, s);
-  if (a.state <= 128) return scan<T, 16, 8>(a, s);
-  return scan<T, 16, 16>(a, s);
+  if (a.state <= 128) return scan<T, 32, 4>(a, s);
+  return scan<T, 32, 8>(a, s);
 }
 
 template <typename T, int G, bool VEC>
@@ -491,7 +528,7 @@ cudaError_t launch_ssm_conv(const SsmArgs& a, cudaStream_t s, bool pdl) {
 
 cudaError_t launch_ssm_split(const SsmArgs& a, cudaStream_t s, bool pdl) {
   if (!ssm_ok(a) || !a.dtr_bf16 || !a.xp_planes || !a.xp_out || a.planes < 1) return cudaErrorInvalidValue;
-  return launch_pdl(ssm_split_kernel, dim3(a.M), dim3(128), 0, s, pdl, a);
+  return launch_pdl(ssm_split_kernel, dim3(a.M, (a.dt_rank + 2 * a.state + 63) / 64), dim3(64), 0, s, pdl, a);
 }
 
 cudaError_t launch_ssm_scan(const SsmArgs& a, cudaStream_t s) {

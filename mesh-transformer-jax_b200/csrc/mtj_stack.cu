@@ -201,7 +201,7 @@ void LayerStack::carve_workspace(Carver& c) {
     xz_bf_ = c.take<__nv_bfloat16>(R * xz);
     u_bf_ = c.take<__nv_bfloat16>(R * u);
     dtr_bf_ = c.take<__nv_bfloat16>(R * dtr);
-    xp_planes_elems_ = xp * std::max<int64_t>(4 * R, 32 * std::min<int64_t>(R, 128));
+    xp_planes_elems_ = xp * std::max<int64_t>(6 * R, 16 * std::min<int64_t>(R, 128));
     xp_planes_ = c.take<float>(xp_planes_elems_);
     act_bf_ = c.take<__nv_bfloat16>(R * act);
     q_pack_ = c.take<__nv_bfloat16>(R * qp);
@@ -427,7 +427,7 @@ int32_t LayerStack::gemm_planes(mtj_handle* h, const Linear& l, const __nv_bfloa
   a.N = l.N;
   a.K = l.K;
   a.partial = xp_planes_;
-  a.ksplit = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({fit, 296 / tiles, (l.K + 127) / 128, 32})));
+  a.ksplit = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>({fit, 296 / tiles, (l.K + 127) / 128, 16})));
   a.dev_err = h->dev_err;
   MTJ_CUDA(launch_gemm_tc(kEpiPlain, &l.map, key, a, s, decode && h->use_pdl && h->tc_pdl));
   h->launches++;
