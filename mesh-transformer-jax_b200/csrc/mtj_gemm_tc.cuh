@@ -299,6 +299,26 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
     tc_fence_after();
     auto do_chunk = [&](int cc, uint32_t (&r)[32]) {
         const int c0 = cc * 32;
+        if constexpr (EPI == kEpiPlain) {
+          // one destination per loop: short code, which matters because every block runs it once
+          const int valid = n_ok ? min(32, a.M - (m0 + c0)) : 0;
+          float* dst = a.partial ? a.partial + (static_cast<size_t>(blockIdx.z) * a.M + m0 + c0) * a.N + n
+                                 : a.out ? a.out + static_cast<size_t>(m0 + c0) * a.ld_out + n : nullptr;
+          const size_t ldd = a.partial ? a.N : a.ld_out;
+          const float add = a.partial ? 0.f : bias;
+          if (dst) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (i < valid) dst[i * ldd] = __uint_as_float(r[i]) + add;
+          }
+          if (a.out_bf16 && !a.partial) {
+            __nv_bfloat16* d16 = a.out_bf16 + static_cast<size_t>(m0 + c0) * a.ld_bf16 + n;
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (i < valid) d16[static_cast<size_t>(i) * a.ld_bf16] = __float2bfloat16_rn(__uint_as_float(r[i]) + add);
+          }
+          return;
+        }
         if (dec) {
           const int pos = dpos;
           const bool any_rot = __any_sync(0xffffffffu, rotary);
@@ -389,9 +409,6 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
             float y = v + bias;
             if (a.residual) y += a.residual[static_cast<size_t>(m) * a.N + n];
             a.out[static_cast<size_t>(m) * a.N + n] = y;
-          } else if (EPI == kEpiPlain) {
-            if (a.out) a.out[static_cast<size_t>(m) * a.ld_out + n] = v + bias;
-            if (a.out_bf16) a.out_bf16[static_cast<size_t>(m) * a.ld_bf16 + n] = __float2bfloat16_rn(v + bias);
           } else {
             a.out[static_cast<size_t>(m) * a.ld_out + n] = v + bias;
           }
@@ -437,7 +454,7 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
         for (int cc = 0; cc < kChunks; ++cc) do_chunk(cc, racc[cc]);
       }
     } else if (ok || (nk == 0 && a.partial)) {
-#pragma unroll
+#pragma unroll(EPI == kEpiPlain ? 1 : kChunks)
       for (int cc = 0; cc < kChunks; ++cc) {
         uint32_t r[32];
         if (ok) {

@@ -80,36 +80,51 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
   const int m0 = blockIdx.x * RT, nr = min(RT, a.M - m0);
   if (blockIdx.y == a.heads) {
     if (blockIdx.z) return;
-    for (int r = 0; r < nr; ++r) {
+    // one row: the whole block; several: a warp per row
+    constexpr int kW = RT == 1 ? kThreads : 32;
+    const int lane = threadIdx.x % kW;
+    for (int r = threadIdx.x / kW; r < nr; r += kThreads / kW) {
       int seq;
       const int p = own_pos(a.rows, a.pad, m0 + r, &seq);
       const float* c = a.p1 + static_cast<size_t>(m0 + r) * a.ld_p1 + a.heads * (a.dim + a.rot);
-      float ss = 0.f;
-      for (int i = threadIdx.x; i < a.rank; i += kThreads) ss = fmaf(c[i], c[i], ss);
-      const float rs = 1.0f / sqrtf(la_block_sum(ss, red) / static_cast<float>(a.rank) + a.eps);
+      constexpr int kC = kLatentMaxRank / kW;
+      float cv[kC], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < kC; ++i) cv[i] = i * kW + lane < a.rank ? c[i * kW + lane] : 0.f;
+#pragma unroll
+      for (int i = 0; i < kC; ++i) ss = fmaf(cv[i], cv[i], ss);
+      ss = RT == 1 ? la_block_sum(ss, red) : warp_sum(ss);
+      const float rs = 1.0f / sqrtf(ss / static_cast<float>(a.rank) + a.eps);
       if (p < 0) continue;
       T* row = static_cast<T*>(a.cache.pool) + cache_row(a.cache, seq, p);
-      for (int i = threadIdx.x; i < a.rank; i += kThreads) st(row + i, c[i] * rs * a.kv_norm[i]);
       const float2* sc = a.sincos + static_cast<size_t>(p) * (a.rot >> 1);
-      for (int j = threadIdx.x; j < a.rot; j += kThreads) st(row + a.cache.kv_ld + j, rotated(c + a.rank, j, sc));
+      for (int j = lane; j < a.rot; j += kW) st(row + a.cache.kv_ld + j, rotated(c + a.rank, j, sc));
+#pragma unroll
+      for (int i = 0; i < kC; ++i)
+        if (i * kW + lane < a.rank) st(row + i * kW + lane, cv[i] * rs * a.kv_norm[i * kW + lane]);
     }
     return;
   }
   const int h = blockIdx.y, hd = a.dim + a.rot;
   float* qs = ab_smem;                                  // [RT][dim]
-  float* part = ab_smem + RT * a.dim;                   // [dsplit][RT][kv_ld]
-  for (int r = 0; r < RT; ++r) {
-    const int m = m0 + min(r, nr - 1);
-    const float* q = a.p1 + static_cast<size_t>(m) * a.ld_p1 + h * hd;
-    for (int j = threadIdx.x; j < a.dim; j += kThreads) qs[r * a.dim + j] = q[j] * a.scale;
-    if (r < nr && blockIdx.z == 0) {
-      int seq;
-      const int p = max(own_pos(a.rows, a.pad, m, &seq), 0);
-      const float2* sc = a.sincos + static_cast<size_t>(p) * (a.rot >> 1);
-      float* o = a.q_abs + (static_cast<size_t>(m) * a.heads + h) * a.cache.row_ld + a.cache.kv_ld;
-      for (int j = threadIdx.x; j < a.cache.row_ld - a.cache.kv_ld; j += kThreads)
-        o[j] = j < a.rot ? rotated(q + a.dim, j, sc) * a.scale : 0.f;
-    }
+  float* part = ab_smem + RT * a.dim;                   // [dsplit][RT][cols]
+  {
+    const float* q = a.p1 + static_cast<size_t>(m0) * a.ld_p1 + h * hd;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < nr * a.dim; i += kThreads)
+      qs[i] = q[static_cast<size_t>(i / a.dim) * a.ld_p1 + i % a.dim] * a.scale;
+    for (int i = nr * a.dim + threadIdx.x; i < RT * a.dim; i += kThreads) qs[i] = 0.f;
+    const int rot_ld = a.cache.row_ld - a.cache.kv_ld;
+    if (blockIdx.z == 0)
+#pragma unroll 2
+      for (int i = threadIdx.x; i < nr * rot_ld; i += kThreads) {
+        const int r = i / rot_ld, j = i % rot_ld;
+        int seq;
+        const int p = max(own_pos(a.rows, a.pad, m0 + r, &seq), 0);
+        const float2* sc = a.sincos + static_cast<size_t>(p) * (a.rot >> 1);
+        a.q_abs[(static_cast<size_t>(m0 + r) * a.heads + h) * a.cache.row_ld + a.cache.kv_ld + j] =
+            j < a.rot ? rotated(q + static_cast<size_t>(r) * a.ld_p1 + a.dim, j, sc) * a.scale : 0.f;
+      }
   }
   __syncthreads();
   if (ds < dsplit) {
@@ -492,15 +507,22 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
   // RT == 1: two threads share a column group, each adding half of the ranges
   constexpr int kParts = RT == 1 ? 2 : 1;
   const int k4 = kv_ld >> 2;
+#pragma unroll 2
   for (int i = threadIdx.x; i < kParts * nr * k4; i += kThreads) {
     const int part = i / (nr * k4), j = i % (nr * k4), r = j / k4, k = j % k4;
     const float4* po = reinterpret_cast<const float4*>(a.part_o + (static_cast<size_t>(m0 + r) * a.heads + h) * a.splits * kv_ld) + k;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 16
-    for (int s = part; s < a.splits; s += kParts) {
-      const float4 p = po[static_cast<size_t>(s) * k4];
-      const float e = ws[r][s];
-      v.x = fmaf(e, p.x, v.x); v.y = fmaf(e, p.y, v.y); v.z = fmaf(e, p.z, v.z); v.w = fmaf(e, p.w, v.w);
+    constexpr int kIn = RT == 1 ? 16 : 4;                // loads in flight
+    for (int s0 = part; s0 < a.splits; s0 += kIn * kParts) {
+      float4 p[kIn];
+#pragma unroll
+      for (int i = 0; i < kIn; ++i) p[i] = po[static_cast<size_t>(min(s0 + i * kParts, a.splits - 1)) * k4];
+#pragma unroll
+      for (int i = 0; i < kIn; ++i) {
+        const int s = s0 + i * kParts;
+        const float e = s < a.splits ? ws[r][s] : 0.f;
+        v.x = fmaf(e, p[i].x, v.x); v.y = fmaf(e, p[i].y, v.y); v.z = fmaf(e, p[i].z, v.z); v.w = fmaf(e, p[i].w, v.w);
+      }
     }
     reinterpret_cast<float4*>(lo_smem)[i] = v;
   }

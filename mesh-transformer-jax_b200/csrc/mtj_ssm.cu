@@ -14,8 +14,25 @@ namespace {
 
 __device__ __forceinline__ float ld(const float* p, size_t i) { return p[i]; }
 __device__ __forceinline__ float ld(const __nv_bfloat16* p, size_t i) { return __bfloat162float(p[i]); }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float silu_exact(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_exact(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// Elementwise functions of a run with T operands: the accurate ones for fp32 runs; serving runs, whose inputs carry bf16
+// rounding, take the fast fp32 intrinsics (log(1 + e) by its series where 1 + e would round e away).
+template <typename T>
+struct Fn;
+template <>
+struct Fn<float> {
+  __device__ static __forceinline__ float silu(float z) { return silu_exact(z); }
+  __device__ static __forceinline__ float softplus(float z) { return softplus_exact(z); }
+};
+template <>
+struct Fn<__nv_bfloat16> {
+  __device__ static __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+  __device__ static __forceinline__ float softplus(float z) {
+    const float e = __expf(-fabsf(z));
+    return fmaxf(z, 0.f) + (e < 0.01f ? e * (1.0f - e * (0.5f - e * 0.33333333f)) : __logf(1.0f + e));
+  }
+};
 
 struct SeqSpan {
   int seq, start, n, row0;       // slot, own position of the first real row, real rows, its row index
@@ -58,7 +75,7 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
         v = fmaf(a.conv_w[static_cast<size_t>(j) * a.ld_u + c], xv, v);
       }
     }
-    v = rel >= 0 ? silu(v) : 0.f;
+    v = rel >= 0 ? Fn<T>::silu(v) : 0.f;
     const size_t o = static_cast<size_t>(row) * a.ld_u + c;
     if (a.u) a.u[o] = v;
     if (a.u_bf16) a.u_bf16[o] = __float2bfloat16_rn(v);
@@ -67,7 +84,7 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a) {
 
 // The same for at most four taps, a thread owning eight neighbouring channels: it walks kVecRows rows with the last
 // TAPS - 1 inputs in registers, one 16-byte load per row.  Columns between inner and the row stride hold zeros.
-constexpr int kVecRows = 8;
+constexpr int kVecRows = 16;
 
 __device__ __forceinline__ void ld8(const __nv_bfloat16* p, float* f) { unpack8(*reinterpret_cast<const uint4*>(p), f); }
 __device__ __forceinline__ void ld8(const float* p, float* f) {
@@ -117,23 +134,25 @@ __global__ void __launch_bounds__(128) ssm_conv_vec_kernel(const SsmArgs a) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
   }
-  typename Raw8<T>::V raw[kVecRows];                      // all rows in flight at once
-#pragma unroll
-  for (int i = 0; i < kVecRows; ++i) raw[i] = Raw8<T>::load(x + static_cast<size_t>(base + min(t0 + i, t1 - 1)) * a.ld_xz);
-#pragma unroll
-  for (int i = 0; i < kVecRows; ++i) {
-    if (t0 + i >= t1) break;
-    const int row = base + t0 + i;
+  // two rows ahead in registers; the loop stays rolled, so its code is fetched once
+  typename Raw8<T>::V raw0 = Raw8<T>::load(x + static_cast<size_t>(base + t0) * a.ld_xz);
+  typename Raw8<T>::V raw1 = Raw8<T>::load(x + static_cast<size_t>(base + min(t0 + 1, t1 - 1)) * a.ld_xz);
+#pragma unroll 1
+  for (int t = t0; t < t1; ++t) {
+    const typename Raw8<T>::V cur = raw0;
+    raw0 = raw1;
+    raw1 = Raw8<T>::load(x + static_cast<size_t>(base + min(t + 2, t1 - 1)) * a.ld_xz);
+    const int row = base + t;
     const bool real = row >= sp.row0;
     float xv[8], v[8];
-    Raw8<T>::get(raw[i], xv);
+    Raw8<T>::get(cur, xv);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       float y = bias[e];
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) y = fmaf(w[j][e], hist[j][e], y);
       y = fmaf(w[TAPS - 1][e], xv[e], y);
-      v[e] = real ? silu(y) : 0.f;
+      v[e] = real ? Fn<T>::silu(y) : 0.f;
     }
     if (real) {
       if constexpr (TAPS > 1) {
@@ -194,7 +213,7 @@ __global__ void __launch_bounds__(256) ssm_conv_step_kernel(const SsmArgs a) {
     if (j > 0) st[static_cast<size_t>(j - 1) * a.ld_u] = xv;
   }
   if (a.taps > 1) st[static_cast<size_t>(a.taps - 2) * a.ld_u] = x;
-  v = silu(v);
+  v = Fn<T>::silu(v);
   const size_t o = static_cast<size_t>(m) * a.ld_u + c;
   if (a.u) a.u[o] = v;
   if (a.u_bf16) a.u_bf16[o] = __float2bfloat16_rn(v);
@@ -221,7 +240,7 @@ __global__ void __launch_bounds__(64) ssm_split_kernel(const SsmArgs a) {
 // dt, u, z (per channel) and B, C (shared) come into its shared memory by cp.async, one tile ahead; step sizes are
 // finished for the whole tile, the recurrence leaves per-lane partial outputs, and the last phase adds them, applies D
 // and the gate.  The bound is the exponentials: one per row, channel and state.
-constexpr int kScanWarps = 4;
+constexpr int kScanWarps = 2;
 
 template <int BYTES>
 __device__ __forceinline__ void cp_async(void* dst, const void* src) {
@@ -242,6 +261,20 @@ __device__ __forceinline__ void tile_rows(T* dst, const T* src, size_t ld_src, i
     const int t = i / kPer, q = i % kPer * kElems;
     if constexpr (kPiece >= 4) cp_async<kPiece>(dst + t * CW + q, src + t * ld_src + q);
     else dst[t * CW + q] = src[t * ld_src + q];
+  }
+}
+
+template <int NS>
+__device__ __forceinline__ void load_states(const float* p, float* v) {
+  if constexpr (NS == 2) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < NS; i += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p + i);
+      v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
+    }
   }
 }
 
@@ -340,34 +373,75 @@ __global__ void __launch_bounds__(32 * kScanWarps) ssm_scan_kernel(const SsmArgs
       cp_wait<0>();
     }
     __syncwarp();
-#pragma unroll 4
-    for (int t = ft; t < nt; t += G) {
-      const float dt = f_ok ? softplus(d.dt[t][fc] + dt_b) : 0.f;
-      sm.step[t][fc] = make_float2(dt, dt * ld(&d.u[t][fc], 0));
-    }
-    __syncwarp();
-#pragma unroll 8
-    for (int t = 0; t < nt; ++t) {
-      const float2 st = sm.step[t][ch];
-      float y = 0.f;
+    // Each phase reads a group of rows into registers before it writes: the compiler cannot move shared-memory loads
+    // over stores whose addresses it does not know.
+    constexpr int kR = kTT / G > 0 ? kTT / G : 1;        // rows per lane of the elementwise phases
+    {
+      float raw[kR], uu[kR];
 #pragma unroll
-      for (int i = 0; i < NS; ++i) {
-        S[i] = fmaf(Decay<T>::f(st.x * A[i]), S[i], st.y * d.B[t][g * NS + i]);
-        y = fmaf(S[i], d.C[t][g * NS + i], y);
+      for (int i = 0; i < kR; ++i) {
+        const int t = min(ft + i * G, kTT - 1);
+        raw[i] = d.dt[t][fc];
+        uu[i] = ld(&d.u[t][fc], 0);
       }
-      sm.y[t][lane] = y;
+#pragma unroll
+      for (int i = 0; i < kR; ++i) {
+        const float dt = f_ok ? Fn<T>::softplus(raw[i] + dt_b) : 0.f;
+        if (ft + i * G < kTT) sm.step[ft + i * G][fc] = make_float2(dt, dt * uu[i]);
+      }
     }
     __syncwarp();
-#pragma unroll 4
-    for (int t = ft; t < nt; t += G) {
-      if (!f_ok) break;
-      float y = 0.f;
+    constexpr int kU = 4;                                // rows per group of the recurrence
+    static_assert(kTT % kU == 0 && (NS == 2 || NS % 4 == 0), "whole groups");
+    auto group = [&](int t1, int rows_left) {
+      float2 st[kU];
+      float Bv[kU][NS], Cv[kU][NS];
 #pragma unroll
-      for (int i = 0; i < G; ++i) y += sm.y[t][fc * G + i];
-      y = fmaf(D, ld(&d.u[t][fc], 0), y) * silu(ld(&d.z[t][fc], 0));
-      const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + fc;
-      if (a.out) a.out[o] = y;
-      if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
+      for (int r = 0; r < kU; ++r) {
+        st[r] = sm.step[t1 + r][ch];
+        load_states<NS>(&d.B[t1 + r][g * NS], Bv[r]);
+        load_states<NS>(&d.C[t1 + r][g * NS], Cv[r]);
+      }
+      float y[kU];
+#pragma unroll
+      for (int r = 0; r < kU; ++r) {
+        y[r] = 0.f;
+        if (r < rows_left) {
+#pragma unroll
+          for (int i = 0; i < NS; ++i) {
+            S[i] = fmaf(Decay<T>::f(st[r].x * A[i]), S[i], st[r].y * Bv[r][i]);
+            y[r] = fmaf(S[i], Cv[r][i], y[r]);
+          }
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < kU; ++r) sm.y[t1 + r][lane] = y[r];
+    };
+    if (nt == kTT) {
+#pragma unroll 2
+      for (int t = 0; t < kTT; t += kU) group(t, kU);
+    } else {
+      for (int t = 0; t < nt; t += kU) group(t, nt - t);
+    }
+    __syncwarp();
+    {
+      float yv[kR];
+#pragma unroll
+      for (int i = 0; i < kR; ++i) {
+        const int t = min(ft + i * G, kTT - 1);
+        float y = 0.f;
+#pragma unroll
+        for (int j = 0; j < G; ++j) y += sm.y[t][fc * G + j];
+        yv[i] = fmaf(D, ld(&d.u[t][fc], 0), y) * Fn<T>::silu(ld(&d.z[t][fc], 0));
+      }
+#pragma unroll
+      for (int i = 0; i < kR; ++i) {
+        const int t = ft + i * G;
+        if (!f_ok || t >= nt) continue;
+        const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + fc;
+        if (a.out) a.out[o] = yv[i];
+        if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(yv[i]);
+      }
     }
     __syncwarp();                                        // the tile may be fetched over, y written again
   }
@@ -397,16 +471,17 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
   float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + cc) * a.state;
   float4 s4 = make_float4(0.f, 0.f, 0.f, 0.f);
   if (VEC && 4 * g < a.state && sp.start > 0) s4 = *reinterpret_cast<const float4*>(state + 4 * g);
+  float dt = a.dt_raw ? a.dt_raw[static_cast<size_t>(m) * a.ld_u + cc] : 0.f;
+  const float u = a.u ? a.u[static_cast<size_t>(m) * a.ld_u + cc] : __bfloat162float(a.u_bf16[static_cast<size_t>(m) * a.ld_u + cc]);
+  const float z = ld(static_cast<const T*>(a.xz), static_cast<size_t>(m) * a.ld_xz + a.z0 + cc);
+  const float dt_b = a.dt_b[cc], D = a.D[cc];
   const int np = a.ld_wdt + 2 * a.state;                  // the dt part padded with zeros to the weight's row length
   for (int i = (a.dt_raw ? a.ld_wdt : 0) + threadIdx.x; i < np; i += 256) {
     const float* row = a.xp + static_cast<size_t>(m) * a.ld_xp;
     st_smem[i] = i < a.dt_rank ? row[i] : i < a.ld_wdt ? 0.f : row[a.dt_rank + i - a.ld_wdt];
   }
   __syncthreads();
-  float dt = 0.f;
-  if (a.dt_raw) {
-    dt = a.dt_raw[static_cast<size_t>(m) * a.ld_u + cc];
-  } else {
+  if (!a.dt_raw) {
 #pragma unroll 4
     for (int k = g * 8; k < a.ld_wdt; k += G * 8) {
       float w8[8];
@@ -417,8 +492,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
 #pragma unroll
     for (int o = G / 2; o > 0; o >>= 1) dt += __shfl_xor_sync(0xffffffffu, dt, o);
   }
-  dt = softplus(dt + a.dt_b[cc]);
-  const float u = a.u ? a.u[static_cast<size_t>(m) * a.ld_u + cc] : __bfloat162float(a.u_bf16[static_cast<size_t>(m) * a.ld_u + cc]);
+  dt = Fn<T>::softplus(dt + dt_b);
   const float du = dt * u;
   const float* B = st_smem + a.ld_wdt;
   const float* C = B + a.state;
@@ -444,8 +518,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
 #pragma unroll
   for (int o = G / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
   if (ok && g == 0) {
-    const float z = ld(static_cast<const T*>(a.xz), static_cast<size_t>(m) * a.ld_xz + a.z0 + c);
-    y = fmaf(a.D[c], u, y) * silu(z);
+    y = fmaf(D, u, y) * Fn<T>::silu(z);
     const size_t o = static_cast<size_t>(m) * a.ld_u + c;
     if (a.out) a.out[o] = y;
     if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(y);
@@ -473,7 +546,9 @@ cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
 
 template <typename T>
 cudaError_t scan_states(const SsmArgs& a, cudaStream_t s) {
-  if (a.state <= 16) return scan<T, 4, 4>(a, s);
+  // one prompt: more lanes per channel, so that every scheduler has a few warps to issue from
+  const bool few = static_cast<int64_t>(a.inner) * a.nseq <= 148 * 4 * 32;
+  if (a.state <= 16) return few ? scan<T, 8, 2>(a, s) : scan<T, 4, 4>(a, s);
   if (a.state <= 32) return scan<T, 8, 4>(a, s);
   if (a.state <= 64) return scan<T, 16, 4>(a, s);
   if (a.state <= 128) return scan<T, 32, 4>(a, s);
