@@ -319,6 +319,18 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
           }
           return;
         }
+        if constexpr (EPI == kEpiSwiGLU) {
+          // rows come in (gate, up) pairs: the even lane finishes the pair
+          const int valid = n_ok ? min(32, a.M - (m0 + c0)) : 0;
+          __nv_bfloat16* d16 = a.out_bf16 + static_cast<size_t>(m0 + c0) * a.ld_bf16 + (n >> 1);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float v = __uint_as_float(r[i]);
+            const float partner = __shfl_xor_sync(0xffffffffu, v, 1);
+            if (i < valid && !(lane & 1)) d16[static_cast<size_t>(i) * a.ld_bf16] = __float2bfloat16_rn(swiglu(v, partner));
+          }
+          return;
+        }
         if (dec) {
           const int pos = dpos;
           const bool any_rot = __any_sync(0xffffffffu, rotary);
@@ -399,9 +411,6 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
               a.act_out[static_cast<size_t>(m) * (a.dl + a.ffl) + a.dl + nn] =
                   __float2bfloat16_rn(gelu_tanh(v + bias));
             }
-          } else if (EPI == kEpiSwiGLU) {
-            // rows come in (gate, up) pairs: the even lane finishes the pair
-            if (!(lane & 1)) a.out_bf16[static_cast<size_t>(m) * a.ld_bf16 + (n >> 1)] = __float2bfloat16_rn(swiglu(v, partner));
           } else if (a.partial) {
             // split-K: raw partial sum; bias / residual are added by the reduction kernel
             a.partial[(static_cast<size_t>(blockIdx.z) * a.M + m) * a.N + n] = v;
@@ -454,7 +463,7 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
         for (int cc = 0; cc < kChunks; ++cc) do_chunk(cc, racc[cc]);
       }
     } else if (ok || (nk == 0 && a.partial)) {
-#pragma unroll(EPI == kEpiPlain ? 1 : kChunks)
+#pragma unroll(EPI >= kEpiPlain ? 1 : kChunks)
       for (int cc = 0; cc < kChunks; ++cc) {
         uint32_t r[32];
         if (ok) {

@@ -266,15 +266,10 @@ __device__ __forceinline__ void tile_rows(T* dst, const T* src, size_t ld_src, i
 
 template <int NS>
 __device__ __forceinline__ void load_states(const float* p, float* v) {
-  if constexpr (NS == 2) {
-    const float2 f = *reinterpret_cast<const float2*>(p);
-    v[0] = f.x; v[1] = f.y;
-  } else {
 #pragma unroll
-    for (int i = 0; i < NS; i += 4) {
-      const float4 f = *reinterpret_cast<const float4*>(p + i);
-      v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
-    }
+  for (int i = 0; i < NS; i += 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p + i);
+    v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
   }
 }
 
@@ -309,7 +304,7 @@ struct ScanSmem {
   static constexpr int kTT = ScanTile<T, G, NS>::kTT;
   ScanTile<T, G, NS> tile[2];
   float2 step[kTT][32 / G];        // (dt, dt u)
-  float y[kTT][32];                // per lane
+  float y[kTT][33];                // per lane; the padding spreads the last phase's reads over the banks
 };
 
 template <typename T, int G, int NS>
@@ -328,12 +323,21 @@ __global__ void __launch_bounds__(32 * kScanWarps) ssm_scan_kernel(const SsmArgs
   const T* z = static_cast<const T*>(a.xz) + static_cast<size_t>(sp.row0) * a.ld_xz + a.z0 + c0;
   const float* dtp = a.dt_raw + static_cast<size_t>(sp.row0) * a.ld_u + c0;
   const float* xp = a.xp + static_cast<size_t>(sp.row0) * a.ld_xp + a.dt_rank;
+  const bool wide = ((a.state | a.dt_rank | a.ld_xp) & 3) == 0;
   auto fetch = [&](int t0, Tile& d) {
     const int nt = min(kTT, sp.n - t0);
     tile_rows<float, CW>(&d.dt[0][0], dtp + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
     tile_rows<T, CW>(&d.u[0][0], u + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
     tile_rows<T, CW>(&d.z[0][0], z + static_cast<size_t>(t0) * a.ld_xz, a.ld_xz, nt, lane);
-    for (int n = lane; n < 2 * a.state; n += 32) {       // B then C: neighbours in the row
+    if (wide) {                                          // B then C: neighbours in the row, 16 bytes at a time
+      const int per = a.state >> 1, half = a.state >> 2;
+      for (int i = lane; i < nt * per; i += 32) {
+        const int t = i / per, q = i - t * per;
+        float* dst = q < half ? &d.B[t][4 * q] : &d.C[t][4 * (q - half)];
+        cp_async<16>(dst, xp + static_cast<size_t>(t0 + t) * a.ld_xp + 4 * q);
+      }
+    } else
+    for (int n = lane; n < 2 * a.state; n += 32) {
       float* dst = n < a.state ? &d.B[0][n] : &d.C[0][n - a.state];
       const float* src = xp + static_cast<size_t>(t0) * a.ld_xp + n;
 #pragma unroll 8
@@ -392,7 +396,7 @@ __global__ void __launch_bounds__(32 * kScanWarps) ssm_scan_kernel(const SsmArgs
     }
     __syncwarp();
     constexpr int kU = 4;                                // rows per group of the recurrence
-    static_assert(kTT % kU == 0 && (NS == 2 || NS % 4 == 0), "whole groups");
+    static_assert(kTT % kU == 0 && NS % 4 == 0, "whole groups");
     auto group = [&](int t1, int rows_left) {
       float2 st[kU];
       float Bv[kU][NS], Cv[kU][NS];
@@ -546,9 +550,7 @@ cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
 
 template <typename T>
 cudaError_t scan_states(const SsmArgs& a, cudaStream_t s) {
-  // one prompt: more lanes per channel, so that every scheduler has a few warps to issue from
-  const bool few = static_cast<int64_t>(a.inner) * a.nseq <= 148 * 4 * 32;
-  if (a.state <= 16) return few ? scan<T, 8, 2>(a, s) : scan<T, 4, 4>(a, s);
+  if (a.state <= 16) return scan<T, 4, 4>(a, s);
   if (a.state <= 32) return scan<T, 8, 4>(a, s);
   if (a.state <= 64) return scan<T, 16, 4>(a, s);
   if (a.state <= 128) return scan<T, 32, 4>(a, s);
