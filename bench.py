@@ -679,7 +679,8 @@ def run_stack(args):
         gptj = dict(GPTJ_6B, layers=len(runs), d_model=d, n_heads=d // 256, n_vocab=kes["vocab"], early_cast=True)
         row = {}
         for name, cfg in (("keselix", kes), ("gptj", gptj)):
-            net = CausalTransformer(dict(cfg), device=device)
+            net = CausalTransformer(dict(cfg), device=device, init_weights=False)
+            net.state = net._init_state(seed=42)
             V = cfg.get("n_vocab", kes["vocab"])
             if name == "keselix":
                 weights, flops = stack_work(cfg, runs, T - 1, window)
