@@ -225,22 +225,55 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
     if (a.post_w) {
       // norm after the sublayer, residual add, and the root mean square of the new residual row
       const int n_out = a.n_valid > 0 ? a.n_valid : a.N;
+      // rows of up to kHold * 4 * 256 numbers live in registers: one round of loads for y and x together
+      constexpr int kHold = 4;
+      const int ldo = a.ld_out > 0 ? a.ld_out : a.N;
+      const bool held = ((n_out | ldo | a.post_ldx) & 3) == 0 && n_out <= kHold * 4 * kGemvThreads;
       for (int bt = 0; bt < nb; ++bt) {
-        const float* row = a.out + static_cast<size_t>(m0 + bt) * (a.ld_out > 0 ? a.ld_out : a.N);
+        const float* row = a.out + static_cast<size_t>(m0 + bt) * ldo;
         float* xrow = a.post_x + static_cast<size_t>(m0 + bt) * a.post_ldx;
-        float s = 0.f;
+        float s = 0.f, q = 0.f;
+        if (held) {
+          float4 y4[kHold], x4[kHold];
+#pragma unroll
+          for (int i = 0; i < kHold; ++i) {
+            const int c = 4 * (i * kGemvThreads + static_cast<int>(threadIdx.x));
+            const bool in = c < n_out;
+            y4[i] = in ? __ldcg(reinterpret_cast<const float4*>(row + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (in) prefetch_l2(a.post_w + c);
+            x4[i] = in ? *reinterpret_cast<const float4*>(xrow + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int i = 0; i < kHold; ++i)
+            s += y4[i].x * y4[i].x + y4[i].y * y4[i].y + y4[i].z * y4[i].z + y4[i].w * y4[i].w;
+          const float rs = a.post_mult / sqrtf(block_sum(s, red) / static_cast<float>(n_out) + a.post_eps);
+#pragma unroll
+          for (int i = 0; i < kHold; ++i) {
+            const int c = 4 * (i * kGemvThreads + static_cast<int>(threadIdx.x));
+            float4 v = x4[i];
+            if (c < n_out) {
+              const float4 w = *reinterpret_cast<const float4*>(a.post_w + c);
+              v.x = fmaf(y4[i].x * rs, w.x, v.x);
+              v.y = fmaf(y4[i].y * rs, w.y, v.y);
+              v.z = fmaf(y4[i].z * rs, w.z, v.z);
+              v.w = fmaf(y4[i].w * rs, w.w, v.w);
+              *reinterpret_cast<float4*>(xrow + c) = v;
+            }
+            q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+          }
+        } else {
 #pragma unroll 8
-        for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
-          const float y = __ldcg(row + i);
-          s = fmaf(y, y, s);
-        }
-        const float rs = a.post_mult / sqrtf(block_sum(s, red) / static_cast<float>(n_out) + a.post_eps);
-        float q = 0.f;
+          for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+            const float y = __ldcg(row + i);
+            s = fmaf(y, y, s);
+          }
+          const float rs = a.post_mult / sqrtf(block_sum(s, red) / static_cast<float>(n_out) + a.post_eps);
 #pragma unroll 8
-        for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
-          const float v = fmaf(__ldcg(row + i) * rs, a.post_w[i], xrow[i]);
-          xrow[i] = v;
-          q = fmaf(v, v, q);
+          for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+            const float v = fmaf(__ldcg(row + i) * rs, a.post_w[i], xrow[i]);
+            xrow[i] = v;
+            q = fmaf(v, v, q);
+          }
         }
         const float ms = block_sum(q, red) / static_cast<float>(n_out);
         if (threadIdx.x == 0) {

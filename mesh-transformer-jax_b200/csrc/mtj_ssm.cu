@@ -235,12 +235,11 @@ __global__ void __launch_bounds__(64) ssm_split_kernel(const SsmArgs a) {
   if (i < a.dt_rank) a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(v);
 }
 
-// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states; a warp works on its
-// CW = 32 / G channels alone (no block barriers, so the warps of an SM are in different phases): tiles of 8 to 32 rows of
-// dt, u, z (per channel) and B, C (shared) come into its shared memory by cp.async, one tile ahead; step sizes are
-// finished for the whole tile, the recurrence leaves per-lane partial outputs, and the last phase adds them, applies D
-// and the gate.  The bound is the exponentials: one per row, channel and state.
-constexpr int kScanWarps = 2;
+// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states.  A block is a pair of
+// warps that works on CW = 32 / G channels: warp 0 runs the recurrence over a tile of rows, leaving per-lane partial
+// outputs, while warp 1 finishes the step sizes of the tile ahead, adds up, gates and stores the outputs of the tile
+// behind, and fetches the tile after the next (cp.async: dt, u, z per channel, B and C shared); one block barrier a
+// tile.  The bound is the exponentials: one per row, channel and state.
 
 template <int BYTES>
 __device__ __forceinline__ void cp_async(void* dst, const void* src) {
@@ -294,7 +293,7 @@ struct Decay<__nv_bfloat16> {
 template <typename T, int G, int NS>
 struct ScanTile {
   static constexpr int CW = 32 / G, NSP = G * NS;
-  static constexpr int kTT = NSP <= 64 ? 32 : NSP <= 128 ? 16 : 8;      // rows
+  static constexpr int kTT = NSP <= 64 ? 16 : 8;         // rows
   float B[kTT][NSP], C[kTT][NSP];
   float dt[kTT][CW];
   T u[kTT][CW], z[kTT][CW];
@@ -302,158 +301,174 @@ struct ScanTile {
 template <typename T, int G, int NS>
 struct ScanSmem {
   static constexpr int kTT = ScanTile<T, G, NS>::kTT;
-  ScanTile<T, G, NS> tile[2];
-  float2 step[kTT][32 / G];        // (dt, dt u)
-  float y[kTT][33];                // per lane; the padding spreads the last phase's reads over the banks
+  ScanTile<T, G, NS> tile[4];      // behind, current, ahead, arriving
+  float2 step[2][kTT][32 / G];     // (dt, dt u)
+  float y[2][kTT][33];             // per lane; the padding spreads the last phase's reads over the banks
 };
 
 template <typename T, int G, int NS>
-__global__ void __launch_bounds__(32 * kScanWarps) ssm_scan_kernel(const SsmArgs a) {
+__global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
   using Tile = ScanTile<T, G, NS>;
   constexpr int CW = Tile::CW, NSP = Tile::NSP, kTT = Tile::kTT;
   extern __shared__ __align__(16) unsigned char sc_smem[];
+  auto& sm = *reinterpret_cast<ScanSmem<T, G, NS>*>(sc_smem);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  auto& sm = reinterpret_cast<ScanSmem<T, G, NS>*>(sc_smem)[warp];
   const SeqSpan sp = seq_span(a, blockIdx.y);
-  const int ch = lane / G, g = lane % G;
-  const int c0 = (blockIdx.x * kScanWarps + warp) * CW, c = c0 + ch;
-  if (c0 >= a.inner) return;                             // whole warps only: nothing below synchronises the block
-  const bool c_ok = c < a.inner;
+  const int c0 = blockIdx.x * CW;
+  const int tiles = (sp.n + kTT - 1) / kTT;
+  for (int i = threadIdx.x; i < static_cast<int>(sizeof(sm.tile) / 4); i += 64) reinterpret_cast<float*>(sm.tile)[i] = 0.f;   // padded states stay zero
+  __syncthreads();
+  if (warp == 0) {
+    const int ch = lane / G, g = lane % G, c = c0 + ch;
+    const bool c_ok = c < a.inner;
+    float S[NS], A[NS];
+    float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + (c_ok ? c : 0)) * a.state;
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      const int n = g * NS + i;
+      const bool ok = c_ok && n < a.state;
+      A[i] = ok ? a.A[static_cast<size_t>(c) * a.state + n] * Decay<T>::kScale : 0.f;
+      S[i] = (ok && sp.start > 0 && sp.n > 0) ? state[n] : 0.f;
+    }
+    __syncthreads();                                     // tile 0 and its steps are ready
+    for (int k = 0; k < tiles; ++k) {
+      const Tile& d = sm.tile[k & 3];
+      const int nt = min(kTT, sp.n - k * kTT);
+      // rows in groups: all shared-memory reads of a group come before its writes, which the compiler could not move
+      // them over
+      constexpr int kU = 4;
+      static_assert(kTT % kU == 0 && NS % 4 == 0, "whole groups");
+      auto group = [&](int t1, int rows_left) {
+        float2 st[kU];
+        float Bv[kU][NS], Cv[kU][NS], y[kU];
+#pragma unroll
+        for (int r = 0; r < kU; ++r) {
+          st[r] = sm.step[k & 1][t1 + r][ch];
+          load_states<NS>(&d.B[t1 + r][g * NS], Bv[r]);
+          load_states<NS>(&d.C[t1 + r][g * NS], Cv[r]);
+        }
+#pragma unroll
+        for (int r = 0; r < kU; ++r) {
+          y[r] = 0.f;
+          if (r < rows_left) {
+#pragma unroll
+            for (int i = 0; i < NS; ++i) {
+              S[i] = fmaf(Decay<T>::f(st[r].x * A[i]), S[i], st[r].y * Bv[r][i]);
+              y[r] = fmaf(S[i], Cv[r][i], y[r]);
+            }
+          }
+        }
+#pragma unroll
+        for (int r = 0; r < kU; ++r) sm.y[k & 1][t1 + r][lane] = y[r];
+      };
+      if (nt == kTT) {
+#pragma unroll
+        for (int t = 0; t < kTT; t += kU) group(t, kU);
+      } else {
+        for (int t = 0; t < nt; t += kU) group(t, nt - t);
+      }
+      __syncthreads();
+    }
+    if (c_ok && sp.n > 0) {
+#pragma unroll
+      for (int i = 0; i < NS; ++i)
+        if (g * NS + i < a.state) state[g * NS + i] = S[i];
+    }
+    return;
+  }
+  // warp 1
   const T* u = (a.u ? reinterpret_cast<const T*>(a.u) : reinterpret_cast<const T*>(a.u_bf16)) + static_cast<size_t>(sp.row0) * a.ld_u + c0;
   const T* z = static_cast<const T*>(a.xz) + static_cast<size_t>(sp.row0) * a.ld_xz + a.z0 + c0;
   const float* dtp = a.dt_raw + static_cast<size_t>(sp.row0) * a.ld_u + c0;
   const float* xp = a.xp + static_cast<size_t>(sp.row0) * a.ld_xp + a.dt_rank;
   const bool wide = ((a.state | a.dt_rank | a.ld_xp) & 3) == 0;
-  auto fetch = [&](int t0, Tile& d) {
-    const int nt = min(kTT, sp.n - t0);
-    tile_rows<float, CW>(&d.dt[0][0], dtp + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
-    tile_rows<T, CW>(&d.u[0][0], u + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
-    tile_rows<T, CW>(&d.z[0][0], z + static_cast<size_t>(t0) * a.ld_xz, a.ld_xz, nt, lane);
-    if (wide) {                                          // B then C: neighbours in the row, 16 bytes at a time
-      const int per = a.state >> 1, half = a.state >> 2;
-      for (int i = lane; i < nt * per; i += 32) {
-        const int t = i / per, q = i - t * per;
-        float* dst = q < half ? &d.B[t][4 * q] : &d.C[t][4 * (q - half)];
-        cp_async<16>(dst, xp + static_cast<size_t>(t0 + t) * a.ld_xp + 4 * q);
+  auto fetch = [&](int k) {                              // always commits a group, so that groups count tiles
+    if (k < tiles) {
+      Tile& d = sm.tile[k & 3];
+      const int t0 = k * kTT, nt = min(kTT, sp.n - t0);
+      tile_rows<float, CW>(&d.dt[0][0], dtp + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
+      tile_rows<T, CW>(&d.u[0][0], u + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
+      tile_rows<T, CW>(&d.z[0][0], z + static_cast<size_t>(t0) * a.ld_xz, a.ld_xz, nt, lane);
+      if (wide) {                                        // B then C: neighbours in the row, 16 bytes at a time
+        const int per = a.state >> 1, half = a.state >> 2;
+        for (int i = lane; i < nt * per; i += 32) {
+          const int t = i / per, q = i - t * per;
+          float* dst = q < half ? &d.B[t][4 * q] : &d.C[t][4 * (q - half)];
+          cp_async<16>(dst, xp + static_cast<size_t>(t0 + t) * a.ld_xp + 4 * q);
+        }
+      } else {
+        for (int n = lane; n < 2 * a.state; n += 32) {
+          float* dst = n < a.state ? &d.B[0][n] : &d.C[0][n - a.state];
+          const float* src = xp + static_cast<size_t>(t0) * a.ld_xp + n;
+#pragma unroll 4
+          for (int t = 0; t < nt; ++t) cp_async<4>(dst + t * NSP, src + static_cast<size_t>(t) * a.ld_xp);
+        }
       }
-    } else
-    for (int n = lane; n < 2 * a.state; n += 32) {
-      float* dst = n < a.state ? &d.B[0][n] : &d.C[0][n - a.state];
-      const float* src = xp + static_cast<size_t>(t0) * a.ld_xp + n;
-#pragma unroll 8
-      for (int t = 0; t < nt; ++t) cp_async<4>(dst + t * NSP, src + static_cast<size_t>(t) * a.ld_xp);
     }
     cp_commit();
   };
-  for (int i = lane; i < static_cast<int>(2 * sizeof(Tile) / 4); i += 32) reinterpret_cast<float*>(sm.tile)[i] = 0.f;   // padded states stay zero
-  __syncwarp();
-  if (sp.n > 0) fetch(0, sm.tile[0]);
-  float S[NS], A[NS];
-  float* state = a.ssm_state + (static_cast<size_t>(sp.seq) * a.inner + (c_ok ? c : 0)) * a.state;
-#pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    const int n = g * NS + i;
-    const bool ok = c_ok && n < a.state;
-    A[i] = ok ? a.A[static_cast<size_t>(c) * a.state + n] * Decay<T>::kScale : 0.f;
-    S[i] = (ok && sp.start > 0 && sp.n > 0) ? state[n] : 0.f;
-  }
-  // phases over (row, channel) pairs: lane -> channel fc, rows t = ft, ft + G, ...
+  // lane -> channel fc, rows t = ft, ft + G, ...
   const int fc = lane % CW, ft = lane / CW;
   const bool f_ok = c0 + fc < a.inner;
   const float dt_b = f_ok ? a.dt_b[c0 + fc] : 0.f, D = f_ok ? a.D[c0 + fc] : 0.f;
+  constexpr int kR = kTT / G > 0 ? kTT / G : 1;          // rows per lane
+  auto steps = [&](int k) {
+    const Tile& d = sm.tile[k & 3];
+    float raw[kR], uu[kR];
+#pragma unroll
+    for (int i = 0; i < kR; ++i) {
+      const int t = min(ft + i * G, kTT - 1);
+      raw[i] = d.dt[t][fc];
+      uu[i] = ld(&d.u[t][fc], 0);
+    }
+#pragma unroll
+    for (int i = 0; i < kR; ++i) {
+      const float dt = f_ok ? Fn<T>::softplus(raw[i] + dt_b) : 0.f;
+      if (ft + i * G < kTT) sm.step[k & 1][ft + i * G][fc] = make_float2(dt, dt * uu[i]);
+    }
+  };
+  const size_t o0 = static_cast<size_t>(sp.row0 + ft) * a.ld_u + c0 + fc, o_step = static_cast<size_t>(G) * a.ld_u;
+  auto finish = [&](int k) {
+    const Tile& d = sm.tile[k & 3];
+    const int nt = min(kTT, sp.n - k * kTT);
+    float yv[kR];
+#pragma unroll
+    for (int i = 0; i < kR; ++i) {
+      const int t = min(ft + i * G, kTT - 1);
+      float y = 0.f;
+#pragma unroll
+      for (int j = 0; j < G; ++j) y += sm.y[k & 1][t][fc * G + j];
+      yv[i] = fmaf(D, ld(&d.u[t][fc], 0), y) * Fn<T>::silu(ld(&d.z[t][fc], 0));
+    }
+    const size_t o = o0 + static_cast<size_t>(k) * kTT * a.ld_u;
+#pragma unroll
+    for (int i = 0; i < kR; ++i) {
+      if (!f_ok || ft + i * G >= nt) continue;
+      if (a.out) a.out[o + i * o_step] = yv[i];
+      if (a.out_bf16) a.out_bf16[o + i * o_step] = __float2bfloat16_rn(yv[i]);
+    }
+  };
+  fetch(0);
+  fetch(1);
   // rows in front of the sequence's start give zeros
   for (int t = ft; t < a.rows.Tc - sp.n; t += G) {
     const size_t o = (static_cast<size_t>(blockIdx.y) * a.rows.Tc + t) * a.ld_u + c0 + fc;
     if (f_ok && a.out) a.out[o] = 0.f;
     if (f_ok && a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(0.f);
   }
-  for (int t0 = 0, k = 0; t0 < sp.n; t0 += kTT, ++k) {
-    Tile& d = sm.tile[k & 1];
-    const int nt = min(kTT, sp.n - t0);
-    if (t0 + kTT < sp.n) {
-      fetch(t0 + kTT, sm.tile[(k + 1) & 1]);
-      cp_wait<1>();
-    } else {
-      cp_wait<0>();
-    }
+  cp_wait<1>();
+  __syncwarp();                                          // every lane's copies of tile 0 are visible to the warp
+  if (tiles > 0) steps(0);
+  __syncthreads();
+  for (int k = 0; k < tiles; ++k) {
+    if (k > 0) finish(k - 1);                            // its tile is overwritten only by fetch(k + 3)
+    fetch(k + 2);
+    cp_wait<1>();
     __syncwarp();
-    // Each phase reads a group of rows into registers before it writes: the compiler cannot move shared-memory loads
-    // over stores whose addresses it does not know.
-    constexpr int kR = kTT / G > 0 ? kTT / G : 1;        // rows per lane of the elementwise phases
-    {
-      float raw[kR], uu[kR];
-#pragma unroll
-      for (int i = 0; i < kR; ++i) {
-        const int t = min(ft + i * G, kTT - 1);
-        raw[i] = d.dt[t][fc];
-        uu[i] = ld(&d.u[t][fc], 0);
-      }
-#pragma unroll
-      for (int i = 0; i < kR; ++i) {
-        const float dt = f_ok ? Fn<T>::softplus(raw[i] + dt_b) : 0.f;
-        if (ft + i * G < kTT) sm.step[ft + i * G][fc] = make_float2(dt, dt * uu[i]);
-      }
-    }
-    __syncwarp();
-    constexpr int kU = 4;                                // rows per group of the recurrence
-    static_assert(kTT % kU == 0 && NS % 4 == 0, "whole groups");
-    auto group = [&](int t1, int rows_left) {
-      float2 st[kU];
-      float Bv[kU][NS], Cv[kU][NS];
-#pragma unroll
-      for (int r = 0; r < kU; ++r) {
-        st[r] = sm.step[t1 + r][ch];
-        load_states<NS>(&d.B[t1 + r][g * NS], Bv[r]);
-        load_states<NS>(&d.C[t1 + r][g * NS], Cv[r]);
-      }
-      float y[kU];
-#pragma unroll
-      for (int r = 0; r < kU; ++r) {
-        y[r] = 0.f;
-        if (r < rows_left) {
-#pragma unroll
-          for (int i = 0; i < NS; ++i) {
-            S[i] = fmaf(Decay<T>::f(st[r].x * A[i]), S[i], st[r].y * Bv[r][i]);
-            y[r] = fmaf(S[i], Cv[r][i], y[r]);
-          }
-        }
-      }
-#pragma unroll
-      for (int r = 0; r < kU; ++r) sm.y[t1 + r][lane] = y[r];
-    };
-    if (nt == kTT) {
-#pragma unroll 2
-      for (int t = 0; t < kTT; t += kU) group(t, kU);
-    } else {
-      for (int t = 0; t < nt; t += kU) group(t, nt - t);
-    }
-    __syncwarp();
-    {
-      float yv[kR];
-#pragma unroll
-      for (int i = 0; i < kR; ++i) {
-        const int t = min(ft + i * G, kTT - 1);
-        float y = 0.f;
-#pragma unroll
-        for (int j = 0; j < G; ++j) y += sm.y[t][fc * G + j];
-        yv[i] = fmaf(D, ld(&d.u[t][fc], 0), y) * Fn<T>::silu(ld(&d.z[t][fc], 0));
-      }
-#pragma unroll
-      for (int i = 0; i < kR; ++i) {
-        const int t = ft + i * G;
-        if (!f_ok || t >= nt) continue;
-        const size_t o = static_cast<size_t>(sp.row0 + t0 + t) * a.ld_u + c0 + fc;
-        if (a.out) a.out[o] = yv[i];
-        if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(yv[i]);
-      }
-    }
-    __syncwarp();                                        // the tile may be fetched over, y written again
+    if (k + 1 < tiles) steps(k + 1);
+    __syncthreads();
   }
-  if (c_ok && sp.n > 0) {
-#pragma unroll
-    for (int i = 0; i < NS; ++i)
-      if (g * NS + i < a.state) state[g * NS + i] = S[i];
-  }
+  if (tiles > 0) finish(tiles - 1);
 }
 
 // Decode, one row per sequence: G lanes per channel do the step size (its projection too, unless dt_raw holds it),
@@ -537,14 +552,14 @@ bool ssm_ok(const SsmArgs& a) {
 
 template <typename T, int G, int NS>
 cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
-  constexpr int smem = static_cast<int>(kScanWarps * sizeof(ScanSmem<T, G, NS>)), CH = kScanWarps * 32 / G;
+  constexpr int smem = static_cast<int>(sizeof(ScanSmem<T, G, NS>)), CW = 32 / G;
   static_assert(smem <= 220 * 1024, "shared memory");
   static DeviceOnce once;
   cudaError_t e = once.run([&] {
     return cudaFuncSetAttribute(ssm_scan_kernel<T, G, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   });
   if (e != cudaSuccess) return e;
-  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CH - 1) / CH, a.nseq), 32 * kScanWarps, smem, s>>>(a);
+  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CW - 1) / CW, a.nseq), 64, smem, s>>>(a);
   return cudaGetLastError();
 }
 
