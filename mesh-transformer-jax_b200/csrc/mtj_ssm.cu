@@ -235,11 +235,10 @@ __global__ void __launch_bounds__(64) ssm_split_kernel(const SsmArgs a) {
   if (i < a.dt_rank) a.dtr_bf16[m * a.ld_dtr + i] = __float2bfloat16_rn(v);
 }
 
-// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states.  A block is a pair of
-// warps that works on CW = 32 / G channels: warp 0 runs the recurrence over a tile of rows, leaving per-lane partial
-// outputs, while warp 1 finishes the step sizes of the tile ahead, adds up, gates and stores the outputs of the tile
-// behind, and fetches the tile after the next (cp.async: dt, u, z per channel, B and C shared); one block barrier a
-// tile.  The bound is the exponentials: one per row, channel and state.
+// The recurrence over a sequence's rows.  G lanes share a channel, each holding NS of its states.  A block is three
+// warps that work on CW = 32 / G channels: warp 0 runs the recurrence over a tile of rows, leaving per-lane partial
+// outputs, while warp 1 fetches the tile after the next (cp.async: dt, u, z per channel, B and C shared) and finishes the
+// step sizes of the next, and warp 2 adds up, gates and stores the outputs of the one behind; one block barrier a tile.  The bound is the exponentials: one per row, channel and state.
 
 template <int BYTES>
 __device__ __forceinline__ void cp_async(void* dst, const void* src) {
@@ -307,7 +306,7 @@ struct ScanSmem {
 };
 
 template <typename T, int G, int NS>
-__global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
+__global__ void __launch_bounds__(96) ssm_scan_kernel(const SsmArgs a) {
   using Tile = ScanTile<T, G, NS>;
   constexpr int CW = Tile::CW, NSP = Tile::NSP, kTT = Tile::kTT;
   extern __shared__ __align__(16) unsigned char sc_smem[];
@@ -316,7 +315,7 @@ __global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
   const SeqSpan sp = seq_span(a, blockIdx.y);
   const int c0 = blockIdx.x * CW;
   const int tiles = (sp.n + kTT - 1) / kTT;
-  for (int i = threadIdx.x; i < static_cast<int>(sizeof(sm.tile) / 4); i += 64) reinterpret_cast<float*>(sm.tile)[i] = 0.f;   // padded states stay zero
+  for (int i = threadIdx.x; i < static_cast<int>(sizeof(sm.tile) / 4); i += 96) reinterpret_cast<float*>(sm.tile)[i] = 0.f;   // padded states stay zero
   __syncthreads();
   if (warp == 0) {
     const int ch = lane / G, g = lane % G, c = c0 + ch;
@@ -376,12 +375,15 @@ __global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
     }
     return;
   }
-  // warp 1
+  // warps 1 and 2
   const T* u = (a.u ? reinterpret_cast<const T*>(a.u) : reinterpret_cast<const T*>(a.u_bf16)) + static_cast<size_t>(sp.row0) * a.ld_u + c0;
   const T* z = static_cast<const T*>(a.xz) + static_cast<size_t>(sp.row0) * a.ld_xz + a.z0 + c0;
   const float* dtp = a.dt_raw + static_cast<size_t>(sp.row0) * a.ld_u + c0;
   const float* xp = a.xp + static_cast<size_t>(sp.row0) * a.ld_xp + a.dt_rank;
   const bool wide = ((a.state | a.dt_rank | a.ld_xp) & 3) == 0;
+  // 16-byte pieces of a row's B and C, rows that a warp copies at once, this lane's place among them
+  const int per = max(a.state >> 1, 1), half = a.state >> 2, rows_at_once = max(32 / per, 1);
+  const int wt = per >= 32 ? 0 : lane < rows_at_once * per ? lane / per : kTT, wq = per >= 32 ? lane : lane % per;
   auto fetch = [&](int k) {                              // always commits a group, so that groups count tiles
     if (k < tiles) {
       Tile& d = sm.tile[k & 3];
@@ -390,11 +392,11 @@ __global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
       tile_rows<T, CW>(&d.u[0][0], u + static_cast<size_t>(t0) * a.ld_u, a.ld_u, nt, lane);
       tile_rows<T, CW>(&d.z[0][0], z + static_cast<size_t>(t0) * a.ld_xz, a.ld_xz, nt, lane);
       if (wide) {                                        // B then C: neighbours in the row, 16 bytes at a time
-        const int per = a.state >> 1, half = a.state >> 2;
-        for (int i = lane; i < nt * per; i += 32) {
-          const int t = i / per, q = i - t * per;
-          float* dst = q < half ? &d.B[t][4 * q] : &d.C[t][4 * (q - half)];
-          cp_async<16>(dst, xp + static_cast<size_t>(t0 + t) * a.ld_xp + 4 * q);
+        for (int t = wt; t < nt; t += rows_at_once) {
+          for (int q = wq; q < per; q += 32) {
+            float* dst = q < half ? &d.B[t][4 * q] : &d.C[t][4 * (q - half)];
+            cp_async<16>(dst, xp + static_cast<size_t>(t0 + t) * a.ld_xp + 4 * q);
+          }
         }
       } else {
         for (int n = lane; n < 2 * a.state; n += 32) {
@@ -448,24 +450,31 @@ __global__ void __launch_bounds__(64) ssm_scan_kernel(const SsmArgs a) {
       if (a.out_bf16) a.out_bf16[o + i * o_step] = __float2bfloat16_rn(yv[i]);
     }
   };
-  fetch(0);
-  fetch(1);
+  if (warp == 1) {
+    fetch(0);
+    fetch(1);
+    cp_wait<1>();
+    __syncwarp();                                        // every lane's copies of tile 0 are visible to the warp
+    if (tiles > 0) steps(0);
+    __syncthreads();
+    for (int k = 0; k < tiles; ++k) {
+      fetch(k + 2);                                      // over tile k - 2, which nobody reads any more
+      cp_wait<1>();
+      __syncwarp();
+      if (k + 1 < tiles) steps(k + 1);
+      __syncthreads();
+    }
+    return;
+  }
   // rows in front of the sequence's start give zeros
   for (int t = ft; t < a.rows.Tc - sp.n; t += G) {
     const size_t o = (static_cast<size_t>(blockIdx.y) * a.rows.Tc + t) * a.ld_u + c0 + fc;
     if (f_ok && a.out) a.out[o] = 0.f;
     if (f_ok && a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(0.f);
   }
-  cp_wait<1>();
-  __syncwarp();                                          // every lane's copies of tile 0 are visible to the warp
-  if (tiles > 0) steps(0);
   __syncthreads();
   for (int k = 0; k < tiles; ++k) {
-    if (k > 0) finish(k - 1);                            // its tile is overwritten only by fetch(k + 3)
-    fetch(k + 2);
-    cp_wait<1>();
-    __syncwarp();
-    if (k + 1 < tiles) steps(k + 1);
+    if (k > 0) finish(k - 1);
     __syncthreads();
   }
   if (tiles > 0) finish(tiles - 1);
@@ -559,7 +568,7 @@ cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
     return cudaFuncSetAttribute(ssm_scan_kernel<T, G, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   });
   if (e != cudaSuccess) return e;
-  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CW - 1) / CW, a.nseq), 64, smem, s>>>(a);
+  ssm_scan_kernel<T, G, NS><<<dim3((a.inner + CW - 1) / CW, a.nseq), 96, smem, s>>>(a);
   return cudaGetLastError();
 }
 
