@@ -281,7 +281,7 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
 
 // The same for several rows at a time with bf16 caches, on the tensor cores: one block = (row, 16 MT heads, key range).
 // The heads are the M dimension of mma.m16n8k16: S[heads, 32 keys] = Q' . C^T, fp32 online softmax, O[heads, latent] +=
-// P . C from the same tile, so a cached byte is read once per 32 heads.  A warp owns NT 8-column blocks of O.  Tiles
+// P . C from the same tile, so a cached byte is read once per 16 MT heads.  A warp owns NT 8-column blocks of O.  Tiles
 // come by cp.async, one ahead.  (M is the number of heads, far below the 128 rows of a tcgen05 tile, and the bound is
 // the cache traffic.)
 __device__ __forceinline__ void ldsm4(uint32_t* r, uint32_t addr) {
@@ -663,19 +663,18 @@ cudaError_t attend_mma(const LatentArgs& a, cudaStream_t s, bool pdl) {
                     mma_smem_bytes<MT>(a.cache.row_ld), s, pdl, a);
 }
 
-// head tiles of the tensor-core form (0: this call takes the CUDA-core form)
-int mma_head_tiles(int M, int heads, int row_ld, int kv_ld, int tensor_cores) {
-  if (!tensor_cores || M < kMmaRows || mma_smem_bytes<1>(row_ld) > 220 * 1024) return 0;
-  return 1;
+// 16 heads per block (two blocks per SM at a 576-column cache row); 32 were slower, one block per SM
+bool use_mma(int M, int row_ld, int tensor_cores) {
+  return tensor_cores && M >= kMmaRows && mma_smem_bytes<1>(row_ld) <= 220 * 1024;
 }
 
 }  // namespace
 
-int latent_attn_splits(int M, int heads, int row_ld, int kv_ld, int tensor_cores, int window) {
-  const int mt = mma_head_tiles(M, heads, row_ld, kv_ld, tensor_cores);
-  const int groups = M * (mt ? (heads + 16 * mt - 1) / (16 * mt) : (heads + kHG - 1) / kHG);
+int latent_attn_splits(int M, int heads, int row_ld, int tensor_cores, int window) {
+  const bool mma = use_mma(M, row_ld, tensor_cores);
+  const int groups = M * (mma ? (heads + 15) / 16 : (heads + kHG - 1) / kHG);
   // one wave of blocks: two per SM for the tensor-core form, four for the other
-  return std::max(1, std::min({kMaxSplits, (window + kTK - 1) / kTK, (mt ? 296 : kLatentBlocks) / groups}));
+  return std::max(1, std::min({kMaxSplits, (window + kTK - 1) / kTK, (mma ? 296 : kLatentBlocks) / groups}));
 }
 
 cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl) {
@@ -686,8 +685,7 @@ cudaError_t launch_latent_absorb(const LatentArgs& a, cudaStream_t s, bool pdl) 
 
 cudaError_t launch_latent_attn(const LatentArgs& a, cudaStream_t s, bool pdl) {
   if (!latent_ok(a) || a.splits < 1 || a.splits > kMaxSplits) return cudaErrorInvalidValue;
-  const int mt = mma_head_tiles(a.M, a.heads, a.cache.row_ld, a.cache.kv_ld, a.tensor_cores && !a.cache.f32);
-  if (mt) {
+  if (use_mma(a.M, a.cache.row_ld, a.tensor_cores && !a.cache.f32)) {
     const int nt = (a.cache.kv_ld + 63) / 64;             // 8-column blocks per warp
     return nt <= 2 ? attend_mma<1, 2>(a, s, pdl) : nt <= 4 ? attend_mma<1, 4>(a, s, pdl) : nt <= 8 ? attend_mma<1, 8>(a, s, pdl) : attend_mma<1, 16>(a, s, pdl);
   }

@@ -621,7 +621,7 @@ int32_t LayerStack::latent(mtj_handle* h, const Run& r, int M, const RowMap& row
         b.rows = rows.Tc == 1 ? RowMap{rows.b0 + t0, 1, rows.pos0_host, rows.pos0_dev}
                               : RowMap{rows.b0 + m0 / per, b.M, rows.pos0_host + t0, rows.pos0_dev};
         b.p1 = p1_ + static_cast<size_t>(m0 + t0) * a.ld_p1;
-        b.splits = latent_attn_splits(b.M, m.heads, l.row_ld, l.kv_ld, tc ? 1 : 0, std::min(m.window, max_pos_));
+        b.splits = latent_attn_splits(b.M, m.heads, l.row_ld, tc ? 1 : 0, std::min(m.window, max_pos_));
         if (tc) b.out_bf16 = act_bf_ + static_cast<size_t>(m0 + t0) * a.ld_out;
         else b.out = act_ + static_cast<size_t>(m0 + t0) * a.ld_out;
         MTJ_CUDA(launch_latent_absorb(b, s, pdl));

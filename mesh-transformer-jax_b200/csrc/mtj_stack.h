@@ -36,7 +36,7 @@ class LayerStack {
   int runs() const { return static_cast<int>(runs_.size()); }
   // residual stream after the last forward, [rows][row stride]
   const float* residual(int* ld) const { *ld = ld_; return x_; }
-  // profiling aid: layer runs to execute (0 = all)
+  // layer runs to execute (0 = all), for mtj_k_stack_residual
   int stop_after = 0;
 
  private:
@@ -81,7 +81,7 @@ class LayerStack {
   bool use_tc(const mtj_handle* h, int M, bool decode) const;
   const TensorMap* xmap(const __nv_bfloat16* buf, int K, int ld, int M);
   int32_t gemm(mtj_handle* h, GemvEpilogue epi, const Linear& l, const __nv_bfloat16* x, int M, float* out, int ld_out,
-               __nv_bfloat16* out_bf16, int ld_bf16, bool decode, cudaStream_t s, int x_row0 = 0, int rows_x = 0);
+               __nv_bfloat16* out_bf16, int ld_bf16, bool decode, cudaStream_t s, int x_row0 = 0, int x_ld = 0);
   int32_t gemm_planes(mtj_handle* h, const Linear& l, const __nv_bfloat16* x, int M, int* planes, bool decode, cudaStream_t s);
   int32_t gemv(mtj_handle* h, GemvEpilogue epi, const Linear& l, const float* x, int ldx, int M, const float* norm, float* out,
                int ld_out, const float* post_w, bool pdl, cudaStream_t s, const int32_t* select = nullptr,

@@ -51,7 +51,7 @@ cudaError_t launch_pack_rows(const void* src, int src_is_bf16, int N, int K, __n
 cudaError_t launch_neg_exp(const void* src, int src_is_bf16, int64_t n, float* dst, cudaStream_t s);
 // src [N, K] -> fp32 dst [K, ld]
 cudaError_t launch_transpose_f32(const void* src, int src_is_bf16, int N, int K, float* dst, int ld, cudaStream_t s);
-// y[m] (+)= x[m] elementwise copies of fp32 rows
+// dst = src, n fp32 elements (a multiple of four)
 cudaError_t launch_copy_rows(const float* src, float* dst, int64_t n, cudaStream_t s, bool pdl);
 
 // ---- mtj_latent_attn.cu: attention over a cached latent (and one rotated key part) shared by all heads
@@ -100,7 +100,7 @@ cudaError_t launch_latent_pack(const LatentArgs& a, cudaStream_t s);
 cudaError_t launch_latent_history(const LatentArgs& a, cudaStream_t s);
 constexpr int kLatentMaxRank = 1024;
 constexpr int kLatentBlocks = 592;       // most (rows x splits x head groups) a call spreads over beyond one per row
-int latent_attn_splits(int M, int heads, int row_ld, int kv_ld, int tensor_cores, int window);
+int latent_attn_splits(int M, int heads, int row_ld, int tensor_cores, int window);
 
 // ---- mtj_ssm.cu: causal convolution and selective scan with carried state
 struct SsmArgs {

@@ -18,7 +18,7 @@ PREFIX = "causal_transformer_shard/~/"
 
 def validate_config(config: dict) -> None:
     """Raises unless the configuration is one its model family can run."""
-    registry.family(config).validate(config)
+    registry.family(config).validate(registry.prepare(config))
 
 
 def param_shapes(config: dict) -> dict:

@@ -92,6 +92,17 @@ def test_window_edges_and_page_borders(cuda_device, path):
 
 
 @pytest.mark.parametrize("path", sorted(su.PATHS))
+def test_one_call_longer_than_a_chunk(cases, path):
+    """The library cuts a long call itself, at max_rows; wanted places in any order across the cuts."""
+    cfg, w, toks, want, _ = cases["odd"]
+    rt = su.runtime(cfg, w, path, max_rows=33)
+    rt.start_batch(1)
+    order = [199, 0, 32, 33, 66, 65, 100, 1, 198]
+    assert su.error(su.extend(rt, 0, toks, order), want[order]) <= su.TOL[path]
+    rt.close()
+
+
+@pytest.mark.parametrize("path", sorted(su.PATHS))
 def test_first_tokens(cases, path):
     """Sequences of 1, 2, 3 ... tokens, each fresh in a slot that has held another."""
     cfg, w, toks, want, _ = cases["odd"]
