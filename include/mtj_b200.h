@@ -77,10 +77,12 @@ typedef struct mtj_config {
 } mtj_config;
 
 /* Layer-stack models (no counterpart in the reference): a list of layers, each a
- * mixer between two RMS norms and, when ff > 0, a SwiGLU feed-forward between two
- * more, x <- x + residual_mult * norm_after(sublayer(norm_before(x))).  Layers
- * loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop), every
- * pass with caches and states of its own, and every pass begins with
+ * mixer and, when ff > 0, a feed-forward.  How a sublayer meets the residual stream
+ * (mtj_stack_desc.residual):
+ *   MTJ_RESIDUAL_SANDWICH_RMS: x <- x + residual_mult * norm_after(sublayer(norm_before(x))), RMS norms;
+ *   MTJ_RESIDUAL_POST_LN:      x <- norm(residual_mult * x + sublayer(x)), layer norms with weight and bias.
+ * Layers loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop),
+ * every pass with caches and states of its own, and every pass begins with
  * x <- W_in [x; embedding output].
  *   MTJ_MIXER_LATENT_ATTENTION: keys and values are linear maps of one
  *     normalised latent of kv_rank numbers per token, plus rot_dim rotated key
@@ -88,31 +90,51 @@ typedef struct mtj_config {
  *     frequencies rot_base^(-2i/rot_dim)); position i sees j with
  *     0 <= i - j < window; scores are multiplied by scale.
  *   MTJ_MIXER_MAMBA1: gated causal convolution (conv taps) and selective scan
- *     (inner channels x state), step sizes through dt_rank numbers. */
-enum { MTJ_MIXER_LATENT_ATTENTION = 0, MTJ_MIXER_MAMBA1 = 1 };
+ *     (inner channels x state), step sizes through dt_rank numbers.
+ *   MTJ_MIXER_GROUPED_ATTENTION: heads query heads over kv_heads key / value heads
+ *     (dim and vdim numbers each), RMS norms over the whole query and key
+ *     projections, causal, queries at position p multiplied by
+ *     1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1) (q_temp_every 0: by one),
+ *     scores by scale.  kv_from >= 0: the layer has no keys and values of its own and reads those of layer kv_from.
+ *   MTJ_MIXER_MATRIX_STATE_SSD: a state of state x vdim numbers per head with one
+ *     decay per head; keys and queries shared by heads / kv_heads heads; the
+ *     causal convolution (conv taps) covers values, keys and queries; gate before an
+ *     RMS norm in norm_groups parts.
+ *   MTJ_MIXER_MATRIX_STATE_DELTA: a state of dim x vdim numbers per head, one decay
+ *     per head and key channel through decay_rank numbers, delta-rule update with
+ *     unit keys, RMS norm per head and an output gate through gate_rank numbers. */
+enum { MTJ_MIXER_LATENT_ATTENTION = 0, MTJ_MIXER_MAMBA1 = 1, MTJ_MIXER_GROUPED_ATTENTION = 2, MTJ_MIXER_MATRIX_STATE_SSD = 3,
+       MTJ_MIXER_MATRIX_STATE_DELTA = 4 };
+enum { MTJ_RESIDUAL_SANDWICH_RMS = 0, MTJ_RESIDUAL_POST_LN = 1 };
+enum { MTJ_FF_SWIGLU = 0, MTJ_FF_SQUARED_RELU = 1 };   /* down(silu(gate) * up) | down(relu(up)^2) */
 typedef struct mtj_layer_desc {
   int32_t mixer;
   int32_t ff;                  /* feed-forward width, 0: no feed-forward         */
   int32_t heads, dim, rot_dim, vdim, kv_rank, window;
   int32_t inner, state, conv, dt_rank;
+  int32_t ff_kind, kv_heads, kv_from, norm_groups, decay_rank, gate_rank;
   float scale;
-  int32_t reserved;
+  float q_temp_coef;
+  double q_temp_every;
   double rot_base;
 } mtj_layer_desc;
 typedef struct mtj_stack_desc {
   const mtj_layer_desc* layers;
   int32_t n_layers;
   int32_t loop_start, loop_stop, loop_times;
+  int32_t residual;            /* MTJ_RESIDUAL_*                                 */
   float residual_mult, norm_eps;
+  float embed_scale;           /* 0: 1                                           */
+  float logit_softcap;         /* logits <- cap * tanh(logits / cap); 0: none    */
   int32_t act_f32;             /* 1: fp32 activations and caches throughout      */
   int32_t tc_min_rows;         /* prompt rows from which a call takes the tensor-core
                                   path; default 16                               */
 } mtj_stack_desc;
 
 const char* mtj_last_error(void);
-/* ABI revision: 4 (2: mtj_config with the tuning fields, mtj_generate, mtj_start_batch / mtj_admit;
+/* ABI revision: 5 (2: mtj_config with the tuning fields, mtj_generate, mtj_start_batch / mtj_admit;
  * 3: top_k in mtj_sample_top_p / mtj_nucleus_filter, mtj_set_top_k; 4: layer-stack models, mtj_extend,
- * mtj_release). */
+ * mtj_release; 5: more mixers and residual forms in mtj_stack_desc). */
 int32_t mtj_version(void);
 
 /* CausalTransformerShard.__init__ (transformer_shard.py:21-45): validates the

@@ -6,7 +6,9 @@
 //   paged  (4, 4): GPT-J, d_head = 256, keys and values in the KV cache's pages;
 //   linear       : keys and values of a chunk and its window's history as plain
 //                  row-major matrices, a key row = per-head columns followed by
-//                  columns all heads share, with a sliding window (mtj_attn_tc_latent.cu).
+//                  columns all heads share, with a sliding window (mtj_attn_tc_latent.cu);
+//   paged rows   : keys and values in pages of row-major rows (all key heads side by side) addressed by the
+//                  position inside the sequence, query heads in groups over them (mtj_attn_tc_grouped.cu).
 // The comments below give the sizes of the paged form.  Reference semantics:
 // layers.py:275-283 (logits / sqrt(d_head), additive masks, softmax, weighted
 // V) with the causal mask of :305-308, the left-pad mask of :353-360 and the
@@ -55,6 +57,7 @@ constexpr int kSoftWarps = 4 * kParts;          // softmax warps: TMEM lane quad
 constexpr int kThreadsTc = 96 + 32 * kSoftWarps;   // TMA warp, two MMA warps (S; P.V), softmax warps
 constexpr int kPartKeys = kKB / kParts;
 constexpr int kKSlots = 3, kVSlots = 2;              // ring depths: a K slot is wanted again one key block sooner than a V slot
+enum KeySource { kPagedHeads = 0, kLinearRows = 1, kPagedRows = 2 };
 template <int QA, int VA>
 struct AttnTcCfg {
   static constexpr uint32_t kQBytes = kQT * QA * 128;        // 64 KB
@@ -161,13 +164,14 @@ __device__ __forceinline__ void tm_st16(uint32_t taddr, const uint32_t* r) {
       : "memory");
 }
 
-template <int QA, int VA, bool LINEAR>
+template <int QA, int VA, int SRC>
 __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                      const __grid_constant__ CUtensorMap map_k,
                                                                      const __grid_constant__ CUtensorMap map_ks,
                                                                      const __grid_constant__ CUtensorMap map_v,
                                                                      const PrefillAttnTcArgs a) {
   using Cfg = AttnTcCfg<QA, VA>;
+  constexpr bool LINEAR = SRC == kLinearRows, ROWS = SRC == kPagedRows;
   constexpr uint32_t kQBytes = Cfg::kQBytes, kKBytes = Cfg::kKBytes, kVBytes = Cfg::kVBytes, kColS = Cfg::kColS,
                      kColO = Cfg::kColO, kColP = Cfg::kColP, kPCols = Cfg::kPCols, kTmemCols = Cfg::kTmemCols;
   constexpr int kDV = Cfg::kDV, kPartCols = Cfg::kPartCols;
@@ -213,16 +217,16 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
   // within a tile, so the tail of the grid is made of the short tiles
   const int tile = gridDim.y - 1 - blockIdx.y, head = blockIdx.x, bi = blockIdx.z;
   const int b = a.rows.b0 + bi;
-  const int pos0 = a.rows.pos0_host;
+  const int pad = ROWS ? 0 : a.kv.pad[b];
+  const int pos0 = ROWS ? a.rows.pos0_host - a.kv.pad[b] : a.rows.pos0_host;   // paged rows: positions inside the sequence
   const int Tc = a.rows.Tc;
   const int row0 = bi * Tc + tile * kQT;                  // first chunk row of this tile
   const int q_rows = min(kQT, Tc - tile * kQT);
-  const int pad = a.kv.pad[b];
   const int limit = a.key_limit ? a.key_limit[b] : 0x7fffffff;
   const int last_key = min(pos0 + tile * kQT + q_rows - 1, limit);
   // positions of the key blocks: blk0 + 64 i (paged: whole cache pages); `lo` = first key any row of the tile sees
   const int blk0 = LINEAR ? pos0 - a.hist : 0;
-  const int lo = LINEAR ? max(pad, pos0 + tile * kQT - a.window + 1) : pad;
+  const int lo = LINEAR || ROWS ? max(pad, pos0 + tile * kQT - a.window + 1) : pad;
   const int first_blk = (lo - blk0) / kKB;
   const int nb = last_key >= lo ? (last_key - blk0) / kKB - first_blk + 1 : 0;
 
@@ -234,8 +238,13 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
       const int32_t* table = LINEAR ? nullptr : a.kv.page_table + static_cast<size_t>(b) * a.kv.ring_pages;
       auto slab_row = [&](int j) {
         return LINEAR ? bi * a.key_rows + (first_blk + j) * kKB
-                      : (table[(first_blk + j) % a.kv.ring_pages] * a.heads + head) * kKB;
+                      : ROWS ? table[(first_blk + j) % a.kv.ring_pages] * kKB
+                             : (table[(first_blk + j) % a.kv.ring_pages] * a.heads + head) * kKB;
       };
+      // first column of this head: the next head's columns in a block's tail meet zero query columns, or end in output
+      // columns that are not stored
+      const int kx = LINEAR ? head * a.k_own * 64 : ROWS ? head / a.kv_group * a.k_cols : 0;
+      const int vx = LINEAR ? head * kDV : ROWS ? head / a.kv_group * a.v_ld : 0;
       auto load_k = [&](int j) {
         const int st = j % kKSlots;
         if (j >= kKSlots && !mbar_wait(k_empty0 + 8 * st, ((j / kKSlots) - 1) & 1)) return false;
@@ -247,7 +256,7 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
           if (LINEAR && kb >= a.k_own)
             tma2d(dk + kb * (kKB * 128), &map_ks, (kb - a.k_own) * 64, row, k_full0 + 8 * st);     // columns all heads share
           else
-            tma2d(dk + kb * (kKB * 128), &map_k, (LINEAR ? head * a.k_own * 64 : 0) + kb * 64, row, k_full0 + 8 * st);
+            tma2d(dk + kb * (kKB * 128), &map_k, kx + kb * 64, row, k_full0 + 8 * st);
         }
         return true;
       };
@@ -259,7 +268,7 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
         mbar_expect_tx(v_full0 + 8 * st, kVBytes);
 #pragma unroll
         for (int kb = 0; kb < VA; ++kb)
-          tma2d(dv + kb * (kKB * 128), &map_v, (LINEAR ? head * kDV : 0) + kb * 64, row, v_full0 + 8 * st);
+          tma2d(dv + kb * (kKB * 128), &map_v, vx + kb * 64, row, v_full0 + 8 * st);
         return true;
       };
       // the waits follow the tensor core's order: S0 S1 | PV0 S2 | PV1 S3 | ...
@@ -335,10 +344,10 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t pair_bar = 1u + static_cast<uint32_t>(quad);   // named barrier of the warps sharing these rows
     auto pair_sync = [&]() { asm volatile("bar.sync %0, %1;" ::"r"(pair_bar), "n"(32 * kParts) : "memory"); };
-    const float c2 = LINEAR ? a.scale_log2 : 0.0625f * 1.4426950408889634f;            // 1/sqrt(256) * log2(e)
+    const float c2 = LINEAR || ROWS ? a.scale_log2 : 0.0625f * 1.4426950408889634f;            // 1/sqrt(256) * log2(e)
     const bool row_ok = r < q_rows;
     const int qpos = pos0 + tile * kQT + r;
-    const int row_lo = LINEAR ? max(pad, qpos - a.window + 1) : pad;            // first key this row sees
+    const int row_lo = LINEAR || ROWS ? max(pad, qpos - a.window + 1) : pad;            // first key this row sees
     float m_ref = -INFINITY, l = 0.f;
     const int warp_qpos0 = pos0 + tile * kQT + quad * 32;       // smallest query position of this warp
     bool ok = nb > 0;
@@ -362,7 +371,7 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
       // every row of this warp sees all of its keys: no mask arithmetic.  Rows past the end of a partial query tile
       // do not exist and are never stored, so they do not force the masked path (with 2047 rows they would, in
       // one warp pair of the LONGEST tile, which paces the whole kernel: the masked pass costs 800 cycles a block).
-      const bool full_blk = ok && kbase >= (LINEAR ? max(pad, warp_qpos0 + 31 - a.window + 1) : pad) &&
+      const bool full_blk = ok && kbase >= (LINEAR || ROWS ? max(pad, warp_qpos0 + 31 - a.window + 1) : pad) &&
                             kbase + kPartKeys - 1 <= min(warp_qpos0, limit);
       float mx = -INFINITY;
       if (full_blk) {
@@ -451,8 +460,8 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
     for (int q = 0; q < kParts; ++q) l += xmax[q][r];        // the same order in every thread of the row
     {
       // the TMEM loads are warp-wide: every lane takes part, only the stores are per row
-      const int out_cols = LINEAR ? a.v_cols : kDV;               // value columns that exist
-      const bool vec = !LINEAR || ((out_cols | a.ld_out) & 7) == 0;
+      const int out_cols = LINEAR || ROWS ? a.v_cols : kDV;               // value columns that exist
+      const bool vec = !(LINEAR || ROWS) || ((out_cols | a.ld_out) & 7) == 0;
       __nv_bfloat16* dst = a.out_bf16 + static_cast<size_t>(row0 + (row_ok ? r : 0)) * a.ld_out + head * out_cols;
       const bool have = nb > 0 && ok;
       const float inv = (have && l > 0.f) ? 1.0f / l : 0.f;
@@ -472,7 +481,7 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
         } else if (row_ok) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
-            if (LINEAR && c0 + i >= out_cols) continue;
+            if ((LINEAR || ROWS) && c0 + i >= out_cols) continue;
             uint4 w;
             w.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
             w.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
@@ -497,18 +506,18 @@ __global__ void __launch_bounds__(kThreadsTc, 1) prefill_attn_tc_kernel(const __
 // near-even finish (longest-processing-time order).  Pairing a long and a short tile inside one block, to get
 // one even wave of blocks, was measured slower (2.35 ms against 2.01 ms per GPT-J-6B prefill): the pipeline
 // drains and refills between a block's two tiles.
-template <int QA, int VA, bool LINEAR>
+template <int QA, int VA, int SRC>
 cudaError_t launch_attn_tc(const void* map_q, const void* map_k, const void* map_ks, const void* map_v,
                            const PrefillAttnTcArgs& a, cudaStream_t s) {
   constexpr int smem = static_cast<int>(AttnTcCfg<QA, VA>::kSmem);
   static DeviceOnce once;
   {
-    cudaError_t e = once.run([&] { return cudaFuncSetAttribute(prefill_attn_tc_kernel<QA, VA, LINEAR>,
+    cudaError_t e = once.run([&] { return cudaFuncSetAttribute(prefill_attn_tc_kernel<QA, VA, SRC>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem); });
     if (e != cudaSuccess) return e;
   }
   const dim3 grid(a.heads, (a.rows.Tc + kQT - 1) / kQT, a.M / a.rows.Tc);
-  prefill_attn_tc_kernel<QA, VA, LINEAR><<<grid, kThreadsTc, smem, s>>>(
+  prefill_attn_tc_kernel<QA, VA, SRC><<<grid, kThreadsTc, smem, s>>>(
       *static_cast<const CUtensorMap*>(map_q), *static_cast<const CUtensorMap*>(map_k),
       *static_cast<const CUtensorMap*>(map_ks), *static_cast<const CUtensorMap*>(map_v), a);
   return cudaGetLastError();

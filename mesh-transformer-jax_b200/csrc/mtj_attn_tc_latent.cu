@@ -17,15 +17,15 @@ cudaError_t launch_prefill_attn_tc_linear(const void* map_q, const void* map_k, 
       a.k_own < 0 || a.k_own > key_blocks)
     return cudaErrorInvalidValue;
   switch (key_blocks * 8 + value_blocks) {
-    case 2 * 8 + 1: return launch_attn_tc<2, 1, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 2 * 8 + 2: return launch_attn_tc<2, 2, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 2 * 8 + 4: return launch_attn_tc<2, 4, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 3 * 8 + 1: return launch_attn_tc<3, 1, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 3 * 8 + 2: return launch_attn_tc<3, 2, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 3 * 8 + 4: return launch_attn_tc<3, 4, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 4 * 8 + 1: return launch_attn_tc<4, 1, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 4 * 8 + 2: return launch_attn_tc<4, 2, true>(map_q, map_k, map_ks, map_v, a, s);
-    case 4 * 8 + 4: return launch_attn_tc<4, 4, true>(map_q, map_k, map_ks, map_v, a, s);
+    case 2 * 8 + 1: return launch_attn_tc<2, 1, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 2 * 8 + 2: return launch_attn_tc<2, 2, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 2 * 8 + 4: return launch_attn_tc<2, 4, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 3 * 8 + 1: return launch_attn_tc<3, 1, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 3 * 8 + 2: return launch_attn_tc<3, 2, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 3 * 8 + 4: return launch_attn_tc<3, 4, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 4 * 8 + 1: return launch_attn_tc<4, 1, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 4 * 8 + 2: return launch_attn_tc<4, 2, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
+    case 4 * 8 + 4: return launch_attn_tc<4, 4, kLinearRows>(map_q, map_k, map_ks, map_v, a, s);
     default: return cudaErrorInvalidValue;
   }
 }

@@ -77,6 +77,7 @@ cudaError_t launch_gemm_tc_wide(GemvEpilogue epi, const void* map_w, const void*
   const CUtensorMap& mw = *static_cast<const CUtensorMap*>(map_w);
   const CUtensorMap& mx = *static_cast<const CUtensorMap*>(map_x);
   if (epi == kEpiPlain || epi == kEpiSwiGLU) return launch_gemm_tc_stack(epi, true, mw, mx, a, s, false);
+  if (epi == kEpiRelu2 || epi == kEpiSoftcap) return launch_gemm_tc_stack_post(epi, true, mw, mx, a, s, false);
   return launch_gemm_tc_gptj(epi, true, mw, mx, nullptr, a, s, false);
 }
 
@@ -102,6 +103,8 @@ cudaError_t launch_gemm_tc(GemvEpilogue epi, const void* map_w, const void* map_
   const CUtensorMap& mx = *static_cast<const CUtensorMap*>(map_x);
   if (epi == kEpiPlain || epi == kEpiSwiGLU)
     return map_x_lo ? cudaErrorInvalidValue : launch_gemm_tc_stack(epi, false, mw, mx, a, s, pdl);
+  if (epi == kEpiRelu2 || epi == kEpiSoftcap)
+    return map_x_lo ? cudaErrorInvalidValue : launch_gemm_tc_stack_post(epi, false, mw, mx, a, s, pdl);
   return launch_gemm_tc_gptj(epi, false, mw, mx, static_cast<const CUtensorMap*>(map_x_lo), a, s, pdl);
 }
 

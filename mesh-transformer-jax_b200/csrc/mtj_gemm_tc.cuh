@@ -35,6 +35,8 @@ cudaError_t launch_gemm_tc_gptj(GemvEpilogue epi, bool wide, const CUtensorMap& 
 // mtj_gemm_tc_stack.cu
 cudaError_t launch_gemm_tc_stack(GemvEpilogue epi, bool wide, const CUtensorMap& map_w, const CUtensorMap& map_x,
                                  const GemmTcArgs& a, cudaStream_t s, bool pdl);
+cudaError_t launch_gemm_tc_stack_post(GemvEpilogue epi, bool wide, const CUtensorMap& map_w, const CUtensorMap& map_x,
+                                 const GemmTcArgs& a, cudaStream_t s, bool pdl);
 
 namespace {
 
@@ -142,6 +144,14 @@ __device__ __forceinline__ uint32_t tc_ld_shared(uint32_t addr) {
   return v;
 }
 
+__device__ __forceinline__ float squared_relu(float v) {
+  const float t = fmaxf(v, 0.f);
+  return t * t;
+}
+// cap * tanh(v / cap); the exponential's overflow and underflow end in +-cap
+__device__ __forceinline__ float softcap(float v, float cap) {
+  return cap - __fdividef(2.0f * cap, 1.0f + __expf(__fdividef(2.0f * v, cap)));
+}
 // silu(gate) * up
 __device__ __forceinline__ float swiglu(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
 
@@ -303,7 +313,7 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
           // one destination per loop: short code, which matters because every block runs it once
           const int valid = n_ok ? min(32, a.M - (m0 + c0)) : 0;
           float* dst = a.partial ? a.partial + (static_cast<size_t>(blockIdx.z) * a.M + m0 + c0) * a.N + n
-                                 : a.out ? a.out + static_cast<size_t>(m0 + c0) * a.ld_out + n : nullptr;
+                                 : a.out && n >= a.f32_from ? a.out + static_cast<size_t>(m0 + c0) * a.ld_out + n - a.f32_from : nullptr;
           const size_t ldd = a.partial ? a.N : a.ld_out;
           const float add = a.partial ? 0.f : bias;
           if (dst) {
@@ -311,12 +321,24 @@ __global__ void __launch_bounds__(kTcThreads) gemm_tc_kernel(const __grid_consta
             for (int i = 0; i < 32; ++i)
               if (i < valid) dst[i * ldd] = __uint_as_float(r[i]) + add;
           }
-          if (a.out_bf16 && !a.partial) {
+          if (a.out_bf16 && !a.partial && (a.f32_from == 0 || n < a.f32_from)) {
             __nv_bfloat16* d16 = a.out_bf16 + static_cast<size_t>(m0 + c0) * a.ld_bf16 + n;
 #pragma unroll
             for (int i = 0; i < 32; ++i)
               if (i < valid) d16[static_cast<size_t>(i) * a.ld_bf16] = __float2bfloat16_rn(__uint_as_float(r[i]) + add);
           }
+          return;
+        }
+        if constexpr (EPI == kEpiRelu2 || EPI == kEpiSoftcap) {
+          const int valid = n_ok ? min(32, a.M - (m0 + c0)) : 0;
+          __nv_bfloat16* d16 = EPI == kEpiRelu2 ? a.out_bf16 + static_cast<size_t>(m0 + c0) * a.ld_bf16 + n : nullptr;
+          float* dst = EPI == kEpiSoftcap ? a.out + static_cast<size_t>(m0 + c0) * a.ld_out + n : nullptr;
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (i < valid) {
+              if (EPI == kEpiRelu2) d16[static_cast<size_t>(i) * a.ld_bf16] = __float2bfloat16_rn(squared_relu(__uint_as_float(r[i])));
+              else dst[static_cast<size_t>(i) * a.ld_out] = softcap(__uint_as_float(r[i]), a.softcap);
+            }
           return;
         }
         if constexpr (EPI == kEpiSwiGLU) {
@@ -852,15 +874,29 @@ __global__ void __launch_bounds__(kPThreads, 1) gemm_tc_persist_kernel(const __g
             if (n_ok && q < valid && !(lane & 1))
               a.out_bf16[static_cast<size_t>(mc + q) * a.ld_bf16 + (n >> 1)] = __float2bfloat16_rn(swiglu(v, partner));
           }
+        } else if (EPI == kEpiRelu2) {
+          if (n_ok && valid > 0) {
+            __nv_bfloat16* dst = a.out_bf16 + static_cast<size_t>(mc) * a.ld_bf16 + n;
+#pragma unroll
+            for (int q = 0; q < 32; ++q)
+              if (q < valid) dst[static_cast<size_t>(q) * a.ld_bf16] = __float2bfloat16_rn(squared_relu(__uint_as_float(r[q])));
+          }
+        } else if (EPI == kEpiSoftcap) {
+          if (n_ok && valid > 0) {
+            float* dst = a.out + static_cast<size_t>(mc) * a.ld_out + n;
+#pragma unroll
+            for (int q = 0; q < 32; ++q)
+              if (q < valid) dst[static_cast<size_t>(q) * a.ld_out] = softcap(__uint_as_float(r[q]), a.softcap);
+          }
         } else if (EPI == kEpiPlain) {
           if (n_ok && valid > 0) {
-            if (a.out) {
-              float* dst = a.out + static_cast<size_t>(mc) * a.ld_out + n;
+            if (a.out && n >= a.f32_from) {
+              float* dst = a.out + static_cast<size_t>(mc) * a.ld_out + n - a.f32_from;
 #pragma unroll
               for (int q = 0; q < 32; ++q)
                 if (q < valid) dst[static_cast<size_t>(q) * a.ld_out] = __uint_as_float(r[q]) + bias;
             }
-            if (a.out_bf16) {
+            if (a.out_bf16 && (a.f32_from == 0 || n < a.f32_from)) {
               __nv_bfloat16* dst = a.out_bf16 + static_cast<size_t>(mc) * a.ld_bf16 + n;
 #pragma unroll
               for (int q = 0; q < 32; ++q)

@@ -14,8 +14,9 @@
 //             block to arrive (layers.py:285,290,313; transformer_shard.py:60)
 //   logits  : final LayerNorm prologue + bias (layers.py:561-564)
 //   SwiGLU  : LayerNorm prologue, rows in (gate, up) pairs, silu(gate) * up (layer-stack models)
+//   Relu2   : no prologue, squared relu (layer-stack models)
 // The LayerNorm prologue with mean = 0 and a zero offset is RMSNorm; the out-proj epilogue can add the residual
-// behind a second RMSNorm (GemvArgs::post_w).
+// behind a second RMSNorm (GemvArgs::post_w), or norm the residual sum (GemvArgs::post_b).
 #include "mtj_common.cuh"
 #include "mtj_kernels.h"
 
@@ -39,7 +40,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 
 template <int BT, int RW, int EPI, int KS>
 __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 3) : 2) gemv_kernel(const GemvArgs a) {
-  constexpr bool kLN = (EPI != kEpiOut);
+  constexpr bool kLN = (EPI != kEpiOut && EPI != kEpiRelu2);
   constexpr int kGroups = kGemvWarps / KS;      // row groups per block; KS warps share one group's K extent
   static_assert(RW * BT <= 32 && (RW & 1) == 0, "one lane finishes one (row, token) pair");
   const int lane = threadIdx.x & 31;
@@ -201,14 +202,19 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
       } else if (EPI == kEpiSwiGLU) {
         // (gate, up) row pairs: the even row finishes the pair
         if (!(r & 1)) a.act2[static_cast<size_t>(m) * a.ld_out + (n >> 1)] = val / (1.0f + expf(-val)) * partner;
+      } else if (EPI == kEpiRelu2) {
+        const float y = fmaxf(val, 0.f);
+        a.act2[static_cast<size_t>(m) * a.ld_out + n] = y * y;
       } else {
-        a.logits[static_cast<size_t>(m) * a.ld_logits + n] = a.bias ? val + a.bias[n] : val;
+        float y = a.bias ? val + a.bias[n] : val;
+        if (a.softcap > 0.f) y = a.softcap * tanhf(y / a.softcap);
+        a.logits[static_cast<size_t>(m) * a.ld_logits + n] = y;
       }
     }
   }
 
   if (EPI == kEpiOut) {
-    if (a.stats_out == nullptr) return;
+    if (a.stats_out == nullptr && a.post_w == nullptr) return;
     // The last block of this token tile to finish computes the LayerNorm
     // statistics of the completed rows for the next layer's prologue.
     __shared__ float red[kGemvWarps];
@@ -222,6 +228,88 @@ __global__ void __launch_bounds__(kGemvThreads, BT == 1 ? (EPI == kEpiOut ? 4 : 
     __syncthreads();
     if (!is_last) return;
     __threadfence();
+    if (a.post_b) {
+      // layer norm of the residual sum; the row lives in registers (kHold float4 a thread) or is read again from L2
+      const int n_out = a.n_valid > 0 ? a.n_valid : a.N;
+      constexpr int kHold = 4;
+      const int ldo = a.ld_out > 0 ? a.ld_out : a.N;
+      const float inv_n = 1.0f / static_cast<float>(n_out);
+      const bool held = ((n_out | ldo | a.post_ldx) & 3) == 0 && n_out <= kHold * 4 * kGemvThreads;
+      for (int bt = 0; bt < nb; ++bt) {
+        const float* row = a.out + static_cast<size_t>(m0 + bt) * ldo;
+        float* xrow = a.post_x + static_cast<size_t>(m0 + bt) * a.post_ldx;
+        float mu2 = 0.f, rs2 = 0.f;
+        if (held) {
+          float4 z[kHold];
+          float s = 0.f, q = 0.f;
+          const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+          for (int i = 0; i < kHold; ++i) {
+            const int c = 4 * (i * kGemvThreads + static_cast<int>(threadIdx.x));
+            const bool in = c < n_out;
+            const float4 y = in ? __ldcg(reinterpret_cast<const float4*>(row + c)) : zero;
+            const float4 x = in ? *reinterpret_cast<const float4*>(xrow + c) : zero;
+            if (in) prefetch_l2(a.post_w + c);
+            if (in) prefetch_l2(a.post_b + c);
+            z[i] = make_float4(fmaf(a.post_mult, x.x, y.x), fmaf(a.post_mult, x.y, y.y), fmaf(a.post_mult, x.z, y.z), fmaf(a.post_mult, x.w, y.w));
+            s += (z[i].x + z[i].y) + (z[i].z + z[i].w);
+          }
+          auto centred = [&](float mu) {                  // sum of squared deviations
+            float v = 0.f;
+#pragma unroll
+            for (int i = 0; i < kHold; ++i)
+              if (4 * (i * kGemvThreads + static_cast<int>(threadIdx.x)) < n_out) {
+                const float dx = z[i].x - mu, dy = z[i].y - mu, dz = z[i].z - mu, dw = z[i].w - mu;
+                v += (dx * dx + dy * dy) + (dz * dz + dw * dw);
+              }
+            return v;
+          };
+          const float mu = block_sum(s, red) * inv_n;
+          const float rs = 1.0f / sqrtf(block_sum(centred(mu), red) * inv_n + a.post_eps);
+#pragma unroll
+          for (int i = 0; i < kHold; ++i) {
+            const int c = 4 * (i * kGemvThreads + static_cast<int>(threadIdx.x));
+            if (c < n_out) {
+              const float4 w = *reinterpret_cast<const float4*>(a.post_w + c), b = *reinterpret_cast<const float4*>(a.post_b + c);
+              z[i] = make_float4(fmaf((z[i].x - mu) * rs, w.x, b.x), fmaf((z[i].y - mu) * rs, w.y, b.y),
+                                 fmaf((z[i].z - mu) * rs, w.z, b.z), fmaf((z[i].w - mu) * rs, w.w, b.w));
+              *reinterpret_cast<float4*>(xrow + c) = z[i];
+              q += (z[i].x + z[i].y) + (z[i].z + z[i].w);
+            }
+          }
+          if (a.stats_out) {
+            mu2 = block_sum(q, red) * inv_n;
+            rs2 = 1.0f / sqrtf(block_sum(centred(mu2), red) * inv_n + a.post_eps);
+          }
+        } else {
+          float s = 0.f, v = 0.f;
+          for (int i = threadIdx.x; i < n_out; i += kGemvThreads) s += fmaf(a.post_mult, xrow[i], __ldcg(row + i));
+          const float mu = block_sum(s, red) * inv_n;
+          for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+            const float z = fmaf(a.post_mult, xrow[i], __ldcg(row + i)) - mu;
+            v = fmaf(z, z, v);
+          }
+          const float rs = 1.0f / sqrtf(block_sum(v, red) * inv_n + a.post_eps);
+          s = v = 0.f;
+          for (int i = threadIdx.x; i < n_out; i += kGemvThreads) {
+            const float x = fmaf((fmaf(a.post_mult, xrow[i], __ldcg(row + i)) - mu) * rs, a.post_w[i], a.post_b[i]);
+            xrow[i] = x;                                  // each thread re-reads only what it wrote
+            s += x;
+          }
+          if (a.stats_out) {
+            mu2 = block_sum(s, red) * inv_n;
+            for (int i = threadIdx.x; i < n_out; i += kGemvThreads) v = fmaf(xrow[i] - mu2, xrow[i] - mu2, v);
+            rs2 = 1.0f / sqrtf(block_sum(v, red) * inv_n + a.post_eps);
+          }
+        }
+        if (threadIdx.x == 0 && a.stats_out) {
+          a.stats_out[2 * (m0 + bt)] = mu2;
+          a.stats_out[2 * (m0 + bt) + 1] = rs2;
+        }
+      }
+      if (threadIdx.x == 0) a.counters[blockIdx.y] = 0u;
+      return;
+    }
     if (a.post_w) {
       // norm after the sublayer, residual add, and the root mean square of the new residual row
       const int n_out = a.n_valid > 0 ? a.n_valid : a.N;
@@ -365,6 +453,7 @@ cudaError_t launch_gemv(GemvEpilogue epi, const GemvArgs& a, cudaStream_t s, boo
     case kEpiInProj: return launch_epi<kEpiInProj>(a, s, pdl);
     case kEpiOut: return launch_epi<kEpiOut>(a, s, pdl);
     case kEpiSwiGLU: return launch_epi<kEpiSwiGLU>(a, s, pdl);
+    case kEpiRelu2: return launch_epi<kEpiRelu2>(a, s, pdl);
     default: return launch_epi<kEpiLogits>(a, s, pdl);
   }
 }

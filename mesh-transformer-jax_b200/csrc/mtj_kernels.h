@@ -29,7 +29,9 @@ enum GemvEpilogue { kEpiInProj = 0, kEpiOut = 1, kEpiLogits = 2,
                     kEpiLogitsCE = 3,     // logits that are never stored: per (128-entry vocabulary group, token) max and
                                           // sum of exp instead, plus the target's logit (persistent GEMM only)
                     kEpiPlain = 4,        // fp32 and / or bf16 result (tensor-core GEMM only)
-                    kEpiSwiGLU = 5 };     // weight rows in (gate, up) pairs: silu(gate) * up
+                    kEpiSwiGLU = 5,       // weight rows in (gate, up) pairs: silu(gate) * up
+                    kEpiRelu2 = 6,        // squared relu
+                    kEpiSoftcap = 7 };    // cap * tanh(result / cap), fp32 (tensor-core GEMM; the GEMV takes GemvArgs.softcap)
 
 struct GemvArgs {
   // y[m, n] = sum_k W[n, k] * act(x[m, k]);  W is bf16 [N, K] (K contiguous).
@@ -73,6 +75,10 @@ struct GemvArgs {
   float* post_x;               // [M, post_ldx]
   int post_ldx;
   float post_mult, post_eps;
+  // with post_b: post_x = LayerNorm(post_mult * post_x + out) * post_w + post_b instead, and stats_out, if given, takes
+  // the (mean, 1 / deviation) of the new post_x
+  const float* post_b;         // [n_valid] or null
+  float softcap;               // logits epilogue: cap * tanh(logit / cap); 0 = none
 };
 
 cudaError_t launch_gemv(GemvEpilogue epi, const GemvArgs& a, cudaStream_t s, bool pdl);
@@ -90,6 +96,8 @@ struct EmbedArgs {
   const uint32_t* slot_sel;    // optional: x += (*slot_sel & 1) * slot_stride (peer all-reduce slots)
   size_t slot_stride;
   int ldx;                     // row stride of x (0 = d)
+  float scale;                 // rows are multiplied by it (0 = 1)
+  __nv_bfloat16* x_bf16;       // optional [M, ldx]: the rows once more in bf16
 };
 cudaError_t launch_embed(const EmbedArgs& a, cudaStream_t s, bool pdl);
 
@@ -142,6 +150,9 @@ struct PrefillAttnTcArgs {
   int k_own;                   // 64-column blocks of a key row that belong to the head (the rest: all heads share them)
   int v_cols;                  // value columns per head that exist (the matrix pads them to whole 64-column blocks)
   float scale_log2;            // score scale times log2(e)
+  // paged rows (launch_prefill_attn_tc_grouped): kv.page_table, kv.ring_pages and kv.pad, window, v_cols, scale_log2, and
+  int kv_group;                // query heads per key head
+  int k_cols, v_ld;            // columns of a key head in the key and value rows, multiples of 8
 };
 cudaError_t launch_prefill_attn_tc(const void* map_q, const void* map_k, const void* map_v,
                                    const PrefillAttnTcArgs& a, cudaStream_t s);
@@ -150,6 +161,11 @@ int attn_tc_key_blocks(int own_dim, int shared_dim);
 int attn_tc_value_blocks(int vdim);
 cudaError_t launch_prefill_attn_tc_linear(const void* map_q, const void* map_k, const void* map_ks, const void* map_v,
                                           int key_blocks, int value_blocks, const PrefillAttnTcArgs& a, cudaStream_t s);
+
+// 64-column blocks of a head the paged-rows form takes, 0 = larger than its instances; query rows are padded to them
+int attn_tc_grouped_blocks(int dim);
+cudaError_t launch_prefill_attn_tc_grouped(const void* map_q, const void* map_k, const void* map_v, int key_blocks,
+                                           int value_blocks, const PrefillAttnTcArgs& a, cudaStream_t s);
 
 // Persistent whole-step decode kernel (mtj_decode_mega.cu), one GPU, 1-4 sequences.
 struct MegaLayer {
@@ -250,8 +266,11 @@ struct GemmTcArgs {
   int ce_T, ce_vocab_start;
   int cluster_k;               // 2 or 4 (token tiles of at most 64 rows, partial == null): split K over a cluster of
                                // blocks that add their accumulators in shared memory before the fused epilogue
-  __nv_bfloat16* out_bf16;     // kEpiPlain: optional bf16 result; kEpiSwiGLU: the result (N / 2 columns)
+  __nv_bfloat16* out_bf16;     // kEpiPlain: optional bf16 result; kEpiSwiGLU: the result (N / 2 columns); kEpiRelu2: the result
   int ld_bf16;
+  int f32_from;                // kEpiPlain, > 0: weight rows from this one on go to `out` (columns counted from it), the rest
+                               // to out_bf16; 0: every row to both
+  float softcap;               // kEpiSoftcap
   int pair;                    // wide kernel only: 1 = clusters of 2 blocks on 256 x 256 tiles (tcgen05 cta_group::2)
   uint32_t* dev_err;
 };

@@ -40,8 +40,9 @@ __global__ void __launch_bounds__(kThreads) embed_kernel(const EmbedArgs a) {
               static_cast<size_t>(m) * (a.ldx > 0 ? a.ldx : a.d);
   float s = 0.f;
   for (int i = threadIdx.x; i < a.d; i += kThreads) {
-    const float v = (hit ? __bfloat162float(row[i]) : 0.f) + (a.bias ? a.bias[i] : 0.f);
+    const float v = ((hit ? __bfloat162float(row[i]) : 0.f) + (a.bias ? a.bias[i] : 0.f)) * (a.scale != 0.f ? a.scale : 1.0f);
     xo[i] = v;
+    if (a.x_bf16) a.x_bf16[static_cast<size_t>(m) * (a.ldx > 0 ? a.ldx : a.d) + i] = __float2bfloat16_rn(v);
     s += v;
   }
   if (a.stats == nullptr) return;

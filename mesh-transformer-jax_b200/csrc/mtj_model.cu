@@ -699,7 +699,7 @@ int32_t mtj_set_error(int32_t code, const char* msg) {
   g_last_error = msg ? msg : "";
   return code;
 }
-int32_t mtj_version(void) { return 4; }
+int32_t mtj_version(void) { return 5; }
 
 int32_t mtj_create(const mtj_config* c, mtj_handle** out) {
   if (!c || !out) return fail(MTJ_ERR_INVALID, "null argument");

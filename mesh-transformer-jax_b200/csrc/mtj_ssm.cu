@@ -553,11 +553,12 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmArgs a) {
   }
 }
 
-bool ssm_ok(const SsmArgs& a) {
-  return a.M > 0 && a.inner > 0 && a.state > 0 && a.state <= kSsmMaxState && a.taps >= 1 && a.nseq > 0 && a.rows.Tc > 0 &&
+bool conv_ok(const SsmArgs& a) {
+  return a.M > 0 && a.inner > 0 && a.taps >= 1 && a.nseq > 0 && a.rows.Tc > 0 &&
          a.M == a.nseq * a.rows.Tc && a.ld_u >= a.inner && (a.ld_u & 7) == 0 && (a.ld_xz & 7) == 0 && (a.u != nullptr) != (a.u_bf16 != nullptr) &&
          (a.u != nullptr) == !a.xz_bf16;
 }
+bool ssm_ok(const SsmArgs& a) { return conv_ok(a) && a.state > 0 && a.state <= kSsmMaxState; }
 
 template <typename T, int G, int NS>
 cudaError_t scan(const SsmArgs& a, cudaStream_t s) {
@@ -613,7 +614,7 @@ cudaError_t conv_vec(const SsmArgs& a, cudaStream_t s, bool pdl) {
 }  // namespace
 
 cudaError_t launch_ssm_conv(const SsmArgs& a, cudaStream_t s, bool pdl) {
-  if (!ssm_ok(a)) return cudaErrorInvalidValue;
+  if (!conv_ok(a)) return cudaErrorInvalidValue;
   const int cb = (a.inner + 255) / 256;
   if (a.rows.Tc == 1)
     return a.xz_bf16 ? launch_pdl(ssm_conv_step_kernel<__nv_bfloat16>, dim3(cb, a.M), dim3(256), 0, s, pdl, a)

@@ -101,6 +101,65 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
   }
 }
 
+// The same for layers with a layer norm behind the residual sum.
+__global__ void __launch_bounds__(kRnThreads) residual_layernorm_kernel(const ResidualLayerNormArgs a) {
+  extern __shared__ float4 rn_row[];
+  __shared__ float red[kRnThreads / 32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int n4 = a.ld >> 2;
+  const size_t m = blockIdx.x;
+  float4* xrow = reinterpret_cast<float4*>(a.x + m * a.ld);
+  const float inv_n = 1.0f / static_cast<float>(a.d);
+  auto norm = [&](float sum, float* mu, float* rs) {
+    *mu = rn_block_sum(sum, red) * inv_n;
+    float v = 0.f;
+    for (int i = threadIdx.x; i < n4; i += kRnThreads) {
+      const float4 z = rn_row[i];
+      const int left = a.d - 4 * i;                       // columns that exist
+      v += dot4(make_float4(left > 0 ? z.x - *mu : 0.f, left > 1 ? z.y - *mu : 0.f, left > 2 ? z.z - *mu : 0.f, left > 3 ? z.w - *mu : 0.f));
+    }
+    *rs = 1.0f / sqrtf(rn_block_sum(v, red) * inv_n + a.eps);
+  };
+  auto scaled = [&](int i, float mu, float rs, const float* w, const float* b) {
+    const float4 z = rn_row[i], w4 = reinterpret_cast<const float4*>(w)[i], b4 = reinterpret_cast<const float4*>(b)[i];
+    return make_float4(fmaf((z.x - mu) * rs, w4.x, b4.x), fmaf((z.y - mu) * rs, w4.y, b4.y), fmaf((z.z - mu) * rs, w4.z, b4.z),
+                       fmaf((z.w - mu) * rs, w4.w, b4.w));
+  };
+  float sum = 0.f, mu, rs;
+  for (int i = threadIdx.x; i < n4; i += kRnThreads) {
+    float4 x = xrow[i];
+    if (a.y) {
+      const float4 y = reinterpret_cast<const float4*>(a.y + m * a.ld)[i];
+      x = make_float4(fmaf(a.alpha, x.x, y.x), fmaf(a.alpha, x.y, y.y), fmaf(a.alpha, x.z, y.z), fmaf(a.alpha, x.w, y.w));
+    }
+    rn_row[i] = x;
+    sum += (x.x + x.y) + (x.z + x.w);
+  }
+  if (a.y) {
+    norm(sum, &mu, &rs);
+    sum = 0.f;
+    for (int i = threadIdx.x; i < n4; i += kRnThreads) {
+      const float4 x = scaled(i, mu, rs, a.w, a.b);       // w and b are zero in the padding
+      rn_row[i] = x;
+      xrow[i] = x;
+      sum += (x.x + x.y) + (x.z + x.w);
+      if (a.xn && !a.w_next) reinterpret_cast<uint2*>(a.xn + m * a.ld)[i] = pack4(x);
+    }
+  } else if (a.xn && !a.w_next) {
+    for (int i = threadIdx.x; i < n4; i += kRnThreads) reinterpret_cast<uint2*>(a.xn + m * a.ld)[i] = pack4(rn_row[i]);
+  }
+  if (!a.w_next && !a.stats) return;
+  norm(sum, &mu, &rs);
+  if (a.stats && threadIdx.x == 0) {
+    a.stats[2 * m] = mu;
+    a.stats[2 * m + 1] = rs;
+  }
+  if (a.xn && a.w_next)
+    for (int i = threadIdx.x; i < n4; i += kRnThreads)
+      reinterpret_cast<uint2*>(a.xn + m * a.ld)[i] = pack4(scaled(i, mu, rs, a.w_next, a.b_next));
+}
+
 __global__ void gather_rows_bf16_kernel(const __nv_bfloat16* __restrict__ src, int ld, const int32_t* __restrict__ rows,
                                         __nv_bfloat16* __restrict__ dst) {
   const uint4* s = reinterpret_cast<const uint4*>(src + static_cast<size_t>(rows[blockIdx.x]) * ld);
@@ -155,6 +214,18 @@ cudaError_t launch_residual_norm(const ResidualNormArgs& a, cudaStream_t s, bool
   });
   if (e != cudaSuccess) return e;
   return launch_pdl(residual_norm_kernel, dim3(a.M), dim3(kRnThreads), smem, s, pdl, a);
+}
+
+cudaError_t launch_residual_layernorm(const ResidualLayerNormArgs& a, cudaStream_t s, bool pdl) {
+  if (a.M <= 0 || a.d <= 0 || a.ld < a.d || (a.ld & 3) || (a.y && (!a.w || !a.b)) || (a.w_next && !a.b_next)) return cudaErrorInvalidValue;
+  const size_t smem = static_cast<size_t>(a.ld) * sizeof(float);
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  static DeviceOnce once;
+  cudaError_t e = once.run([&] {
+    return cudaFuncSetAttribute(residual_layernorm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  });
+  if (e != cudaSuccess) return e;
+  return launch_pdl(residual_layernorm_kernel, dim3(a.M), dim3(kRnThreads), smem, s, pdl, a);
 }
 
 cudaError_t launch_gather_rows_bf16(const __nv_bfloat16* src, int ld, const int32_t* rows, int n, __nv_bfloat16* dst,

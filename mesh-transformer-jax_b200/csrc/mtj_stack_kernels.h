@@ -42,6 +42,19 @@ struct ResidualNormArgs {
   __nv_bfloat16* cat_bf16;     // [M, 2 ld] or null
 };
 cudaError_t launch_residual_norm(const ResidualNormArgs& a, cudaStream_t s, bool pdl);
+// One row per block:  x = LayerNorm(alpha * x + y) * w + b;  then xn = x in bf16, or, with w_next, the layer norm of the
+// new x in bf16, and its (mean, 1 / deviation) into stats.  y == null: x stays, only what follows is done.
+struct ResidualLayerNormArgs {
+  float* x;                    // [M, ld]; columns d .. ld - 1 of every buffer here are zero
+  int M, d, ld;
+  const float* y;              // [M, ld] or null
+  const float *w, *b;          // [ld]
+  float alpha, eps;
+  __nv_bfloat16* xn;           // [M, ld] or null
+  const float *w_next, *b_next;  // [ld] or null
+  float* stats;                // [M, 2] or null
+};
+cudaError_t launch_residual_layernorm(const ResidualLayerNormArgs& a, cudaStream_t s, bool pdl);
 cudaError_t launch_gather_rows_bf16(const __nv_bfloat16* src, int ld, const int32_t* rows, int n, __nv_bfloat16* dst,
                                     cudaStream_t s);
 // src [N, K] (bf16 or fp32) -> bf16 dst[(r0 + n / gin * gout + n % gin) * ld + (k < csplit ? k : k + cshift)]
@@ -101,6 +114,87 @@ cudaError_t launch_latent_history(const LatentArgs& a, cudaStream_t s);
 constexpr int kLatentMaxRank = 1024;
 constexpr int kLatentBlocks = 592;       // most (rows x splits x head groups) a call spreads over beyond one per row
 int latent_attn_splits(int M, int heads, int row_ld, int tensor_cores, int window);
+
+// ---- mtj_grouped_attn.cu: softmax attention of query heads over shared key / value heads, causal or windowed
+struct GroupedCache {
+  void *k, *v;                 // [pages][kPageTokens][kv_heads * up8(dim)] | [..][kv_heads * up8(vdim)], bf16 or fp32
+  int f32;
+  const int32_t* page_table;   // [sequences][ring_pages]; ring slot of own position p: (p / kPageTokens) % ring_pages
+  int ring_pages, k_ld, v_ld;
+};
+struct GroupedAttnArgs {
+  int M, heads, kv_heads, dim, vdim, window;
+  float scale, eps;
+  float q_temp_coef;
+  double q_temp_every;         // 0: no temperature
+  RowMap rows;
+  const int32_t* pad;
+  GroupedCache cache;
+  const float* p1;             // [M, ld_p1] q | k | v (only q where own_kv is 0)
+  int ld_p1, own_kv;
+  const float *q_norm, *k_norm;
+  // queries, normed and scaled by the temperature: bf16 heads of q_cols columns, zero-padded, or fp32 heads of up8(dim)
+  __nv_bfloat16* q_bf16;
+  float* q_f32;
+  int q_cols;
+  int splits;                  // key ranges per row
+  float* part_o;               // [M, heads, splits, vdim]
+  float* part_ml;              // [M, heads, splits, 2]
+  uint32_t* counters;          // [M * kv_heads * ceil(heads / kv_heads / 8)], zero between launches
+  float* out;                  // [M, ld_out] or null
+  __nv_bfloat16* out_bf16;     // [M, ld_out] or null
+  int ld_out;
+};
+// norms the queries and keys, writes the queries and, into the cache, keys and values
+cudaError_t launch_grouped_prep(const GroupedAttnArgs& a, cudaStream_t s, bool pdl);
+// every row of the call by itself, from the cache
+cudaError_t launch_grouped_attn(const GroupedAttnArgs& a, cudaStream_t s, bool pdl);
+constexpr int kGroupedMaxDim = 512;
+constexpr int kGroupedBlocks = 592;      // most (rows x key heads x splits) a call spreads over beyond one per row and head
+int grouped_attn_splits(int M, int heads, int kv_heads, int window);
+int grouped_counters(int heads, int kv_heads);   // per row
+
+// ---- mtj_matrix_state.cu: recurrences whose state is a matrix per head, keys x values
+//   SSD    S <- exp(A dt) S + dt k v^T,  o = S^T q + D v, with dt = softplus(decay + decay_b) per head
+//   delta  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q, with unit k and q (q times q_scale),
+//          g = exp(A softplus(decay + decay_b)) per head and key channel, beta = sigmoid
+struct MatrixStateArgs {
+  int M, heads, key_heads, dim, vdim;
+  int delta;
+  RowMap rows;
+  int nseq;
+  const int32_t* pad;
+  const void* u;               // [M, ld_u] convolved keys, queries and values at columns k0, q0, v0; fp32 or bf16
+  int u_bf16, ld_u, q0, k0, v0;
+  const float* decay;          // [M, ld_decay]
+  int ld_decay;
+  const float* decay_b;        // [heads] | [heads * dim]
+  const float* A;              // [heads], negative
+  const float* beta;           // [M, ld_beta], delta
+  int ld_beta;
+  const float* D;              // [heads], SSD
+  float q_scale;
+  float* state;                // [slots][heads][dim][vdim]
+  float* out;                  // [M, ld_out]
+  int ld_out;
+};
+cudaError_t launch_matrix_scan(const MatrixStateArgs& a, cudaStream_t s, bool pdl);
+// the outputs' norm and gate: parts of part_n neighbouring columns, each by its own root mean square;
+// gate_first: RMSNorm(y * silu(gate)) * w[column], else RMSNorm(y) * w[column within the part] * sigmoid(gate)
+struct GatedNormArgs {
+  int M, parts, part_n, gate_first;
+  float eps;
+  const float* y;              // [M, ld_y]
+  int ld_y;
+  const void* gate;            // [M, ld_gate], fp32 or bf16
+  int gate_bf16, ld_gate;
+  const float* w;
+  float* out;                  // [M, ld_out] or null
+  __nv_bfloat16* out_bf16;
+  int ld_out;
+};
+cudaError_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl);
+constexpr int kMatrixMaxDim = 256;
 
 // ---- mtj_ssm.cu: causal convolution and selective scan with carried state
 struct SsmArgs {

@@ -32,15 +32,17 @@ class MtjConfig(ctypes.Structure):
 
 class MtjLayerDesc(ctypes.Structure):
     _fields_ = ([(n, ctypes.c_int32) for n in (
-        "mixer", "ff", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "inner", "state", "conv", "dt_rank")]
-        + [("scale", ctypes.c_float), ("reserved", ctypes.c_int32), ("rot_base", ctypes.c_double)])
+        "mixer", "ff", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "inner", "state", "conv", "dt_rank",
+        "ff_kind", "kv_heads", "kv_from", "norm_groups", "decay_rank", "gate_rank")]
+        + [("scale", ctypes.c_float), ("q_temp_coef", ctypes.c_float), ("q_temp_every", ctypes.c_double),
+           ("rot_base", ctypes.c_double)])
 
 
 class MtjStackDesc(ctypes.Structure):
     _fields_ = ([("layers", ctypes.POINTER(MtjLayerDesc))]
-                + [(n, ctypes.c_int32) for n in ("n_layers", "loop_start", "loop_stop", "loop_times")]
-                + [("residual_mult", ctypes.c_float), ("norm_eps", ctypes.c_float), ("act_f32", ctypes.c_int32),
-                   ("tc_min_rows", ctypes.c_int32)])
+                + [(n, ctypes.c_int32) for n in ("n_layers", "loop_start", "loop_stop", "loop_times", "residual")]
+                + [(n, ctypes.c_float) for n in ("residual_mult", "norm_eps", "embed_scale", "logit_softcap")]
+                + [("act_f32", ctypes.c_int32), ("tc_min_rows", ctypes.c_int32)])
 
 
 def _load():

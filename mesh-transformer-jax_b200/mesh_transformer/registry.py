@@ -7,6 +7,9 @@ A family is a class with static methods
     param_shapes(config)  {module: {leaf: per-shard shape}}
     create(config, caps, handle)   makes the library handle, returns its status
     init_state(config, rank, device, seed)   random ``state``
+and, to load model folders,
+    fit_tensors(config, shapes)   the configuration with the sizes that only the tensors' shapes tell
+    state_from_tensors(config, tensors)   the parameter tree of ``state``
 A configuration without the key is the reference's GPT-J (its config JSON has no such key).
 """
 from __future__ import annotations
@@ -16,7 +19,7 @@ import json
 import os
 
 _FAMILIES: dict = {}
-_MODULES = {"gptj": "_runtime", "Keselix": "layer_stack"}     # where each family registers itself
+_MODULES = {"gptj": "_runtime", "Keselix": "layer_stack", "Bavutar": "layer_stack"}     # where each family registers itself
 
 
 def register(*names):
@@ -60,7 +63,8 @@ def load_network(folder: str, device=None, **overrides):
     fam = family(config)
     if not hasattr(fam, "state_from_tensors"):
         raise NotImplementedError("this family does not load model folders; use load_ckpt or hf_interchange")
-    net = CausalTransformer(config, device=device, init_weights=False)
     tensors = read_safetensors(os.path.join(folder, "model.safetensors"))
+    config = fam.fit_tensors(config, {n: tuple(t.shape) for n, t in tensors.items()})
+    net = CausalTransformer(config, device=device, init_weights=False)
     net.state = {"params": fam.state_from_tensors(config, tensors), "step": np.array(0), "opt_state": None}
     return net

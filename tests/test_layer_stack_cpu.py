@@ -26,7 +26,7 @@ def test_tensor_names_and_shapes(name):
 
 def test_registry_picks_families_and_rejects_what_it_cannot_run():
     from mesh_transformer import registry
-    assert registry.names() == ["Keselix", "gptj"]
+    assert registry.names() == ["Bavutar", "Keselix", "gptj"]
     assert registry.family({}).__name__ == "GptJ"
     with pytest.raises(NotImplementedError):
         registry.family({"architecture": "no such design"})
