@@ -612,7 +612,7 @@ def run_mtj(args):
 
 
 # ------------------------------------------------------- layer-stack models ----
-def stack_model(d):
+def keselix_model(d):
     """A Keselix model with layers of a real model's proportions at width d: a state-space layer and a latent-attention
     layer in turn, the middle two run twice."""
     attn = {"type": "latent_attention",
@@ -624,22 +624,56 @@ def stack_model(d):
             "loop": {"start": 1, "stop": 3, "times": 2}, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "seq": 2048}
 
 
-def stack_work(cfg, runs, T, window):
-    """(weight elements a decode step reads, flops of a T-token prompt without the logits) over the layer runs."""
+def bavutar_model(d):
+    """A Bavutar model with layers of a real model's proportions at width d: delta-rule, attention, Mamba-2 and delta-rule
+    layers, an attention layer that reads the first one's keys and values, and a Mamba-2 layer."""
+    mlp = {"kind": "dense", "ff": 3 * d}
+    attn = {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": d // 128, "kv_heads": d // 512, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                      "q_temp": {"coef": 0.1, "every": 8192}}}
+    delta = {"type": "channel_delta", "mlp": mlp,
+             "mixer": {"heads": d // 128, "kv_heads": d // 128, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}}
+    ssd = {"type": "mamba2", "mlp": mlp,
+           "mixer": {"heads": d // 32, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}}
+    late = dict(attn, mixer=dict(attn["mixer"], kv_from=1))
+    return {"architecture": "Bavutar", "vocab": 32768, "width": d, "layers": [delta, attn, ssd, delta, late, ssd], "norm": {"eps": 1e-5},
+            "postln_alpha": 2.0, "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "seq": 2048}
+
+
+def stack_work(cfg, runs, T):
+    """(weight elements a decode step reads, flops of a T-token prompt without the logits, bytes of caches and states a
+    sequence of T tokens moves in a decode step) over the layer runs."""
     from mesh_transformer.layer_stack import tensor_shapes
     import math
     shapes = tensor_shapes(cfg)
-    weights = sum(math.prod(v) for i in runs for k, v in shapes.items() if k.startswith(f"l{i}.") and len(v) > 1)
-    weights += cfg["loop"]["times"] * math.prod(shapes["loop.in"])
-    pairs = sum(min(t + 1, window) for t in range(T))
-    attn = sum(2 * pairs * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
-               for m in (cfg["layers"][i]["mixer"] for i in runs if cfg["layers"][i]["type"] == "latent_attention"))
-    return weights, 2 * weights * T + attn
+    weights = sum(math.prod(v) for i in runs for k, v in shapes.items()
+                  if k.startswith(f"l{i}.") and len(v) > 1 and "conv" not in k and "A_log" not in k)
+    if cfg.get("loop"):
+        weights += cfg["loop"]["times"] * math.prod(shapes["loop.in"])
+    extra, moved = 0, 0
+    for i in runs:
+        kind, m = cfg["layers"][i]["type"], cfg["layers"][i]["mixer"]
+        if kind == "latent_attention":
+            w = m["mask"]["size"]
+            extra += 2 * sum(min(t + 1, w) for t in range(T)) * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
+            moved += min(T, w) * (m["kv_rank"] + m["rot_dim"]) * 2
+        elif kind == "attention":
+            extra += T * (T + 1) * m["heads"] * (m["dim"] + m["vdim"])
+            moved += T * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+        elif kind == "mamba1":
+            extra += 6 * T * m["inner"] * m["state"]
+            moved += 2 * m["inner"] * 4 * (m["state"] + m["conv"] - 1)
+        else:
+            n = m["state"] if kind == "mamba2" else m["dim"]
+            extra += (6 if kind == "mamba2" else 8) * T * m["heads"] * n * m["vdim"]
+            moved += 2 * m["heads"] * n * m["vdim"] * 4
+    return weights, 2 * weights * T + extra, moved
 
 
 def run_stack(args):
-    """Keselix beside GPT-J (the closest model) at equal width and number of layer runs, one GPU, random weights:
-    prefill of one 2048-token prompt, decode of 1, 8 and 32 sequences behind such prompts, kernel families."""
+    """A layer-stack model beside another at equal width and number of layer runs (Keselix beside GPT-J, Bavutar beside
+    Keselix), one GPU, random weights: prefill of one 2048-token prompt, decode of 1, 8 and 32 sequences behind such
+    prompts, kernel families."""
     import torch
     import __graft_entry__ as ge
     if args.gpus != 1:
@@ -672,21 +706,18 @@ def run_stack(args):
     t_wall0 = time.time()
     T, K, W = 2048, args.steps, args.warmup
     sizes, launches = {}, 0
+    names = {"keselix": ("keselix", "gptj"), "bavutar": ("bavutar", "keselix")}[args.stack_model]
     for d in [int(v) for v in args.stack_widths.split(",")]:
-        kes = stack_model(d)
-        runs = [0, 1, 2, 1, 2, 3]
-        window = kes["layers"][1]["mixer"]["mask"]["size"]
-        gptj = dict(GPTJ_6B, layers=len(runs), d_model=d, n_heads=d // 256, n_vocab=kes["vocab"], early_cast=True)
+        models = {"keselix": lambda: (keselix_model(d), [0, 1, 2, 1, 2, 3]), "bavutar": lambda: (bavutar_model(d), list(range(6))),
+                  "gptj": lambda: (dict(GPTJ_6B, layers=6, d_model=d, n_heads=d // 256, n_vocab=32768, early_cast=True), list(range(6)))}
         row = {}
-        for name, cfg in (("keselix", kes), ("gptj", gptj)):
+        for name in names:
+            cfg, runs = models[name]()
             net = CausalTransformer(dict(cfg), device=device, init_weights=False)
             net.state = net._init_state(seed=42)
-            V = cfg.get("n_vocab", kes["vocab"])
-            if name == "keselix":
-                weights, flops = stack_work(cfg, runs, T - 1, window)
-                m = kes["layers"][1]["mixer"]
-                cache = 3 * window * (m["kv_rank"] + m["rot_dim"]) * 2          # three attention runs
-                cache += 3 * 2 * (2 * d * 16 * 4 + 2 * d * 3 * 4)                # three states, read and written
+            V = 32768
+            if name != "gptj":
+                weights, flops, cache = stack_work(cfg, runs, T - 1)
             else:
                 weights = 12 * d * d * len(runs)
                 flops = 2 * weights * (T - 1) + len(runs) * 2 * d * (T - 1) * T
@@ -731,16 +762,16 @@ def run_stack(args):
             row[name] = out
         sizes[str(d)] = row
     sampler.stop()
-    top = sizes[str(args.stack_widths.split(",")[-1])]["keselix"]
+    top = sizes[str(args.stack_widths.split(",")[-1])][names[0]]
     print(json.dumps({
-        "metric": "keselix_decode_tokens_per_s", "value": top["decode_b1"]["tokens_per_s"], "unit": UNIT, "n_gpus": 1,
+        "metric": names[0] + "_decode_tokens_per_s", "value": top["decode_b1"]["tokens_per_s"], "unit": UNIT, "n_gpus": 1,
         "steps": K, "warmup": W, "ms_per_step": top["decode_b1"]["ms_per_step"], "higher_is_better": True, "scaling": "strong",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "gpu_launches": launches,
         "clocks": sampler.summary(t_wall0, time.time()),
         "peaks": {"hbm_gbs": hbm, "bf16_tflops": tc, "source": "measured" if peaks else "fallback"},
-        "config": {"workload": "layer-stack model (state-space and latent-attention layers) beside GPT-J at equal width and "
-                               "number of layer runs; random weights; one 2048-token prompt, greedy decode",
-                   "l2": "every step reads more weights than L2 holds (looped layers twice)", "parallelism": "mp1"},
+        "config": {"workload": f"layer-stack model ({names[0]}) beside {names[1]} at equal width and number of layer runs; "
+                               "random weights; one 2048-token prompt, greedy decode",
+                   "l2": "every step reads more weights than L2 holds", "parallelism": "mp1"},
         "sizes": sizes}), flush=True)
 
 
@@ -755,8 +786,10 @@ def main():
                     help="6b: GPT-J-6B (the headline); 22b: the L48 d6144 h24 scale-up (fits 8 GPUs)")
     ap.add_argument("--workload", default="headline", choices=["headline", "serving", "stack"],
                     help="headline: full-window greedy decode; serving: 1024-token prompts + nucleus sampling; stack: a "
-                         "layer-stack model (Keselix) beside GPT-J at equal widths")
+                         "layer-stack model (--stack-model) beside the closest other one at equal widths")
     ap.add_argument("--stack-widths", default="2048,4096", help="widths of --workload stack")
+    ap.add_argument("--stack-model", default="keselix", choices=["keselix", "bavutar"],
+                    help="model of --workload stack: keselix (beside GPT-J) or bavutar (beside keselix)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--headline-only", action="store_true",
                     help="skip the eval 8 x 2048, serving batch-32 and (8 GPUs) 22B blocks of the JSON line")
