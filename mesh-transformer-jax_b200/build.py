@@ -21,7 +21,7 @@ FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std
 FAMILIES = {
     None: None,
     "stack": ("mtj_model", "mtj_stack", "mtj_stack_kernels", "mtj_latent_attn", "mtj_attn_tc_latent", "mtj_ssm", "mtj_gemm_tc",
-              "mtj_gemm_tc_stack", "mtj_gemm_tc_stack_post", "mtj_grouped_attn", "mtj_attn_tc_grouped", "mtj_matrix_state", "mtj_gemv", "mtj_misc", "mtj_sample", "mtj_loss", "mtj_family_stubs"),
+              "mtj_gemm_tc_stack", "mtj_gemm_tc_stack_post", "mtj_grouped_attn", "mtj_attn_tc_grouped", "mtj_matrix_state", "mtj_matrix_chunk", "mtj_gemv", "mtj_misc", "mtj_sample", "mtj_loss", "mtj_family_stubs"),
 }
 
 

@@ -5,8 +5,9 @@
 // blocks own column groups of a head and nothing is exchanged between them.  A sequence whose first row is in the call
 // starts from zeros whatever its slot holds; rows before the start (left padding) change nothing and give zeros.
 //
-// This file walks the rows one by one (decoding, short portions, 32-bit runs); mtj_matrix_chunk.cu takes long prompts
-// in chunks on the tensor cores.
+// This file walks the rows one by one: matrix_scan_kernel (short portions, 32-bit runs) and matrix_step_kernel (one row
+// per sequence: the state passes through registers once, 16 bytes a load); mtj_matrix_chunk.cu takes long prompts in
+// chunks on the tensor cores.
 #include <math.h>
 
 #include <algorithm>
@@ -200,6 +201,142 @@ cudaError_t scan_keys(const MatrixStateArgs& a, cudaStream_t s, bool pdl) {
   return scan<T, DELTA, 32>(a, s, pdl);
 }
 
+// ---- one row per sequence.  A block owns up to 128 columns of a head; a thread holds four neighbouring columns of
+// every RPP-th key, so a row of the state is read and written in whole lines.
+constexpr int kStepThreads = 256, kStepCols = 128;
+
+template <typename T, bool DELTA, int NI>
+__global__ void __launch_bounds__(kStepThreads) matrix_step_kernel(const MatrixStateArgs a, const GatedNormArgs nm, int norm) {
+  __shared__ float sk[kMatrixMaxDim], sq[kMatrixMaxDim], sg[DELTA ? kMatrixMaxDim : 1], su[kStepCols], sv[kStepCols];
+  __shared__ __align__(16) float part[4 * kStepThreads];
+  __shared__ float red[3][kStepThreads / 32];
+  const int head = blockIdx.x, c0 = blockIdx.y * kStepCols, cols = min(kStepCols, a.vdim - c0), m = blockIdx.z;
+  const int lpr = cols >> 2, rpp = kStepThreads / lpr, r = threadIdx.x / lpr, c4 = threadIdx.x % lpr * 4;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = threadIdx.x;
+  const int kh = head / (a.heads / a.key_heads);
+  const float A = a.A[head];
+  float bias = 0.f;
+  if (DELTA) bias = t < a.dim ? a.decay_b[head * a.dim + t] : 0.f;
+  else bias = a.decay_b[head];
+  // the state was written kernels ago: it does not wait for the predecessor
+  const MsSpan sp = ms_span(a, m);
+  float4* state = reinterpret_cast<float4*>(a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim + c0 + c4);
+  const int ld4 = a.vdim >> 2;
+  float4 S[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int n = r + i * rpp;
+    S[i] = r < rpp && n < a.dim && sp.start > 0 ? state[static_cast<size_t>(n) * ld4] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  const T* row = static_cast<const T*>(a.u) + static_cast<size_t>(m) * a.ld_u;
+  const float k = t < a.dim ? ms_ld(row, a.k0 + kh * a.dim + t) : 0.f, q = t < a.dim ? ms_ld(row, a.q0 + kh * a.dim + t) : 0.f;
+  if (t < cols) sv[t] = ms_ld(row, a.v0 + head * a.vdim + c0 + t);
+  float c_decay = 0.f, c_in = 0.f;                       // SSD: decay and step size; delta: update strength in c_in
+  if (DELTA) {
+    const float d = t < a.dim ? a.decay[static_cast<size_t>(m) * a.ld_decay + head * a.dim + t] + bias : 0.f;
+    c_in = MsFn<T>::sigmoid(a.beta[static_cast<size_t>(m) * a.ld_beta + head]);
+    const float ks = warp_sum(k * k), qs = warp_sum(q * q);
+    if (lane == 0) {
+      red[0][warp] = ks;
+      red[1][warp] = qs;
+    }
+    if (t < a.dim) sg[t] = MsFn<T>::exp(A * MsFn<T>::softplus(d));
+    __syncthreads();
+    float kt = 0.f, qt = 0.f;
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) {
+      kt += red[0][i];
+      qt += red[1][i];
+    }
+    if (t < a.dim) {
+      sk[t] = k / sqrtf(kt + kUnitEps);
+      sq[t] = q * a.q_scale / sqrtf(qt + kUnitEps);
+    }
+  } else {
+    c_in = MsFn<T>::softplus(a.decay[static_cast<size_t>(m) * a.ld_decay + head] + bias);
+    c_decay = MsFn<T>::exp(A * c_in);
+    if (t < a.dim) {
+      sk[t] = k;
+      sq[t] = q;
+    }
+  }
+  __syncthreads();
+  auto column = [&](int c) {                             // sum of the threads' partial results for column c
+    float v = 0.f;
+#pragma unroll 8
+    for (int i = 0; i < rpp; ++i) v += part[i * cols + c];
+    return v;
+  };
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (DELTA) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int n = r + i * rpp;
+      const float g = n < a.dim ? sg[n] : 0.f, kn = n < a.dim ? sk[n] : 0.f;
+      S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
+      acc.x = fmaf(S[i].x, kn, acc.x); acc.y = fmaf(S[i].y, kn, acc.y); acc.z = fmaf(S[i].z, kn, acc.z); acc.w = fmaf(S[i].w, kn, acc.w);
+    }
+    if (r < rpp) *reinterpret_cast<float4*>(&part[r * cols + c4]) = acc;
+    __syncthreads();
+    if (t < cols) su[t] = c_in * (sv[t] - column(t));
+  } else if (t < cols) {
+    su[t] = c_in * sv[t];
+  }
+  __syncthreads();
+  const float4 u = r < rpp ? *reinterpret_cast<const float4*>(&su[c4]) : make_float4(0.f, 0.f, 0.f, 0.f);
+  acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int n = r + i * rpp;
+    const float kn = n < a.dim ? sk[n] : 0.f, qn = n < a.dim ? sq[n] : 0.f;
+    float4 s = S[i];
+    if (!DELTA) { s.x *= c_decay; s.y *= c_decay; s.z *= c_decay; s.w *= c_decay; }
+    s.x = fmaf(kn, u.x, s.x); s.y = fmaf(kn, u.y, s.y); s.z = fmaf(kn, u.z, s.z); s.w = fmaf(kn, u.w, s.w);
+    acc.x = fmaf(s.x, qn, acc.x); acc.y = fmaf(s.y, qn, acc.y); acc.z = fmaf(s.z, qn, acc.z); acc.w = fmaf(s.w, qn, acc.w);
+    if (r < rpp && n < a.dim && sp.n > 0) state[static_cast<size_t>(n) * ld4] = s;
+  }
+  if (r < rpp) *reinterpret_cast<float4*>(&part[r * cols + c4]) = acc;
+  __syncthreads();
+  float y = 0.f;
+  if (t < cols) {
+    y = column(t);
+    if (!DELTA) y = fmaf(a.D[head], sv[t], y);
+    if (sp.n <= 0) y = 0.f;
+  }
+  if (DELTA && norm) {                                   // the block holds the whole head
+    const float s = warp_sum(y * y);
+    if (lane == 0) red[2][warp] = s;
+    __syncthreads();
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) ss += red[2][i];
+    if (t < cols) {
+      const int c = head * a.vdim + t;
+      y *= nm.w[t] / sqrtf(ss / static_cast<float>(a.vdim) + nm.eps);
+      y *= MsFn<T>::sigmoid(ms_ld(static_cast<const T*>(nm.gate), static_cast<size_t>(m) * nm.ld_gate + c));
+      const size_t o = static_cast<size_t>(m) * nm.ld_out + c;
+      if (nm.out) nm.out[o] = y;
+      if (nm.out_bf16) nm.out_bf16[o] = __float2bfloat16_rn(y);
+    }
+  } else if (t < cols) {
+    a.out[static_cast<size_t>(m) * a.ld_out + head * a.vdim + c0 + t] = y;
+  }
+}
+
+template <typename T, bool DELTA>
+cudaError_t step(const MatrixStateArgs& a, const GatedNormArgs* norm, cudaStream_t s, bool pdl) {
+  const dim3 grid(a.heads, (a.vdim + kStepCols - 1) / kStepCols, a.M);
+  const int rpp = kStepThreads / (std::min(a.vdim, kStepCols) / 4), ni = (a.dim + rpp - 1) / rpp;
+  const GatedNormArgs nm = norm ? *norm : GatedNormArgs{};
+  auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(kStepThreads), 0, s, pdl, a, nm, norm ? 1 : 0); };
+  if (ni <= 4) return go(matrix_step_kernel<T, DELTA, 4>);
+  if (ni <= 8) return go(matrix_step_kernel<T, DELTA, 8>);
+  if (ni <= 16) return go(matrix_step_kernel<T, DELTA, 16>);
+  return go(matrix_step_kernel<T, DELTA, 32>);
+}
+
 // ---- norm and gate of the outputs: one group of TH threads per (row, part)
 template <typename T, int TH>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormArgs a) {
@@ -265,6 +402,16 @@ cudaError_t launch_matrix_scan(const MatrixStateArgs& a, cudaStream_t s, bool pd
   if (!matrix_state_ok(a)) return cudaErrorInvalidValue;
   if (a.u_bf16) return a.delta ? scan_keys<__nv_bfloat16, true>(a, s, pdl) : scan_keys<__nv_bfloat16, false>(a, s, pdl);
   return a.delta ? scan_keys<float, true>(a, s, pdl) : scan_keys<float, false>(a, s, pdl);
+}
+
+bool matrix_step_ok(const MatrixStateArgs& a) { return a.rows.Tc == 1 && (a.vdim & 3) == 0 && a.M <= 65535; }
+bool matrix_step_norms(const MatrixStateArgs& a) { return matrix_step_ok(a) && a.delta && a.vdim <= kStepCols; }
+
+cudaError_t launch_matrix_step(const MatrixStateArgs& a, const GatedNormArgs* norm, cudaStream_t s, bool pdl) {
+  if (!matrix_state_ok(a) || !matrix_step_ok(a) || (norm && !matrix_step_norms(a))) return cudaErrorInvalidValue;
+  if (norm && (norm->gate_bf16 != 0) != (a.u_bf16 != 0)) return cudaErrorInvalidValue;
+  if (a.u_bf16) return a.delta ? step<__nv_bfloat16, true>(a, norm, s, pdl) : step<__nv_bfloat16, false>(a, norm, s, pdl);
+  return a.delta ? step<float, true>(a, norm, s, pdl) : step<float, false>(a, norm, s, pdl);
 }
 
 cudaError_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl) {

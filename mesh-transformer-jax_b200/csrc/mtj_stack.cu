@@ -19,6 +19,7 @@ int up8(int64_t v) { return static_cast<int>(align_up(v, 8)); }
 int up4(int v) { return (v + 3) & ~3; }
 constexpr int kAbsorbRows = 256;       // rows of the absorbed attention's scratch
 constexpr int kSelectGemvRows = 4;
+constexpr int kChunkedRows = 2 * kMatrixChunk;   // rows of a sequence from which matrix-state mixers work in chunks
 }  // namespace
 
 int32_t LayerStack::create(const mtj_config& cfg, const mtj_stack_desc& desc, int max_pos, LayerStack** out) {
@@ -226,7 +227,7 @@ void LayerStack::carve_workspace(Carver& c) {
   s_begin_ = c.base ? c.base + c.off : nullptr;
   rows_a_ = static_cast<int>(std::min<int64_t>(R, kAbsorbRows));
   int64_t p1 = 8, act = 8, u = 0, xp = 0, dtr = 0, xz = 0, qabs = 0, po = 0, ml = 0, qp = 0, cl = 0, kr = 0, kv = 0, hist = 0;
-  int64_t dtw = 0, gate = 0, aux = 0, mix = 0, qf = 0, gpo = 0, gml = 0, cnt = 0;
+  int64_t dtw = 0, gate = 0, aux = 0, mix = 0, qf = 0, gpo = 0, gml = 0, cnt = 0, rec = 0;
   for (const Layer& l : layers_) {
     const mtj_layer_desc& m = l.d;
     p1 = std::max<int64_t>(p1, up8(l.in.N));
@@ -251,6 +252,7 @@ void LayerStack::carve_workspace(Carver& c) {
       aux = std::max<int64_t>(aux, up8(l.aux));
       mix = std::max<int64_t>(mix, l.out.ld);
       if (l.dt.N) dtw = std::max<int64_t>(dtw, up8(l.dt.N));
+      if (m.mixer == MTJ_MIXER_MATRIX_STATE_DELTA) rec = std::max(rec, m.heads * matrix_chunk_record_bytes(m.dim));
       if (l.gate2.N) gate = std::max<int64_t>(gate, up8(l.gate2.N));
     } else {
       qabs = std::max<int64_t>(qabs, static_cast<int64_t>(m.heads) * l.row_ld);
@@ -302,6 +304,8 @@ void LayerStack::carve_workspace(Carver& c) {
     xp_planes_ = c.take<float>(xp_planes_elems_);
     act_bf_ = c.take<__nv_bfloat16>(R * act);
     gate_bf_ = c.take<__nv_bfloat16>(R * gate);
+    // sequences of at least kChunkedRows rows: their chunks, the last one of each may be partial
+    chunk_records_ = c.take<char>((R / kMatrixChunk + R / kChunkedRows + 1) * rec);
     q_pack_ = c.take<__nv_bfloat16>(R * qp);
     c_lin_ = c.take<__nv_bfloat16>(lin_rows_ * cl);
     kr_lin_ = c.take<__nv_bfloat16>(lin_rows_ * kr);
@@ -972,7 +976,8 @@ int32_t LayerStack::matrix(mtj_handle* h, const Run& r, int M, const RowMap& row
   a.state = r.ssm_state;
   a.out = mix_;
   a.ld_out = ld_mix_;
-  MTJ_CUDA(launch_matrix_scan(a, s, pdl));
+  a.chunk_records = chunk_records_;
+  a.dev_err = h->dev_err;
   GatedNormArgs g = {};
   g.M = M;
   g.parts = ssd ? m.norm_groups : m.heads;
@@ -989,8 +994,12 @@ int32_t LayerStack::matrix(mtj_handle* h, const Run& r, int M, const RowMap& row
   if (tc) g.out_bf16 = act_bf_;
   else g.out = act_;
   g.ld_out = l.out.ld;
-  MTJ_CUDA(launch_gated_norm(g, s, pdl));
-  h->launches += 2;
+  const bool step = matrix_step_ok(a), normed = step && matrix_step_norms(a);
+  if (step) MTJ_CUDA(launch_matrix_step(a, normed ? &g : nullptr, s, pdl));
+  else if (tc && rows.Tc >= kChunkedRows) MTJ_CUDA(launch_matrix_chunks(a, s));
+  else MTJ_CUDA(launch_matrix_scan(a, s, pdl));
+  if (!normed) MTJ_CUDA(launch_gated_norm(g, s, pdl));
+  h->launches += (normed ? 1 : 2) + (!ssd && tc && rows.Tc >= kChunkedRows ? 1 : 0);
   h->prof_end(s);
   h->prof_begin(MTJ_FAMILY_OUTPROJ, s);
   if (tc) MTJ_DO(gemm(h, kEpiPlain, l.out, act_bf_, M, y_, ld_, nullptr, 0, decode, s));

@@ -140,6 +140,7 @@ class LayerStack {
         *dt_raw_ = nullptr, *gate_raw_ = nullptr, *aux_ = nullptr, *mix_ = nullptr, *q_f32_ = nullptr, *act_ = nullptr, *xp_planes_ = nullptr, *q_abs_ = nullptr, *part_o_ = nullptr, *part_ml_ = nullptr;
   __nv_bfloat16 *xn_bf_ = nullptr, *cat_bf_ = nullptr, *xz_bf_ = nullptr, *u_bf_ = nullptr, *dtr_bf_ = nullptr, *act_bf_ = nullptr,
                 *sel_bf_ = nullptr, *q_pack_ = nullptr, *c_lin_ = nullptr, *kr_lin_ = nullptr, *kv_lin_ = nullptr, *gate_bf_ = nullptr;
+  char* chunk_records_ = nullptr;
   uint32_t *counters_ = nullptr, *attn_counters_ = nullptr;
   int ld_aux_ = 0, ld_mix_ = 0;
   std::map<std::tuple<const void*, int, int>, std::array<TensorMap, 3>> xmaps_;

@@ -158,6 +158,20 @@ int grouped_counters(int heads, int kv_heads);   // per row
 //   SSD    S <- exp(A dt) S + dt k v^T,  o = S^T q + D v, with dt = softplus(decay + decay_b) per head
 //   delta  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q, with unit k and q (q times q_scale),
 //          g = exp(A softplus(decay + decay_b)) per head and key channel, beta = sigmoid
+// the outputs' norm and gate: parts of part_n neighbouring columns, each by its own root mean square;
+// gate_first: RMSNorm(y * silu(gate)) * w[column], else RMSNorm(y) * w[column within the part] * sigmoid(gate)
+struct GatedNormArgs {
+  int M, parts, part_n, gate_first;
+  float eps;
+  const float* y;              // [M, ld_y]
+  int ld_y;
+  const void* gate;            // [M, ld_gate], fp32 or bf16
+  int gate_bf16, ld_gate;
+  const float* w;
+  float* out;                  // [M, ld_out] or null
+  __nv_bfloat16* out_bf16;
+  int ld_out;
+};
 struct MatrixStateArgs {
   int M, heads, key_heads, dim, vdim;
   int delta;
@@ -177,22 +191,19 @@ struct MatrixStateArgs {
   float* state;                // [slots][heads][dim][vdim]
   float* out;                  // [M, ld_out]
   int ld_out;
+  void* chunk_records;         // launch_matrix_chunks, delta: nseq * ceil(Tc / kMatrixChunk) * heads records, 16-byte aligned
+  uint32_t* dev_err;
 };
+// row by row
 cudaError_t launch_matrix_scan(const MatrixStateArgs& a, cudaStream_t s, bool pdl);
-// the outputs' norm and gate: parts of part_n neighbouring columns, each by its own root mean square;
-// gate_first: RMSNorm(y * silu(gate)) * w[column], else RMSNorm(y) * w[column within the part] * sigmoid(gate)
-struct GatedNormArgs {
-  int M, parts, part_n, gate_first;
-  float eps;
-  const float* y;              // [M, ld_y]
-  int ld_y;
-  const void* gate;            // [M, ld_gate], fp32 or bf16
-  int gate_bf16, ld_gate;
-  const float* w;
-  float* out;                  // [M, ld_out] or null
-  __nv_bfloat16* out_bf16;
-  int ld_out;
-};
+// one row per sequence; with `norm`, if matrix_step_norms(a), the norm and gate of the outputs too (out is not written)
+cudaError_t launch_matrix_step(const MatrixStateArgs& a, const GatedNormArgs* norm, cudaStream_t s, bool pdl);
+bool matrix_step_ok(const MatrixStateArgs& a);      // sizes that kernel takes
+bool matrix_step_norms(const MatrixStateArgs& a);
+// ---- mtj_matrix_chunk.cu: the same over long prompts, in chunks on the tensor cores (bf16 operands)
+constexpr int kMatrixChunk = 16;
+int64_t matrix_chunk_record_bytes(int dim);
+cudaError_t launch_matrix_chunks(const MatrixStateArgs& a, cudaStream_t s);
 cudaError_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl);
 constexpr int kMatrixMaxDim = 256;
 
