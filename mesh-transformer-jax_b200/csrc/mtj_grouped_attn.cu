@@ -21,6 +21,7 @@ namespace mtj {
 namespace {
 
 constexpr int kPrepThreads = 256;
+constexpr int kPiece = 16;        // keys per step of a warp; key ranges are multiples of it
 constexpr int kMaxSplits = 64;
 
 __device__ __forceinline__ void st(float* p, float v) { *p = v; }
@@ -120,15 +121,16 @@ __global__ void __launch_bounds__(kPrepThreads) grouped_prep_kernel(const Groupe
 
 // ---- what the row-at-a-time kernels share: the key range of a block and the end of a (row, key head)
 struct Range {
-  int seq, k0, k1;
+  int seq, k0, k1, lo;                // keys [max(k0, lo), k1)
 };
 __device__ __forceinline__ Range key_range(const GroupedAttnArgs& a, int m, int split) {
   Range r;
   const int p = own_pos(a.rows, a.pad, m, &r.seq);
   const int lo = max(0, p - a.window + 1), n = p - lo + 1;            // n <= 0: a padding row
-  const int per = ((max(n, 0) + a.splits - 1) / a.splits + 15) / 16 * 16;
-  r.k0 = lo + split * per;
+  const int first = lo / kPiece * kPiece, per = ((max(n, 0) + lo - first + a.splits - 1) / a.splits + kPiece - 1) / kPiece * kPiece;
+  r.k0 = first + split * per;                          // pieces lie inside one page
   r.k1 = min(r.k0 + per, p + 1);
+  r.lo = lo;
   return r;
 }
 __device__ __forceinline__ float ex2(float x) {
@@ -141,10 +143,10 @@ __device__ __forceinline__ float weight_of(float m, float ref) {      // exp of 
   return m == -INFINITY ? 0.f : BASE2 ? ex2(m - ref) : expf(m - ref);
 }
 
-// Adds the key ranges of `nh` query heads once the last block of them has arrived; all threads of every block call it
-// behind their stores to part_o / part_ml.  ws: at least kMaxSplits floats of shared memory.
+// Adds the key ranges of `nh` query heads once the last block of them has arrived, a warp per head; all threads of every
+// block call it behind their stores to part_o / part_ml.  ws: kMaxSplits floats of shared memory per warp.
 template <bool BASE2, int THREADS>
-__device__ __forceinline__ void finish_heads(const GroupedAttnArgs& a, int m, int h0, int nh, uint32_t* counter, float* ws) {
+__device__ __forceinline__ void finish_heads(const GroupedAttnArgs& a, int m, int h0, int nh, uint32_t* counter, float* ws_all) {
   __shared__ bool is_last;
   __threadfence();
   __syncthreads();
@@ -153,33 +155,54 @@ __device__ __forceinline__ void finish_heads(const GroupedAttnArgs& a, int m, in
   if (!is_last) return;
   __threadfence();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int h = h0; h < h0 + nh; ++h) {
+  float* ws = ws_all + warp * kMaxSplits;
+  for (int h = h0 + warp; h < h0 + nh; h += THREADS / 32) {
     const size_t base = (static_cast<size_t>(m) * a.heads + h) * a.splits;
-    if (warp == 0) {
-      const float* ml = a.part_ml + 2 * base;
-      float mx = -INFINITY, l = 0.f;
-      for (int s = lane; s < a.splits; s += 32) mx = fmaxf(mx, __ldcg(ml + 2 * s));
-      mx = warp_max(mx);
-      for (int s = lane; s < a.splits; s += 32) {
-        const float e = weight_of<BASE2>(__ldcg(ml + 2 * s), mx);
-        ws[s] = e;
-        l = fmaf(e, __ldcg(ml + 2 * s + 1), l);
-      }
-      l = warp_sum(l);
-      const float inv = l > 0.f ? 1.0f / l : 0.f;
-      for (int s = lane; s < a.splits; s += 32) ws[s] *= inv;
+    const float* ml = a.part_ml + 2 * base;
+    constexpr int kPer = kMaxSplits / 32;
+    float2 r[kPer];                                    // (maximum, denominator) of ranges lane, lane + 32
+    float mx = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int s = lane + 32 * i;
+      r[i] = s < a.splits ? make_float2(__ldcg(ml + 2 * s), __ldcg(ml + 2 * s + 1)) : make_float2(-INFINITY, 0.f);
+      mx = fmaxf(mx, r[i].x);
     }
-    __syncthreads();
+    mx = warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      r[i].x = weight_of<BASE2>(r[i].x, mx);
+      l = fmaf(r[i].x, r[i].y, l);
+    }
+    l = warp_sum(l);
+    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    __syncwarp();                                      // the last head's weights are read
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) ws[lane + 32 * i] = r[i].x * inv;
+    __syncwarp();
     const float* po = a.part_o + base * a.vdim;
-    for (int c = threadIdx.x; c < a.vdim; c += THREADS) {
-      float v = 0.f;
+    const size_t o = static_cast<size_t>(m) * a.ld_out + h * a.vdim;
+    if (((a.vdim | a.ld_out) & 3) == 0) {
+      for (int c = 4 * lane; c < a.vdim; c += 128) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-      for (int s = 0; s < a.splits; ++s) v = fmaf(ws[s], __ldcg(po + static_cast<size_t>(s) * a.vdim + c), v);
-      const size_t o = static_cast<size_t>(m) * a.ld_out + h * a.vdim + c;
-      if (a.out) a.out[o] = v;
-      if (a.out_bf16) a.out_bf16[o] = __float2bfloat16_rn(v);
+        for (int s = 0; s < a.splits; ++s) {
+          const float4 p = __ldcg(reinterpret_cast<const float4*>(po + static_cast<size_t>(s) * a.vdim + c));
+          const float e = ws[s];
+          v.x = fmaf(e, p.x, v.x); v.y = fmaf(e, p.y, v.y); v.z = fmaf(e, p.z, v.z); v.w = fmaf(e, p.w, v.w);
+        }
+        if (a.out) st4(a.out + o + c, v);
+        if (a.out_bf16) st4(a.out_bf16 + o + c, v);
+      }
+    } else {
+      for (int c = lane; c < a.vdim; c += 32) {
+        float v = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < a.splits; ++s) v = fmaf(ws[s], __ldcg(po + static_cast<size_t>(s) * a.vdim + c), v);
+        if (a.out) a.out[o + c] = v;
+        if (a.out_bf16) a.out_bf16[o + c] = __float2bfloat16_rn(v);
+      }
     }
-    __syncthreads();
   }
   if (threadIdx.x == 0) *counter = 0u;
 }
@@ -196,7 +219,7 @@ __host__ __device__ __forceinline__ int row_stride(int n) {        // floats; an
 template <typename T, int NC>
 __global__ void __launch_bounds__(32 * kHG) grouped_attn_kernel(const GroupedAttnArgs a) {
   extern __shared__ __align__(16) float ga_smem[];
-  __shared__ float ws[kMaxSplits];
+  __shared__ float ws[kMaxSplits * kHG];
   const int kst = row_stride(a.dim), vst = (a.vdim + 3) & ~3;
   float* qs = ga_smem;                     // [kHG][kst]
   float* ks = qs + kHG * kst;              // [kTK][kst]
@@ -218,7 +241,7 @@ __global__ void __launch_bounds__(32 * kHG) grouped_attn_kernel(const GroupedAtt
   for (int kt = r.k0; kt < r.k1; kt += kTK) {
     __syncthreads();
     for (int key = warp; key < kTK; key += kHG) {
-      const bool in = kt + key < r.k1;
+      const bool in = kt + key < r.k1 && kt + key >= r.lo;
       const size_t row = in ? cache_row(a.cache, r.seq, kt + key) : 0;
       const T* kp = static_cast<const T*>(a.cache.k) + row * a.cache.k_ld + g * kc;
       const T* vp = static_cast<const T*>(a.cache.v) + row * a.cache.v_ld + g * vc;
@@ -233,9 +256,9 @@ __global__ void __launch_bounds__(32 * kHG) grouped_attn_kernel(const GroupedAtt
       const float4 x = *reinterpret_cast<const float4*>(q + i), y = *reinterpret_cast<const float4*>(k + i);
       s = fmaf(x.x, y.x, s); s2 = fmaf(x.y, y.y, s2); s = fmaf(x.z, y.z, s); s2 = fmaf(x.w, y.w, s2);
     }
-    s = kt + lane < r.k1 ? s + s2 : -INFINITY;
-    const float m_new = fmaxf(mx, warp_max(s));                     // the tile holds at least one key
-    const float corr = expf(mx - m_new), w = expf(s - m_new);
+    s = kt + lane < r.k1 && kt + lane >= r.lo ? s + s2 : -INFINITY;
+    const float m_new = fmaxf(mx, warp_max(s));                     // -inf: no key of the tile is seen, nor any before
+    const float corr = weight_of<false>(mx, m_new), w = weight_of<false>(s, m_new);
     l = l * corr + warp_sum(w);
     mx = m_new;
 #pragma unroll
@@ -276,7 +299,6 @@ __global__ void __launch_bounds__(32 * kHG) grouped_attn_kernel(const GroupedAtt
 // ----------------------------------------------------------------------------------------- tensor cores
 constexpr int kWarps = 4;         // warps per block, each with key pieces of its own
 constexpr int kHM = 16;           // query heads per block (rows of the MMA)
-constexpr int kPiece = 16;        // keys per step of a warp
 constexpr int kStages = 3;        // pieces in a warp's ring
 
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
@@ -304,7 +326,7 @@ size_t mma_smem(int dim, int vdim) {
 template <int VT>
 __global__ void __launch_bounds__(32 * kWarps) grouped_attn_mma_kernel(const GroupedAttnArgs a) {
   extern __shared__ __align__(16) unsigned char gm_smem[];
-  __shared__ float ws[kMaxSplits];
+  __shared__ float ws[kMaxSplits * kWarps];
   __shared__ float2 wml[kWarps][kHM];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int kst = mma_ld(a.dim), vst = mma_ld(a.vdim), kd = kst - 8, vd = vst - 8;
@@ -324,21 +346,24 @@ __global__ void __launch_bounds__(32 * kWarps) grouped_attn_mma_kernel(const Gro
   pdl_launch_dependents();
   const Range r = key_range(a, m, split);
   const int n_pieces = r.k1 > r.k0 ? (r.k1 - r.k0 + kPiece - 1) / kPiece : 0;
-  const int kv8 = kc >> 3, vv8 = vc >> 3, all8 = kv8 + vv8;
+  // a lane copies the same 16 bytes of every kper-th key
+  const int kv8 = kc >> 3, vv8 = vc >> 3, kper = 32 / kv8, vper = 32 / vv8;
+  const int kkey = lane / kv8 < kper ? lane / kv8 : kPiece, vkey = lane / vv8 < vper ? lane / vv8 : kPiece;
+  const int kcol = lane % kv8 * 8, vcol = lane % vv8 * 8;
   auto fetch = [&](int piece, int slot) {
     if (piece < n_pieces) {
-      const int kt = r.k0 + piece * kPiece;
-      for (int i = lane; i < kPiece * all8; i += 32) {
-        const int key = i / all8, c = i % all8;
-        __nv_bfloat16* dst = c < kv8 ? ring + (slot * kPiece + key) * kst + c * 8 : vring + (slot * kPiece + key) * vst + (c - kv8) * 8;
-        if (kt + key < r.k1) {
-          const size_t row = cache_row(a.cache, r.seq, kt + key);
-          const __nv_bfloat16* src = c < kv8 ? static_cast<const __nv_bfloat16*>(a.cache.k) + row * a.cache.k_ld + g * kc + c * 8
-                                             : static_cast<const __nv_bfloat16*>(a.cache.v) + row * a.cache.v_ld + g * vc + (c - kv8) * 8;
-          cp16(smem_u32(dst), src);
-        } else {
-          *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
-        }
+      const int kt = r.k0 + piece * kPiece, n = r.k1 - kt;   // keys of the piece that exist: the rest is zero
+      const size_t row = cache_row(a.cache, r.seq, kt);
+      const __nv_bfloat16* ks = static_cast<const __nv_bfloat16*>(a.cache.k) + row * a.cache.k_ld + g * kc + kcol;
+      const __nv_bfloat16* vs = static_cast<const __nv_bfloat16*>(a.cache.v) + row * a.cache.v_ld + g * vc + vcol;
+      __nv_bfloat16 *kd2 = ring + slot * kPiece * kst + kcol, *vd2 = vring + slot * kPiece * vst + vcol;
+      for (int key = kkey; key < kPiece; key += kper) {
+        if (key < n) cp16(smem_u32(kd2 + key * kst), ks + key * a.cache.k_ld);
+        else *reinterpret_cast<uint4*>(kd2 + key * kst) = make_uint4(0u, 0u, 0u, 0u);
+      }
+      for (int key = vkey; key < kPiece; key += vper) {
+        if (key < n) cp16(smem_u32(vd2 + key * vst), vs + key * a.cache.v_ld);
+        else *reinterpret_cast<uint4*>(vd2 + key * vst) = make_uint4(0u, 0u, 0u, 0u);
       }
     }
     cp_commit();                                            // always, so that groups count pieces
@@ -380,20 +405,20 @@ __global__ void __launch_bounds__(32 * kWarps) grouped_attn_mma_kernel(const Gro
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           float& v = s[j][2 * h + e];
-          v = key0 + 8 * j + e < r.k1 ? v * c2 : -INFINITY;
+          v = key0 + 8 * j + e < r.k1 && key0 + 8 * j + e >= r.lo ? v * c2 : -INFINITY;
           t = fmaxf(t, v);
         }
       t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, 1));
       t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, 2));
-      const float m_new = fmaxf(mx[h], t);                   // the piece holds at least one key
-      corr[h] = ex2(mx[h] - m_new);
+      const float m_new = fmaxf(mx[h], t), ref = m_new == -INFINITY ? 0.f : m_new;      // -inf: no key is seen so far
+      corr[h] = ex2(mx[h] - ref);
       mx[h] = m_new;
       float sum = 0.f;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          s[j][2 * h + e] = ex2(s[j][2 * h + e] - m_new);
+          s[j][2 * h + e] = ex2(s[j][2 * h + e] - ref);
           sum += s[j][2 * h + e];
         }
       l[h] = l[h] * corr[h] + sum;
@@ -511,7 +536,18 @@ int grouped_counters(int heads, int kv_heads) { return kv_heads * ((heads / kv_h
 
 int grouped_attn_splits(int M, int heads, int kv_heads, int window) {
   const int groups = M * kv_heads * ((heads / kv_heads + kHM - 1) / kHM);
-  return std::max(1, std::min({kMaxSplits, (window + kPageTokens - 1) / kPageTokens, kGroupedBlocks / groups}));
+  const int most = std::max(1, std::min(kMaxSplits, (window + kPageTokens - 1) / kPageTokens));
+  // two blocks fit an SM: the fewest ranges whose last wave wastes little, merging counted as one more key in fifty
+  int best = 1;
+  double cost = 1e30;
+  for (int s = 1; s <= most && (s == 1 || static_cast<int64_t>(groups) * s <= kGroupedBlocks); ++s) {
+    const double c = ((static_cast<int64_t>(groups) * s + 295) / 296) * (1.0 / s + 0.02);
+    if (c < cost * 0.999) {
+      cost = c;
+      best = s;
+    }
+  }
+  return best;
 }
 
 cudaError_t launch_grouped_prep(const GroupedAttnArgs& a, cudaStream_t s, bool pdl) {

@@ -8,13 +8,15 @@
 // where the delta rule's G is per key channel.  Every decay is the product of per-row factors, none is divided by
 // another, so nothing overflows and rows that forget at once are exact.
 //
-// What does not depend on the state (delta: K~, the scaled queries and keys, T, the masked products) is computed for
-// all chunks at once by delta_prep_kernel and left as one record per (chunk, head) in the layout the scan reads.  In
-// the scan a warp owns 16 value columns of a head and keeps its S^T [16, keys] in fp32 accumulators, which are at the
-// same time the left operands of the next products; records come by bulk copies through a ring.  Operands that are not
-// exact in bf16 are split into two bf16 numbers (the second the rounding error of the first) and multiplied as hi.hi +
-// hi.lo + lo.hi with fp32 accumulation: about 16 mantissa bits, so the state keeps its 32-bit character.
-// (mma.sync: the M dimension is 16 columns of a state that must stay in registers between dependent products.)
+// What does not depend on the state is computed for all chunks at once and left as one record per (chunk, head) in the
+// layout the scan reads: delta_prep_kernel (K~, the scaled queries and keys, T, the masked products q.k) and
+// ssd_prep_kernel (the masked products C.B and the rows' decays).  In the scans two warps share 16 value columns of a
+// head, each keeping the S^T [16, keys / 2] of half the keys in fp32 accumulators, which are at the same time the left
+// operands of the next products; they add their partial sums through shared memory, once a chunk.  Records and rows
+// come through rings.  Operands that are not exact in bf16 are split into two bf16 numbers (the second the rounding error
+// of the first) and multiplied as hi.hi + hi.lo + lo.hi with fp32 accumulation: about 16 mantissa bits, so the state
+// keeps its 32-bit character.  (mma.sync: the M dimension is 16 columns of a state that must stay in registers between
+// dependent products.)
 #include <math.h>
 
 #include <algorithm>
@@ -63,46 +65,54 @@ __device__ __forceinline__ void zero_front(const MatrixStateArgs& a, const MsSpa
   }
 }
 
-// S^T of 16 columns: tile n holds keys 8 n .. 8 n + 7
-template <int DP>
-__device__ __forceinline__ void load_state(const MatrixStateArgs& a, const float* state, int col, int lane, bool have, float (*S)[4]) {
+// S^T of 16 columns and NT * 8 keys from key0 on: tile n holds keys key0 + 8 n .. + 7
+template <int NT>
+__device__ __forceinline__ void load_state(const MatrixStateArgs& a, const float* state, int key0, int col, int lane, bool have, float (*S)[4]) {
 #pragma unroll
-  for (int n = 0; n < DP / 8; ++n)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int key = 8 * n + (lane & 3) * 2 + (e & 1), c = col + (lane >> 2) + (e >> 1) * 8;
+      const int key = key0 + 8 * n + (lane & 3) * 2 + (e & 1), c = col + (lane >> 2) + (e >> 1) * 8;
       S[n][e] = have && key < a.dim && c < a.vdim ? state[static_cast<size_t>(key) * a.vdim + c] : 0.f;
     }
 }
-template <int DP>
-__device__ __forceinline__ void store_state(const MatrixStateArgs& a, float* state, int col, int lane, const float (*S)[4]) {
+template <int NT>
+__device__ __forceinline__ void store_state(const MatrixStateArgs& a, float* state, int key0, int col, int lane, const float (*S)[4]) {
 #pragma unroll
-  for (int n = 0; n < DP / 8; ++n)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int key = 8 * n + (lane & 3) * 2 + (e & 1), c = col + (lane >> 2) + (e >> 1) * 8;
+      const int key = key0 + 8 * n + (lane & 3) * 2 + (e & 1), c = col + (lane >> 2) + (e >> 1) * 8;
       if (key < a.dim && c < a.vdim) state[static_cast<size_t>(key) * a.vdim + c] = S[n][e];
     }
 }
-// The values of this lane's accumulator places: rows (lane & 3) * 2 + {0, 1} (+ 8), columns lane / 4 (+ 8) of a chunk, as
-// packed bf16 pairs of neighbouring rows: v[0], v[1] = columns lane / 4 and + 8 of rows 0 .. 7, v[2], v[3] of rows 8 .. 15.
-__device__ __forceinline__ void load_values(const __nv_bfloat16* v, int ld, int nt, int cols_left, int lane, uint32_t* out) {
+// The values of this lane's accumulator places -- rows (lane & 3) * 2 + {0, 1} (+ 8), columns lane / 4 (+ 8) of a chunk --
+// as loaded, one chunk ahead.  Rows past the end repeat the last one and columns past the head's the last one: their
+// weights are zero, their results are not stored.
+struct Values {
+  unsigned short r[4][2];            // [columns lane / 4 and + 8 of rows 0 .. 7, then of rows 8 .. 15][row of the pair]
+  __device__ __forceinline__ void load(const __nv_bfloat16* v, int ld, int nt, int cols_left, int lane) {
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int t = (lane & 3) * 2 + (i >> 1) * 8, c = (lane >> 2) + (i & 1) * 8;
-    const unsigned short* p = reinterpret_cast<const unsigned short*>(v) + static_cast<size_t>(t) * ld + c;
-    const uint32_t x = c < cols_left && t < nt ? *p : 0u, y = c < cols_left && t + 1 < nt ? p[ld] : 0u;
-    out[i] = x | (y << 16);
-  }
-}
-__device__ __forceinline__ void store_outputs(float* out, int ld, int nt, int cols_left, int lane, const float (*o)[4]) {
-#pragma unroll
-  for (int t8 = 0; t8 < 2; ++t8)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int t = (lane & 3) * 2 + (e & 1) + t8 * 8, c = (lane >> 2) + (e >> 1) * 8;
-      if (t < nt && c < cols_left) out[static_cast<size_t>(t) * ld + c] = o[t8][e];
+    for (int i = 0; i < 4; ++i) {
+      const int t = (lane & 3) * 2 + (i >> 1) * 8, c = max(0, min((lane >> 2) + (i & 1) * 8, cols_left - 1));
+      const unsigned short* p = reinterpret_cast<const unsigned short*>(v) + c;
+      r[i][0] = p[min(t, nt - 1) * ld];
+      r[i][1] = p[min(t + 1, nt - 1) * ld];
     }
+  }
+  __device__ __forceinline__ void pack(uint32_t* out) const {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) out[i] = r[i][0] | (static_cast<uint32_t>(r[i][1]) << 16);
+  }
+};
+__device__ __forceinline__ void pair_sync(int id) { asm volatile("bar.sync %0, 64;" ::"r"(id) : "memory"); }
+// one 8-row tile of outputs
+__device__ __forceinline__ void store_tile(float* out, int ld, int t0, int nt, int cols_left, int lane, const float* o) {
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const int t = t0 + (lane & 3) * 2 + (e & 1), c = (lane >> 2) + (e >> 1) * 8;
+    if (t < nt && c < cols_left) out[t * ld + c] = o[e];
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ delta rule
@@ -116,10 +126,14 @@ struct Record {                      // of one (chunk, head); byte offsets
 
 template <int DP>
 struct PrepSmem {
-  float k[kC][DP + 1], q[kC][DP + 1], g[kC][DP + 1];
+  float k[kC][DP], q[kC][DP], g[kC][DP];
   float L[kC][kC + 4], M[kC][kC + 4];                 // products, rows i, columns j
   float beta[kC];
 };
+
+__device__ __forceinline__ float dot4(const float4& x, const float4& y, float s) {
+  return fmaf(x.w, y.w, fmaf(x.z, y.z, fmaf(x.y, y.y, fmaf(x.x, y.x, s))));
+}
 
 // One block of 4 warps per (chunk, head).
 template <int DP>
@@ -164,49 +178,73 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const MatrixStateArgs a
     }
     if (lane == 0) sm.beta[t] = t < nt ? MsFn<__nv_bfloat16>::sigmoid(a.beta[m * a.ld_beta + head]) : 0.f;
   }
-  for (int i = threadIdx.x; i < kC * kC; i += 128) {
-    if (i / kC < i % kC) sm.M[i / kC][i % kC] = 0.f;
-    if (i / kC <= i % kC) sm.L[i / kC][i % kC] = 0.f;
-  }
   __syncthreads();
-  // L_ij and M_ij for i = j .. 15, lanes over the key channels; a warp takes columns j of a balanced total length
+  // L_ij and M_ij, lanes over the key channels (four neighbours each); a warp takes columns j of a balanced total
+  // length and walks the rows in fours, whose eight sums are brought together by a transposing reduction
+  constexpr int N4 = (DP + 127) / 128;
 #pragma unroll 1
   for (int s = 0; s < 4; ++s) {
     const int j = s == 0 ? warp : s == 1 ? 15 - warp : s == 2 ? 4 + warp : 11 - warp;
-    float d[NC], mine_l = 0.f, mine_m = 0.f;
+    float4 d[N4];
 #pragma unroll
-    for (int c = 0; c < NC; ++c) d[c] = sm.k[j][c * 32 + lane];
-#pragma unroll 2
-    for (int i = j; i < kC; ++i) {
-      float l = 0.f, m = 0.f;
+    for (int c = 0; c < N4; ++c)
+      d[c] = c * 128 + 4 * lane < DP ? *reinterpret_cast<const float4*>(&sm.k[j][c * 128 + 4 * lane]) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 1
+    for (int i0 = 0; i0 < kC; i0 += 4) {
+      float v[8];                                     // L of four rows, then M
 #pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        const int n = c * 32 + lane;
-        if (i > j) d[c] *= sm.g[i][n];
-        l = fmaf(sm.k[i][n], d[c], l);
-        m = fmaf(sm.q[i][n], d[c], m);
+      for (int r = 0; r < 4; ++r) {
+        const int i = i0 + r;
+        v[r] = v[4 + r] = 0.f;
+        if (i >= j) {
+#pragma unroll
+          for (int c = 0; c < N4; ++c) {
+            const int n = c * 128 + 4 * lane;
+            if (n < DP) {
+              if (i > j) {
+                const float4 g = *reinterpret_cast<const float4*>(&sm.g[i][n]);
+                d[c].x *= g.x; d[c].y *= g.y; d[c].z *= g.z; d[c].w *= g.w;
+                v[r] = dot4(*reinterpret_cast<const float4*>(&sm.k[i][n]), d[c], v[r]);
+              }
+              v[4 + r] = dot4(*reinterpret_cast<const float4*>(&sm.q[i][n]), d[c], v[4 + r]);
+            }
+          }
+        }
       }
-      // both sums at once: the lower half of the warp goes on with l, the upper with m
-      const float send = lane < 16 ? m : l, keep = lane < 16 ? l : m;
-      float v = keep + __shfl_xor_sync(0xffffffffu, send, 16);
+      if (i0 + 3 >= j) {
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-      if ((lane & 15) == i) mine_l = v;               // lane i keeps l, lane 16 + i keeps m
-    }
-    mine_m = __shfl_down_sync(0xffffffffu, mine_l, 16);
-    if (lane < 16 && lane >= j) {
-      if (lane > j) sm.L[lane][j] = mine_l;
-      sm.M[lane][j] = mine_m;
+        for (int w = 4; w > 0; w >>= 1) {             // lane bits 16, 8, 4 pick one of the eight
+          const bool up = lane & (4 * w);
+#pragma unroll
+          for (int r = 0; r < w; ++r) {
+            const float send = up ? v[r] : v[r + w], keep = up ? v[r + w] : v[r];
+            v[r] = keep + __shfl_xor_sync(0xffffffffu, send, 4 * w);
+          }
+        }
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], 2);
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+      }
+      if ((lane & 3) == 0) {
+        const int which = lane >> 2, i = i0 + (which & 3);
+        (which < 4 ? sm.L : sm.M)[i][j] = v[0];       // zero above the diagonal, L zero on it too
+      }
     }
   }
   __syncthreads();
   unsigned char* rec = static_cast<unsigned char*>(a.chunk_records) +
                        ((static_cast<size_t>(blockIdx.z) * gridDim.x + chunk) * a.heads + head) * Rec::kBytes;
-  auto put = [&](int at, int bytes, int row, int ld, int col, float x, float y) {
+  auto put2 = [&](int at, int row, int col, float x, float y) {
     uint32_t hi, lo;
     split2(x, y, hi, lo);
-    *reinterpret_cast<uint32_t*>(rec + at + (row * ld + col) * 2) = hi;
-    *reinterpret_cast<uint32_t*>(rec + at + bytes + (row * ld + col) * 2) = lo;
+    *reinterpret_cast<uint32_t*>(rec + at + (row * kSq + col) * 2) = hi;
+    *reinterpret_cast<uint32_t*>(rec + at + Rec::kSmall + (row * kSq + col) * 2) = lo;
+  };
+  auto put4 = [&](int at, int row, int col, const float4& v) {
+    uint2 hi, lo;
+    split2(v.x, v.y, hi.x, lo.x);
+    split2(v.z, v.w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(rec + at + (row * Rec::LD + col) * 2) = hi;
+    *reinterpret_cast<uint2*>(rec + at + Rec::kMat + (row * Rec::LD + col) * 2) = lo;
   };
   if (warp == 3) {
     // T column by column: lane c < 16 solves for column c
@@ -223,33 +261,34 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const MatrixStateArgs a
 #pragma unroll
     for (int i = 0; i < kC; ++i) {
       const float other = __shfl_down_sync(0xffffffffu, T[i], 1);
-      if (lane < 16 && !(lane & 1)) put(Rec::kT, Rec::kSmall, i, kSq, c, T[i], other);
+      if (lane < 16 && !(lane & 1)) put2(Rec::kT, i, c, T[i], other);
     }
     for (int i = lane; i < kC * kC / 2; i += 32) {
       const int r = i / (kC / 2), cc = i % (kC / 2) * 2;
-      put(Rec::kM, Rec::kSmall, r, kSq, cc, sm.M[r][cc], sm.M[r][cc + 1]);
+      put2(Rec::kM, r, cc, sm.M[r][cc], sm.M[r][cc + 1]);
     }
+    return;
   }
-  // scaled keys and queries: jobs of two neighbouring channels, prefix products (K~, Q~, the whole chunk's decay) or
-  // suffix products (keys for the new state)
-  for (int job = threadIdx.x; job < DP; job += 128) {
-    const int n = job % (DP / 2) * 2;
-    float px = 1.0f, py = 1.0f;
-    if (job < DP / 2) {
+  // warp 0: K~ and the whole chunk's decay, warp 1: the scaled queries (prefix products), warp 2: the keys for the new
+  // state (suffix products)
+#pragma unroll
+  for (int c = 0; c < N4; ++c) {
+    const int n = c * 128 + 4 * lane;
+    if (n >= DP) continue;
+    float4 p = make_float4(1.f, 1.f, 1.f, 1.f);
+    auto times = [&](const float4& x) { return make_float4(x.x * p.x, x.y * p.y, x.z * p.z, x.w * p.w); };
+    if (warp < 2) {
 #pragma unroll
       for (int i = 0; i < kC; ++i) {
-        px *= sm.g[i][n];
-        py *= sm.g[i][n + 1];
-        put(Rec::kKt, Rec::kMat, i, Rec::LD, n, sm.k[i][n] * px, sm.k[i][n + 1] * py);
-        put(Rec::kQt, Rec::kMat, i, Rec::LD, n, sm.q[i][n] * px, sm.q[i][n + 1] * py);
+        p = times(*reinterpret_cast<const float4*>(&sm.g[i][n]));
+        put4(warp ? Rec::kQt : Rec::kKt, i, n, times(*reinterpret_cast<const float4*>(warp ? &sm.q[i][n] : &sm.k[i][n])));
       }
-      *reinterpret_cast<float2*>(rec + Rec::kE + n * 4) = make_float2(px, py);
+      if (warp == 0) *reinterpret_cast<float4*>(rec + Rec::kE + n * 4) = p;
     } else {
 #pragma unroll
       for (int i = kC - 1; i >= 0; --i) {
-        put(Rec::kKh, Rec::kMat, i, Rec::LD, n, sm.k[i][n] * px, sm.k[i][n + 1] * py);
-        px *= sm.g[i][n];
-        py *= sm.g[i][n + 1];
+        put4(Rec::kKh, i, n, times(*reinterpret_cast<const float4*>(&sm.k[i][n])));
+        p = times(*reinterpret_cast<const float4*>(&sm.g[i][n]));
       }
     }
   }
@@ -264,11 +303,13 @@ __device__ __forceinline__ void arrive(uint32_t bar) { asm volatile("mbarrier.ar
 
 constexpr int kRing = 3;
 
-// One block = (head, 16 NW columns, sequence): NW scan warps and one that fetches records.
-template <int DP, int NW>
-__global__ void __launch_bounds__(32 * (NW + 1)) delta_chunk_kernel(const MatrixStateArgs a, int chunks_max) {
+// One block = (head, 16 NG columns, sequence): two scan warps per 16 columns and one that fetches records.
+template <int DP, int NG>
+__global__ void __launch_bounds__(32 * (2 * NG + 1)) delta_chunk_kernel(const MatrixStateArgs a, int chunks_max) {
   using Rec = Record<DP>;
+  constexpr int NW = 2 * NG, NT = DP / 16;               // warps; 8-key tiles per warp
   extern __shared__ __align__(128) unsigned char dc_smem[];
+  __shared__ __align__(16) float4 swap[2][NW][3][32];     // partial sums for the partner, two chunks in turn
   __shared__ __align__(8) uint64_t bars[2 * kRing];
   __shared__ uint32_t failed;
   const int head = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -283,7 +324,7 @@ __global__ void __launch_bounds__(32 * (NW + 1)) delta_chunk_kernel(const Matrix
   }
   __syncthreads();
   const MsSpan sp = ms_span(a, blockIdx.z);
-  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NW;
+  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NG;
   if (warp == NW) {
     if (lane == 0) {
       const unsigned char* rec = static_cast<const unsigned char*>(a.chunk_records) +
@@ -302,28 +343,27 @@ __global__ void __launch_bounds__(32 * (NW + 1)) delta_chunk_kernel(const Matrix
       for (int k = max(0, issued - kRing); k < issued; ++k) mbar_wait(full + 8 * (k % kRing), (k / kRing) & 1);   // no copy outlives the block
     }
   } else {
-    const int col = c0 + warp * 16, left = a.vdim - col;
+    const int grp = warp >> 1, half = warp & 1, col = c0 + grp * 16, left = a.vdim - col, key0 = half * (DP / 2);
     float* state = a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim;
-    float S[DP / 8][4];
-    load_state<DP>(a, state, col, lane, sp.start > 0 && sp.n > 0, S);
-    zero_front(a, sp, blockIdx.z, head, c0, 16 * NW, 32 * NW);
-    const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u + a.v0 + head * a.vdim + col;
+    float S[NT][4];
+    load_state<NT>(a, state, key0, col, lane, sp.start > 0 && sp.n > 0, S);
+    zero_front(a, sp, blockIdx.z, head, c0, 16 * NG, 32 * NW);
+    const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u + a.v0 + head * a.vdim + min(col, a.vdim - 1);
     float* out = a.out + static_cast<size_t>(sp.row0) * a.ld_out + head * a.vdim + col;
-    uint32_t vals[4] = {0u, 0u, 0u, 0u};
-    if (chunks > 0) load_values(v, a.ld_u, min(kC, sp.n), left, lane, vals);
-    const int on = rows_as_n(lane, Rec::LD) * 2, ot = rows_as_m(lane, Rec::LD) * 2, os = rows_as_n(lane, kSq) * 2;
-    bool ok = true;
-    for (int k = 0; k < chunks && ok; ++k) {
+    Values vals;
+    if (chunks > 0) vals.load(v, a.ld_u, min(kC, sp.n), left, lane);
+    const int on = (rows_as_n(lane, Rec::LD) + key0) * 2, ot = (rows_as_m(lane, Rec::LD) + key0) * 2, os = rows_as_n(lane, kSq) * 2;
+    bool ok = true;                                      // a wait that runs out is remembered; the pair barriers go on
+    for (int k = 0; k < chunks; ++k) {
       const int s = k % kRing, nt = min(kC, sp.n - k * kC);
-      ok = mbar_wait(full + 8 * s, (k / kRing) & 1);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
+      if (ok) ok = mbar_wait(full + 8 * s, (k / kRing) & 1);
       const uint32_t r = base + s * Rec::kBytes;
-      uint32_t cur[4] = {vals[0], vals[1], vals[2], vals[3]};
-      if (k + 1 < chunks) load_values(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, sp.n - (k + 1) * kC, left, lane, vals);
+      uint32_t cur[4];
+      vals.pack(cur);
+      if (k + 1 < chunks) vals.load(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, min(kC, sp.n - (k + 1) * kC), left, lane);
       float R[3][2][4] = {}, O[3][2][4] = {};            // the three products of the split operands
 #pragma unroll
-      for (int ks = 0; ks < DP / 16; ++ks) {
+      for (int ks = 0; ks < NT / 2; ++ks) {
         uint32_t hi[4], lo[4], bh[4], bl[4];
         split_a(S[2 * ks], S[2 * ks + 1], hi, lo);
         ldsm4(bh, r + Rec::kKt + on + 32 * ks);
@@ -343,15 +383,31 @@ __global__ void __launch_bounds__(32 * (NW + 1)) delta_chunk_kernel(const Matrix
           mma(O[2][t], lo, bh + 2 * t);
         }
       }
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          R[0][t][e] += R[1][t][e] + R[2][t][e];
+          O[0][t][e] += O[1][t][e] + O[2][t][e];
+        }
+      // the other half of the keys: both warps need all of R, of the outputs each finishes the tile `half`
+      float4* mine = swap[k & 1][warp][0] + lane;
+      const float4* theirs = swap[k & 1][warp ^ 1][0] + lane;
+      mine[0] = make_float4(R[0][0][0], R[0][0][1], R[0][0][2], R[0][0][3]);
+      mine[32] = make_float4(R[0][1][0], R[0][1][1], R[0][1][2], R[0][1][3]);
+      mine[64] = half ? make_float4(O[0][0][0], O[0][0][1], O[0][0][2], O[0][0][3]) : make_float4(O[0][1][0], O[0][1][1], O[0][1][2], O[0][1][3]);
+      pair_sync(1 + grp);
       uint32_t hi[4], lo[4], bh[4], bl[4];
+      const float4 r0 = theirs[0], r1 = theirs[32], po = theirs[64];
       {
         float X[2][4];                                   // V - K~ S0, transposed
+        const float rt[2][4] = {{r0.x, r0.y, r0.z, r0.w}, {r1.x, r1.y, r1.z, r1.w}};
 #pragma unroll
         for (int t = 0; t < 2; ++t)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const uint32_t p = cur[2 * t + (e >> 1)];
-            X[t][e] = ((e & 1) ? bf16_hi(p) : bf16_lo(p)) - (R[0][t][e] + (R[1][t][e] + R[2][t][e]));
+            X[t][e] = ((e & 1) ? bf16_hi(p) : bf16_lo(p)) - (R[0][t][e] + rt[t][e]);
           }
         split_a(X[0], X[1], hi, lo);
       }
@@ -370,36 +426,39 @@ __global__ void __launch_bounds__(32 * (NW + 1)) delta_chunk_kernel(const Matrix
         for (int e = 0; e < 4; ++e) U[0][t][e] += U[1][t][e] + U[2][t][e];
       split_a(U[0][0], U[0][1], hi, lo);
 #pragma unroll
-      for (int p = 0; p < DP / 16; ++p) {                // the new state
+      for (int p = 0; p < NT / 2; ++p) {                 // the new state
         ldsm4t(bh, r + Rec::kKh + ot + 32 * p);
         ldsm4t(bl, r + Rec::kKh + Rec::kMat + ot + 32 * p);
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           float* st = S[2 * p + t];
           float ex, ey;
-          asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(ex), "=f"(ey) : "r"(r + Rec::kE + (8 * (2 * p + t) + (lane & 3) * 2) * 4) : "memory");
+          asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(ex), "=f"(ey) : "r"(r + Rec::kE + (key0 + 8 * (2 * p + t) + (lane & 3) * 2) * 4) : "memory");
           st[0] *= ex; st[1] *= ey; st[2] *= ex; st[3] *= ey;
-          mma(st, hi, bh + 2 * t);
-          mma(st, hi, bl + 2 * t);
-          mma(st, lo, bh + 2 * t);
+        }
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma(S[2 * p + t], hi, bh + 2 * t);
+          mma(S[2 * p + t], hi, bl + 2 * t);
+          mma(S[2 * p + t], lo, bh + 2 * t);
         }
       }
       ldsm4(bh, r + Rec::kM + os);
       ldsm4(bl, r + Rec::kM + Rec::kSmall + os);
       __syncwarp();
       if (lane == 0) arrive(empty + 8 * s);              // the record is read
+      float y[4];
 #pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        mma(O[0][t], hi, bh + 2 * t);
-        mma(O[1][t], hi, bl + 2 * t);
-        mma(O[2][t], lo, bh + 2 * t);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) O[0][t][e] += O[1][t][e] + O[2][t][e];
-      }
-      store_outputs(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, nt, left, lane, O[0]);
+      for (int e = 0; e < 4; ++e) y[e] = half ? O[0][1][e] : O[0][0][e];
+      y[0] += po.x; y[1] += po.y; y[2] += po.z; y[3] += po.w;
+      const uint32_t mh[2] = {half ? bh[2] : bh[0], half ? bh[3] : bh[1]}, ml[2] = {half ? bl[2] : bl[0], half ? bl[3] : bl[1]};
+      mma(y, hi, mh);
+      mma(y, hi, ml);
+      mma(y, lo, mh);
+      store_tile(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, half * 8, nt, left, lane, y);
     }
-    if (!ok && lane == 0) atomicOr(&failed, 1u);
-    if (sp.n > 0 && ok) store_state<DP>(a, state, col, lane, S);
+    if (!ok) atomicOr(&failed, 1u);
+    if (sp.n > 0 && __all_sync(0xffffffffu, ok)) store_state<NT>(a, state, key0, col, lane, S);
   }
   __syncthreads();
   if (threadIdx.x == 0 && failed && a.dev_err) atomicOr(a.dev_err, kDevErrTimeout);
@@ -413,150 +472,230 @@ __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_grou
 template <int N>
 __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <int DP, int NW>
-__global__ void __launch_bounds__(32 * NW) ssd_chunk_kernel(const MatrixStateArgs a) {
-  constexpr int LD = DP + 8, kTile = kC * LD, kThreads = 32 * NW;
-  extern __shared__ __align__(16) __nv_bfloat16 sd_smem[];             // [kRing][B | C][kC][LD]
-  const int head = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const MsSpan sp = ms_span(a, blockIdx.z);
-  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NW, col = c0 + warp * 16, left = a.vdim - col;
-  const int kh = head / (a.heads / a.key_heads);
-  const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u;
-  const int kb = a.k0 + kh * a.dim, qb = a.q0 + kh * a.dim;
-  const bool vec = ((a.dim | kb | qb | a.ld_u) & 7) == 0;
-  for (int i = threadIdx.x; i < kRing * 2 * kTile / 8; i += kThreads) reinterpret_cast<uint4*>(sd_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
-  __syncthreads();
-  auto fetch = [&](int k) {
-    if (k < chunks) {
-      __nv_bfloat16* dst = sd_smem + (k % kRing) * 2 * kTile;
-      const int nt = min(kC, sp.n - k * kC);
-      const __nv_bfloat16* src = u + static_cast<size_t>(k) * kC * a.ld_u;
-      if (vec) {
-        const int per = a.dim >> 3;
-        for (int i = threadIdx.x; i < 2 * kC * per; i += kThreads) {
-          const int which = i / (kC * per), t = i / per % kC, c = i % per * 8;
-          __nv_bfloat16* d = dst + which * kTile + t * LD + c;
-          if (t < nt) cp16(smem_u32(d), src + static_cast<size_t>(t) * a.ld_u + (which ? qb : kb) + c);
-          else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
-        }
-      } else {
-        for (int i = threadIdx.x; i < 2 * kC * a.dim; i += kThreads) {
-          const int which = i / (kC * a.dim), t = i / a.dim % kC, c = i % a.dim;
-          dst[which * kTile + t * LD + c] = t < nt ? src[static_cast<size_t>(t) * a.ld_u + (which ? qb : kb) + c] : __float2bfloat16_rn(0.f);
-        }
-      }
+struct SsdRecord {                   // of one (chunk, head); byte offsets
+  static constexpr int kSmall = kC * kSq * 2;          // masked products [i][j], hi then lo
+  static constexpr int kG = 2 * kSmall;                // floats: e^(G_i) [16], e^(G_C - G_j) dt_j [16], e^(G_C)
+  static constexpr int kBytes = kG + 4 * 36;
+};
+static_assert(SsdRecord::kBytes % 16 == 0, "whole pieces");
+
+// 16 rows of `dim` columns -> [kC][LD] in shared memory by `threads` threads; rows from nt on are zero
+__device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int LD, const __nv_bfloat16* src, int ld, int dim, int nt, bool vec, int t, int threads) {
+  if (vec) {
+    const int per = dim >> 3;
+    for (int i = t; i < kC * per; i += threads) {
+      const int row = i / per, c = i % per * 8;
+      __nv_bfloat16* d = dst + row * LD + c;
+      if (row < nt) cp16(smem_u32(d), src + static_cast<size_t>(row) * ld + c);
+      else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
     }
-    cp_commit();                                         // always, so that groups count chunks
-  };
-  fetch(0);
-  fetch(1);
-  const float A = a.A[head], D = a.D[head], bias = a.decay_b[head];
-  float* state = a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim;
-  float S[DP / 8][4];
-  load_state<DP>(a, state, col, lane, sp.start > 0 && sp.n > 0, S);
-  zero_front(a, sp, blockIdx.z, head, c0, 16 * NW, kThreads);
-  const __nv_bfloat16* v = u + a.v0 + head * a.vdim + col;
-  float* out = a.out + static_cast<size_t>(sp.row0) * a.ld_out + head * a.vdim + col;
-  const float* raw = a.decay + static_cast<size_t>(sp.row0) * a.ld_decay + head;
-  uint32_t vals[4] = {0u, 0u, 0u, 0u};
-  float dt_raw = 0.f;
-  if (chunks > 0) {
-    load_values(v, a.ld_u, min(kC, sp.n), left, lane, vals);
-    if ((lane & 15) < sp.n) dt_raw = raw[static_cast<size_t>(lane & 15) * a.ld_decay];
+  } else {
+    for (int i = t; i < kC * dim; i += threads) {
+      const int row = i / dim, c = i % dim;
+      dst[row * LD + c] = row < nt ? src[static_cast<size_t>(row) * ld + c] : __float2bfloat16_rn(0.f);
+    }
   }
-  const int on = rows_as_n(lane, LD) * 2, om = rows_as_m(lane, LD) * 2;
-  for (int k = 0; k < chunks; ++k) {
-    const int nt = min(kC, sp.n - k * kC);
-    cp_wait<1>();
-    __syncthreads();                                     // chunk k has arrived for everyone; chunk k - 1 is read
-    fetch(k + 2);
-    const uint32_t rb = smem_u32(sd_smem + (k % kRing) * 2 * kTile), rc = rb + kTile * 2;
-    const uint32_t x[4] = {vals[0], vals[1], vals[2], vals[3]};
-    const float dt = (lane & 15) < nt ? MsFn<__nv_bfloat16>::softplus(dt_raw + bias) : 0.f;
-    if (k + 1 < chunks) {
-      const int more = sp.n - (k + 1) * kC;
-      load_values(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, more, left, lane, vals);
-      if ((lane & 15) < more) dt_raw = raw[static_cast<size_t>((k + 1) * kC + (lane & 15)) * a.ld_decay];
-    }
-    float G = A * dt;                                    // running sum over the chunk's rows, lane = row
+}
+
+// One block of 4 warps per (chunk, key head): C B^T once, then the records of the heads that share it.
+template <int DP>
+__global__ void __launch_bounds__(128) ssd_prep_kernel(const MatrixStateArgs a) {
+  constexpr int LD = DP + 8;
+  __shared__ __align__(16) __nv_bfloat16 tile[2][kC * LD];           // B, C
+  const int chunk = blockIdx.x, kh = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const MsSpan sp = ms_span(a, blockIdx.z);
+  const int nt = min(kC, sp.n - chunk * kC);
+  if (nt <= 0) return;
+  const size_t row0 = static_cast<size_t>(sp.row0 + chunk * kC);
+  const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u) + row0 * a.ld_u;
+  const int kb = a.k0 + kh * a.dim, qb = a.q0 + kh * a.dim, rep = a.heads / a.key_heads;
+  const bool vec = ((a.dim | kb | qb | a.ld_u) & 7) == 0;
+  if (a.dim < DP)
+    for (int i = threadIdx.x; i < 2 * kC * LD / 8; i += 128) reinterpret_cast<uint4*>(tile[0])[i] = make_uint4(0u, 0u, 0u, 0u);
+  __syncthreads();
+  fetch_rows(tile[0], LD, u + kb, a.ld_u, a.dim, nt, vec, threadIdx.x, 128);
+  fetch_rows(tile[1], LD, u + qb, a.ld_u, a.dim, nt, vec, threadIdx.x, 128);
+  cp_commit();
+  cp_wait<0>();
+  __syncthreads();
+  float P[2][4] = {};                                    // C B^T [i, j]
+  const uint32_t rb = smem_u32(tile[0]) + rows_as_n(lane, LD) * 2, rc = smem_u32(tile[1]) + rows_as_m(lane, LD) * 2;
+#pragma unroll
+  for (int ks = 0; ks < DP / 16; ++ks) {
+    uint32_t ca[4], bn[4];
+    ldsm4(ca, rc + 32 * ks);
+    ldsm4(bn, rb + 32 * ks);
+    mma(P[0], ca, bn);
+    mma(P[1], ca, bn + 2);
+  }
+  for (int head = kh * rep + warp; head < (kh + 1) * rep; head += 4) {
+    const int t = lane & 15;
+    const float dt = t < nt ? MsFn<__nv_bfloat16>::softplus(a.decay[(row0 + t) * a.ld_decay + head] + a.decay_b[head]) : 0.f;
+    float G = a.A[head] * dt;                            // running sum over the chunk's rows, lane = row
 #pragma unroll
     for (int o = 1; o < 16; o <<= 1) {
       const float up = __shfl_up_sync(0xffffffffu, G, o, 16);
-      if ((lane & 15) >= o) G += up;
+      if (t >= o) G += up;
     }
     const float last = __shfl_sync(0xffffffffu, G, 15);
-    const float Gr[2] = {__shfl_sync(0xffffffffu, G, lane >> 2), __shfl_sync(0xffffffffu, G, (lane >> 2) + 8)};
-    float Gc[4], dc[4];                                  // rows (lane & 3) * 2 + {0, 1} (+ 8)
+    unsigned char* rec = static_cast<unsigned char*>(a.chunk_records) +
+                         ((static_cast<size_t>(blockIdx.z) * gridDim.x + chunk) * a.heads + head) * SsdRecord::kBytes;
+    float* fl = reinterpret_cast<float*>(rec + SsdRecord::kG);
+    if (lane < 16) {
+      fl[t] = __expf(G);
+      fl[16 + t] = __expf(last - G) * dt;
+      if (t == 0) fl[32] = __expf(last);
+    }
+    float Gj[4], dj[4];                                  // rows j = (lane & 3) * 2 + {0, 1} (+ 8)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int t = (lane & 3) * 2 + (e & 1) + (e >> 1) * 8;
-      Gc[e] = __shfl_sync(0xffffffffu, G, t);
-      dc[e] = __shfl_sync(0xffffffffu, dt, t);
+      const int j = (lane & 3) * 2 + (e & 1) + (e >> 1) * 8;
+      Gj[e] = __shfl_sync(0xffffffffu, G, j);
+      dj[e] = __shfl_sync(0xffffffffu, dt, j);
     }
-    float P[2][4] = {}, O[2][2][4] = {};                 // C B^T [i, j]; S0^T C^T by the split of S0
 #pragma unroll
-    for (int ks = 0; ks < DP / 16; ++ks) {
-      uint32_t hi[4], lo[4], ca[4], cn[4], bn[4];
-      split_a(S[2 * ks], S[2 * ks + 1], hi, lo);
-      ldsm4(cn, rc + on + 32 * ks);
-      ldsm4(ca, rc + om + 32 * ks);
-      ldsm4(bn, rb + on + 32 * ks);
-#pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        mma(O[0][t], hi, cn + 2 * t);
-        mma(O[1][t], lo, cn + 2 * t);
-        mma(P[t], ca, bn + 2 * t);
-      }
-    }
-    // masked and decayed products as the right operand: the accumulator layout of [i, j] is that of an operand with j as K
-    uint32_t mh[2][2], ml[2][2];
-#pragma unroll
-    for (int i8 = 0; i8 < 2; ++i8)
+    for (int i8 = 0; i8 < 2; ++i8) {
+      const int i = (lane >> 2) + 8 * i8;
+      const float Gi = __shfl_sync(0xffffffffu, G, i);
 #pragma unroll
       for (int j8 = 0; j8 < 2; ++j8) {
         float w[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int i = (lane >> 2) + 8 * i8, j = (lane & 3) * 2 + e + 8 * j8;
-          w[e] = j <= i ? P[j8][2 * i8 + e] * __expf(Gr[i8] - Gc[2 * j8 + e]) * dc[2 * j8 + e] : 0.f;
+          const int j = (lane & 3) * 2 + e + 8 * j8;
+          w[e] = j <= i ? P[j8][2 * i8 + e] * __expf(Gi - Gj[2 * j8 + e]) * dj[2 * j8 + e] : 0.f;
         }
-        split2(w[0], w[1], mh[i8][j8], ml[i8][j8]);
+        uint32_t hi, lo;
+        split2(w[0], w[1], hi, lo);
+        const int at = (i * kSq + (lane & 3) * 2 + 8 * j8) * 2;
+        *reinterpret_cast<uint32_t*>(rec + at) = hi;
+        *reinterpret_cast<uint32_t*>(rec + SsdRecord::kSmall + at) = lo;
       }
-    float o[2][4];
+    }
+  }
+}
+
+template <int DP>
+struct SsdStage {
+  static constexpr int LD = DP + 8;
+  __nv_bfloat16 B[kC * LD], C[kC * LD];
+  unsigned char rec[SsdRecord::kBytes];
+};
+
+// One block = (head, 16 NG columns, sequence), two warps per 16 columns.
+template <int DP, int NG>
+__global__ void __launch_bounds__(64 * NG) ssd_chunk_kernel(const MatrixStateArgs a, int chunks_max) {
+  constexpr int LD = DP + 8, NW = 2 * NG, NT = DP / 16, kThreads = 32 * NW, kStages = 4;
+  extern __shared__ __align__(16) unsigned char sd_smem[];
+  SsdStage<DP>* stage = reinterpret_cast<SsdStage<DP>*>(sd_smem);
+  __shared__ __align__(16) float4 swap[2][NW][32];
+  const int head = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const MsSpan sp = ms_span(a, blockIdx.z);
+  const int grp = warp >> 1, half = warp & 1, key0 = half * (DP / 2);
+  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NG, col = c0 + grp * 16, left = a.vdim - col;
+  const int kh = head / (a.heads / a.key_heads);
+  const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u;
+  const unsigned char* rec = static_cast<const unsigned char*>(a.chunk_records) +
+                             (static_cast<size_t>(blockIdx.z) * chunks_max * a.heads + head) * SsdRecord::kBytes;
+  const int kb = a.k0 + kh * a.dim, qb = a.q0 + kh * a.dim;
+  const bool vec = ((a.dim | kb | qb | a.ld_u) & 7) == 0;
+  if (a.dim < DP)
+    for (int i = threadIdx.x; i < kStages * static_cast<int>(sizeof(SsdStage<DP>)) / 16; i += kThreads) reinterpret_cast<uint4*>(sd_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
+  __syncthreads();
+  auto fetch = [&](int k) {
+    if (k < chunks) {
+      SsdStage<DP>& d = stage[k % kStages];
+      const int nt = min(kC, sp.n - k * kC);
+      const __nv_bfloat16* src = u + static_cast<size_t>(k) * kC * a.ld_u;
+      fetch_rows(d.B, LD, src + kb, a.ld_u, a.dim, nt, vec, threadIdx.x, kThreads);
+      fetch_rows(d.C, LD, src + qb, a.ld_u, a.dim, nt, vec, threadIdx.x, kThreads);
+      for (int i = threadIdx.x; i < SsdRecord::kBytes / 16; i += kThreads)
+        cp16(smem_u32(d.rec) + 16 * i, rec + static_cast<size_t>(k) * a.heads * SsdRecord::kBytes + 16 * i);
+    }
+    cp_commit();                                         // always, so that groups count chunks
+  };
+#pragma unroll
+  for (int i = 0; i < kStages - 1; ++i) fetch(i);
+  const float D = a.D[head];
+  float* state = a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim;
+  float S[NT][4];
+  load_state<NT>(a, state, key0, col, lane, sp.start > 0 && sp.n > 0, S);
+  zero_front(a, sp, blockIdx.z, head, c0, 16 * NG, kThreads);
+  const __nv_bfloat16* v = u + a.v0 + head * a.vdim + min(col, a.vdim - 1);
+  float* out = a.out + static_cast<size_t>(sp.row0) * a.ld_out + head * a.vdim + col;
+  Values vals;
+  if (chunks > 0) vals.load(v, a.ld_u, min(kC, sp.n), left, lane);
+  const int on = (rows_as_n(lane, LD) + key0) * 2, om = (rows_as_m(lane, LD) + key0) * 2, os = rows_as_n(lane, kSq) * 2;
+  for (int k = 0; k < chunks; ++k) {
+    const int nt = min(kC, sp.n - k * kC);
+    cp_wait<kStages - 2>();
+    __syncthreads();                                     // chunk k has arrived for everyone; chunk k - 1 is read
+    fetch(k + kStages - 1);
+    const SsdStage<DP>& d = stage[k % kStages];
+    const uint32_t rb = smem_u32(d.B), rc = smem_u32(d.C), rr = smem_u32(d.rec);
+    const float* fl = reinterpret_cast<const float*>(d.rec + SsdRecord::kG);
+    uint32_t x[4];
+    vals.pack(x);
+    if (k + 1 < chunks) vals.load(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, min(kC, sp.n - (k + 1) * kC), left, lane);
+    float O[2][2][4] = {};                               // S0^T C^T by the split of S0
+#pragma unroll
+    for (int ks = 0; ks < NT / 2; ++ks) {
+      uint32_t hi[4], lo[4], cn[4];
+      split_a(S[2 * ks], S[2 * ks + 1], hi, lo);
+      ldsm4(cn, rc + on + 32 * ks);
+#pragma unroll
+      for (int t = 0; t < 2; ++t) {
+        mma(O[0][t], hi, cn + 2 * t);
+        mma(O[1][t], lo, cn + 2 * t);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[0][t][e] += O[1][t][e];
+    // of the outputs this warp finishes the tile `half`; the partner gets the partial sums of the other
+    swap[k & 1][warp][lane] = half ? make_float4(O[0][0][0], O[0][0][1], O[0][0][2], O[0][0][3])
+                                   : make_float4(O[0][1][0], O[0][1][1], O[0][1][2], O[0][1][3]);
     uint32_t uh[4], ul[4];
 #pragma unroll
     for (int t = 0; t < 2; ++t) {
-      const float e0 = __expf(Gc[2 * t]), e1 = __expf(Gc[2 * t + 1]);
-      const float f0 = __expf(last - Gc[2 * t]) * dc[2 * t], f1 = __expf(last - Gc[2 * t + 1]) * dc[2 * t + 1];
+      const float2 f = *reinterpret_cast<const float2*>(fl + 16 + 8 * t + (lane & 3) * 2);
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const float x0 = bf16_lo(x[2 * t + h]), x1 = bf16_hi(x[2 * t + h]);
-        o[t][2 * h] = fmaf(D, x0, (O[0][t][2 * h] + O[1][t][2 * h]) * e0);
-        o[t][2 * h + 1] = fmaf(D, x1, (O[0][t][2 * h + 1] + O[1][t][2 * h + 1]) * e1);
-        split2(x0 * f0, x1 * f1, uh[2 * t + h], ul[2 * t + h]);
-      }
+      for (int h = 0; h < 2; ++h) split2(bf16_lo(x[2 * t + h]) * f.x, bf16_hi(x[2 * t + h]) * f.y, uh[2 * t + h], ul[2 * t + h]);
     }
-    const float el = __expf(last);
+    const float el = fl[32];
 #pragma unroll
-    for (int p = 0; p < DP / 16; ++p) {
+    for (int n = 0; n < NT; ++n) {
+      S[n][0] *= el; S[n][1] *= el; S[n][2] *= el; S[n][3] *= el;
+    }
+#pragma unroll
+    for (int p = 0; p < NT / 2; ++p) {
       uint32_t b[4];
       ldsm4t(b, rb + om + 32 * p);
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
-        float* st = S[2 * p + t];
-        st[0] *= el; st[1] *= el; st[2] *= el; st[3] *= el;
-        mma(st, uh, b + 2 * t);
-        mma(st, ul, b + 2 * t);
+        mma(S[2 * p + t], uh, b + 2 * t);
+        mma(S[2 * p + t], ul, b + 2 * t);
       }
     }
-#pragma unroll
-    for (int t = 0; t < 2; ++t) {
-      mma(o[t], x, mh[t]);
-      mma(o[t], x, ml[t]);
-    }
-    store_outputs(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, nt, left, lane, o);
+    uint32_t mh[4], ml[4];
+    ldsm4(mh, rr + os);
+    ldsm4(ml, rr + SsdRecord::kSmall + os);
+    const float2 eg = *reinterpret_cast<const float2*>(fl + 8 * half + (lane & 3) * 2);
+    pair_sync(1 + grp);
+    const float4 po = swap[k & 1][warp ^ 1][lane];
+    const uint32_t x0 = half ? x[2] : x[0], x1 = half ? x[3] : x[1];
+    float y[4];
+    y[0] = fmaf(D, bf16_lo(x0), ((half ? O[0][1][0] : O[0][0][0]) + po.x) * eg.x);
+    y[1] = fmaf(D, bf16_hi(x0), ((half ? O[0][1][1] : O[0][0][1]) + po.y) * eg.y);
+    y[2] = fmaf(D, bf16_lo(x1), ((half ? O[0][1][2] : O[0][0][2]) + po.z) * eg.x);
+    y[3] = fmaf(D, bf16_hi(x1), ((half ? O[0][1][3] : O[0][0][3]) + po.w) * eg.y);
+    const uint32_t th[2] = {half ? mh[2] : mh[0], half ? mh[3] : mh[1]}, tl[2] = {half ? ml[2] : ml[0], half ? ml[3] : ml[1]};
+    mma(y, x, th);
+    mma(y, x, tl);
+    store_tile(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, half * 8, nt, left, lane, y);
   }
-  if (sp.n > 0) store_state<DP>(a, state, col, lane, S);
+  if (sp.n > 0) store_state<NT>(a, state, key0, col, lane, S);
 }
 
 template <typename K>
@@ -564,14 +703,14 @@ cudaError_t allow_smem(DeviceOnce& once, K kernel, int bytes) {
   return once.run([&] { return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes); });
 }
 
-template <int DP, int NW>
+template <int DP, int NG>
 cudaError_t delta_cols(const MatrixStateArgs& a, int chunks, cudaStream_t s) {
   constexpr int smem = kRing * Record<DP>::kBytes;
-  static_assert(smem <= 220 * 1024 && Record<DP>::kBytes % 16 == 0, "shared memory");
+  static_assert(smem <= 200 * 1024 && Record<DP>::kBytes % 16 == 0, "shared memory");
   static DeviceOnce once;
-  cudaError_t e = allow_smem(once, delta_chunk_kernel<DP, NW>, smem);
+  cudaError_t e = allow_smem(once, delta_chunk_kernel<DP, NG>, smem);
   if (e != cudaSuccess) return e;
-  delta_chunk_kernel<DP, NW><<<dim3(a.heads, (a.vdim + 16 * NW - 1) / (16 * NW), a.nseq), 32 * (NW + 1), smem, s>>>(a, chunks);
+  delta_chunk_kernel<DP, NG><<<dim3(a.heads, (a.vdim + 16 * NG - 1) / (16 * NG), a.nseq), 32 * (2 * NG + 1), smem, s>>>(a, chunks);
   return cudaGetLastError();
 }
 
@@ -587,31 +726,41 @@ cudaError_t delta(const MatrixStateArgs& a, cudaStream_t s) {
   if (e != cudaSuccess) return e;
   // as few columns per block as still give every SM a block
   const int64_t cols = static_cast<int64_t>(a.heads) * a.nseq * ((a.vdim + 15) / 16);
-  return cols <= 148 * 4 ? delta_cols<DP, 2>(a, chunks, s) : delta_cols<DP, 4>(a, chunks, s);
+  return cols <= 148 * 2 ? delta_cols<DP, 2>(a, chunks, s) : delta_cols<DP, 4>(a, chunks, s);
+}
+
+template <int DP, int NG>
+cudaError_t ssd_cols(const MatrixStateArgs& a, int chunks, cudaStream_t s) {
+  constexpr int smem = 4 * static_cast<int>(sizeof(SsdStage<DP>));
+  static_assert(smem <= 200 * 1024 && sizeof(SsdStage<DP>) % 16 == 0, "shared memory");
+  static DeviceOnce once;
+  cudaError_t e = allow_smem(once, ssd_chunk_kernel<DP, NG>, smem);
+  if (e != cudaSuccess) return e;
+  ssd_chunk_kernel<DP, NG><<<dim3(a.heads, (a.vdim + 16 * NG - 1) / (16 * NG), a.nseq), 64 * NG, smem, s>>>(a, chunks);
+  return cudaGetLastError();
 }
 
 template <int DP>
 cudaError_t ssd(const MatrixStateArgs& a, cudaStream_t s) {
-  constexpr int smem = kRing * 2 * kC * (DP + 8) * 2, NW = 4;
-  static DeviceOnce once;
-  cudaError_t e = allow_smem(once, ssd_chunk_kernel<DP, NW>, smem);
+  const int chunks = (a.rows.Tc + kC - 1) / kC;
+  ssd_prep_kernel<DP><<<dim3(chunks, a.key_heads, a.nseq), 128, 0, s>>>(a);
+  const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  ssd_chunk_kernel<DP, NW><<<dim3(a.heads, (a.vdim + 16 * NW - 1) / (16 * NW), a.nseq), 32 * NW, smem, s>>>(a);
-  return cudaGetLastError();
+  const int64_t cols = static_cast<int64_t>(a.heads) * a.nseq * ((a.vdim + 15) / 16);
+  return cols <= 148 * 2 ? ssd_cols<DP, 2>(a, chunks, s) : ssd_cols<DP, 4>(a, chunks, s);
 }
 
 }  // namespace
 
-int64_t matrix_chunk_record_bytes(int dim) {
+int64_t matrix_chunk_record_bytes(int dim, int delta) {
+  if (!delta) return SsdRecord::kBytes;
   return dim <= 32 ? Record<32>::kBytes : dim <= 64 ? Record<64>::kBytes : dim <= 128 ? Record<128>::kBytes : Record<256>::kBytes;
 }
 
 cudaError_t launch_matrix_chunks(const MatrixStateArgs& a, cudaStream_t s) {
   if (!matrix_state_ok(a) || !a.u_bf16 || a.nseq > 65535 || a.heads > 65535) return cudaErrorInvalidValue;
-  if (a.delta) {
-    if (!a.chunk_records || (reinterpret_cast<uintptr_t>(a.chunk_records) & 15)) return cudaErrorInvalidValue;
-    return a.dim <= 32 ? delta<32>(a, s) : a.dim <= 64 ? delta<64>(a, s) : a.dim <= 128 ? delta<128>(a, s) : delta<256>(a, s);
-  }
+  if (!a.chunk_records || (reinterpret_cast<uintptr_t>(a.chunk_records) & 15)) return cudaErrorInvalidValue;
+  if (a.delta) return a.dim <= 32 ? delta<32>(a, s) : a.dim <= 64 ? delta<64>(a, s) : a.dim <= 128 ? delta<128>(a, s) : delta<256>(a, s);
   return a.dim <= 32 ? ssd<32>(a, s) : a.dim <= 64 ? ssd<64>(a, s) : a.dim <= 128 ? ssd<128>(a, s) : ssd<256>(a, s);
 }
 

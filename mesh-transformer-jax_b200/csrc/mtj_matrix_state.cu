@@ -338,6 +338,63 @@ cudaError_t step(const MatrixStateArgs& a, const GatedNormArgs* norm, cudaStream
 }
 
 // ---- norm and gate of the outputs: one group of TH threads per (row, part)
+__device__ __forceinline__ float4 ms_ld4(const float* p, size_t i) { return *reinterpret_cast<const float4*>(p + i); }
+__device__ __forceinline__ float4 ms_ld4(const __nv_bfloat16* p, size_t i) {
+  const uint2 w = *reinterpret_cast<const uint2*>(p + i);
+  return make_float4(bf16_lo(w.x), bf16_hi(w.x), bf16_lo(w.y), bf16_hi(w.y));
+}
+__device__ __forceinline__ float4 mul4(const float4& x, const float4& y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); }
+template <typename F>
+__device__ __forceinline__ float4 map4(const float4& x, F&& f) { return make_float4(f(x.x), f(x.y), f(x.z), f(x.w)); }
+
+// part_n and the row strides multiples of four, part_n up to 16 TH: four neighbouring columns a thread, loads first
+template <typename T, int TH>
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const GatedNormArgs a) {
+  __shared__ float red[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  constexpr int kGroups = 256 / TH, kHold = 4;
+  const int grp = threadIdx.x / TH, t = threadIdx.x % TH;
+  const int64_t id = static_cast<int64_t>(blockIdx.x) * kGroups + grp;
+  if (id >= static_cast<int64_t>(a.M) * a.parts) return;   // whole groups leave; with TH = 256 the grid is exact
+  const size_t m = static_cast<size_t>(id / a.parts);
+  const int c0 = static_cast<int>(id % a.parts) * a.part_n;
+  const float* y = a.y + m * a.ld_y + c0;
+  const T* gate = static_cast<const T*>(a.gate) + m * a.ld_gate + c0;
+  float4 v[kHold], g[kHold];
+#pragma unroll
+  for (int j = 0; j < kHold; ++j) {
+    const int i = 4 * (j * TH + t);
+    v[j] = i < a.part_n ? ms_ld4(y, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    g[j] = i < a.part_n ? ms_ld4(gate, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kHold; ++j) {
+    if (a.gate_first) v[j] = mul4(v[j], map4(g[j], [](float z) { return MsFn<T>::silu(z); }));
+    ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+  }
+  ss = warp_sum(ss);
+  if (TH > 32) {
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += red[i];
+  }
+  const float rs = 1.0f / sqrtf(ss / static_cast<float>(a.part_n) + a.eps);
+#pragma unroll
+  for (int j = 0; j < kHold; ++j) {
+    const int i = 4 * (j * TH + t);
+    if (i >= a.part_n) continue;
+    float4 o = mul4(map4(v[j], [&](float z) { return z * rs; }), ms_ld4(a.w, a.gate_first ? c0 + i : i));
+    if (!a.gate_first) o = mul4(o, map4(g[j], [](float z) { return MsFn<T>::sigmoid(z); }));
+    const size_t at = m * a.ld_out + c0 + i;
+    if (a.out) *reinterpret_cast<float4*>(a.out + at) = o;
+    if (a.out_bf16) *reinterpret_cast<uint2*>(a.out_bf16 + at) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+  }
+}
+
 template <typename T, int TH>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormArgs a) {
   __shared__ float red[8];
@@ -392,6 +449,9 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormArgs a) 
 template <typename T>
 cudaError_t gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl) {
   const int64_t n = static_cast<int64_t>(a.M) * a.parts;
+  if (((a.part_n | a.ld_y | a.ld_gate | a.ld_out) & 3) == 0 && a.part_n <= 16 * 256)
+    return a.part_n <= 16 * 32 ? launch_pdl(gated_norm_vec_kernel<T, 32>, dim3(static_cast<unsigned>((n + 7) / 8)), dim3(256), 0, s, pdl, a)
+                               : launch_pdl(gated_norm_vec_kernel<T, 256>, dim3(static_cast<unsigned>(n)), dim3(256), 0, s, pdl, a);
   if (a.part_n <= 256) return launch_pdl(gated_norm_kernel<T, 32>, dim3(static_cast<unsigned>((n + 7) / 8)), dim3(256), 0, s, pdl, a);
   return launch_pdl(gated_norm_kernel<T, 256>, dim3(static_cast<unsigned>(n)), dim3(256), 0, s, pdl, a);
 }

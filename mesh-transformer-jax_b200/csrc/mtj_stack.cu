@@ -252,7 +252,7 @@ void LayerStack::carve_workspace(Carver& c) {
       aux = std::max<int64_t>(aux, up8(l.aux));
       mix = std::max<int64_t>(mix, l.out.ld);
       if (l.dt.N) dtw = std::max<int64_t>(dtw, up8(l.dt.N));
-      if (m.mixer == MTJ_MIXER_MATRIX_STATE_DELTA) rec = std::max(rec, m.heads * matrix_chunk_record_bytes(m.dim));
+      rec = std::max(rec, m.heads * matrix_chunk_record_bytes(m.dim, m.mixer == MTJ_MIXER_MATRIX_STATE_DELTA));
       if (l.gate2.N) gate = std::max<int64_t>(gate, up8(l.gate2.N));
     } else {
       qabs = std::max<int64_t>(qabs, static_cast<int64_t>(m.heads) * l.row_ld);
@@ -999,7 +999,7 @@ int32_t LayerStack::matrix(mtj_handle* h, const Run& r, int M, const RowMap& row
   else if (tc && rows.Tc >= kChunkedRows) MTJ_CUDA(launch_matrix_chunks(a, s));
   else MTJ_CUDA(launch_matrix_scan(a, s, pdl));
   if (!normed) MTJ_CUDA(launch_gated_norm(g, s, pdl));
-  h->launches += (normed ? 1 : 2) + (!ssd && tc && rows.Tc >= kChunkedRows ? 1 : 0);
+  h->launches += (normed ? 1 : 2) + (!step && tc && rows.Tc >= kChunkedRows ? 1 : 0);
   h->prof_end(s);
   h->prof_begin(MTJ_FAMILY_OUTPROJ, s);
   if (tc) MTJ_DO(gemm(h, kEpiPlain, l.out, act_bf_, M, y_, ld_, nullptr, 0, decode, s));

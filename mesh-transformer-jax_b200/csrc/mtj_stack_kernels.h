@@ -150,7 +150,7 @@ cudaError_t launch_grouped_prep(const GroupedAttnArgs& a, cudaStream_t s, bool p
 // every row of the call by itself, from the cache
 cudaError_t launch_grouped_attn(const GroupedAttnArgs& a, cudaStream_t s, bool pdl);
 constexpr int kGroupedMaxDim = 512;
-constexpr int kGroupedBlocks = 592;      // most (rows x key heads x splits) a call spreads over beyond one per row and head
+constexpr int kGroupedBlocks = 2368;     // most (rows x key heads x splits) a call spreads over beyond one per row and head
 int grouped_attn_splits(int M, int heads, int kv_heads, int window);
 int grouped_counters(int heads, int kv_heads);   // per row
 
@@ -191,7 +191,7 @@ struct MatrixStateArgs {
   float* state;                // [slots][heads][dim][vdim]
   float* out;                  // [M, ld_out]
   int ld_out;
-  void* chunk_records;         // launch_matrix_chunks, delta: nseq * ceil(Tc / kMatrixChunk) * heads records, 16-byte aligned
+  void* chunk_records;         // launch_matrix_chunks: nseq * ceil(Tc / kMatrixChunk) * heads records, 16-byte aligned
   uint32_t* dev_err;
 };
 // row by row
@@ -202,7 +202,7 @@ bool matrix_step_ok(const MatrixStateArgs& a);      // sizes that kernel takes
 bool matrix_step_norms(const MatrixStateArgs& a);
 // ---- mtj_matrix_chunk.cu: the same over long prompts, in chunks on the tensor cores (bf16 operands)
 constexpr int kMatrixChunk = 16;
-int64_t matrix_chunk_record_bytes(int dim);
+int64_t matrix_chunk_record_bytes(int dim, int delta);
 cudaError_t launch_matrix_chunks(const MatrixStateArgs& a, cudaStream_t s);
 cudaError_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl);
 constexpr int kMatrixMaxDim = 256;
