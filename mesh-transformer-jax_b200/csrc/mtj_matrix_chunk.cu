@@ -135,6 +135,20 @@ __device__ __forceinline__ float dot4(const float4& x, const float4& y, float s)
   return fmaf(x.w, y.w, fmaf(x.z, y.z, fmaf(x.y, y.y, fmaf(x.x, y.x, s))));
 }
 
+// elements n .. n + 3 of a row, zeros from `have` on
+__device__ __forceinline__ float4 four(const float* p, int n, int have, bool vec) {
+  if (vec) return n < have ? *reinterpret_cast<const float4*>(p + n) : make_float4(0.f, 0.f, 0.f, 0.f);
+  return make_float4(n < have ? p[n] : 0.f, n + 1 < have ? p[n + 1] : 0.f, n + 2 < have ? p[n + 2] : 0.f, n + 3 < have ? p[n + 3] : 0.f);
+}
+__device__ __forceinline__ float4 four(const __nv_bfloat16* p, int n, int have, bool vec) {
+  if (vec) {
+    const uint2 w = n < have ? *reinterpret_cast<const uint2*>(p + n) : make_uint2(0u, 0u);
+    return make_float4(bf16_lo(w.x), bf16_hi(w.x), bf16_lo(w.y), bf16_hi(w.y));
+  }
+  return make_float4(n < have ? __bfloat162float(p[n]) : 0.f, n + 1 < have ? __bfloat162float(p[n + 1]) : 0.f,
+                     n + 2 < have ? __bfloat162float(p[n + 2]) : 0.f, n + 3 < have ? __bfloat162float(p[n + 3]) : 0.f);
+}
+
 // One block of 4 warps per (chunk, head).
 template <int DP>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const MatrixStateArgs a) {
@@ -148,40 +162,48 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const MatrixStateArgs a
   const int kh = head / (a.heads / a.key_heads);
   const float A = a.A[head];
   const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u);
-  constexpr int NC = DP / 32;
+  // a warp per row, a lane four neighbouring channels
+  constexpr int N4 = (DP + 127) / 128;
+  const int kcol = a.k0 + kh * a.dim, qcol = a.q0 + kh * a.dim, dcol = head * a.dim;
+  const bool vec = ((a.dim | kcol | qcol | a.ld_u | a.ld_decay) & 3) == 0;
+  float4 bias[N4];
 #pragma unroll
-  for (int i = 0; i < kC / 4; ++i) {                  // a warp per row
+  for (int c = 0; c < N4; ++c) bias[c] = four(a.decay_b + dcol, c * 128 + 4 * lane, a.dim, vec);
+#pragma unroll
+  for (int i = 0; i < kC / 4; ++i) {
     const int t = warp + 4 * i;
     const size_t m = static_cast<size_t>(sp.row0 + chunk * kC + min(t, nt - 1));
     const __nv_bfloat16* row = u + m * a.ld_u;
-    float kv[NC], qv[NC], gv[NC], ks = 0.f, qs = 0.f;
+    const int have = t < nt ? a.dim : 0;
+    float4 kv[N4], qv[N4], gv[N4];
+    float ks = 0.f, qs = 0.f;
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int n = c * 32 + lane;
-      const bool in = t < nt && n < a.dim;
-      kv[c] = in ? __bfloat162float(row[a.k0 + kh * a.dim + n]) : 0.f;
-      qv[c] = in ? __bfloat162float(row[a.q0 + kh * a.dim + n]) : 0.f;
-      gv[c] = in ? a.decay[m * a.ld_decay + head * a.dim + n] + a.decay_b[head * a.dim + n] : 0.f;
+    for (int c = 0; c < N4; ++c) {
+      const int n = c * 128 + 4 * lane;
+      kv[c] = four(row + kcol, n, have, vec);
+      qv[c] = four(row + qcol, n, have, vec);
+      gv[c] = four(a.decay + m * a.ld_decay + dcol, n, have, vec);
     }
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      ks = fmaf(kv[c], kv[c], ks);
-      qs = fmaf(qv[c], qv[c], qs);
+    for (int c = 0; c < N4; ++c) {
+      ks = dot4(kv[c], kv[c], ks);
+      qs = dot4(qv[c], qv[c], qs);
     }
     const float kr = 1.0f / sqrtf(warp_sum(ks) + kUnitEps), qr = a.q_scale / sqrtf(warp_sum(qs) + kUnitEps);
 #pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int n = c * 32 + lane;
-      sm.k[t][n] = kv[c] * kr;
-      sm.q[t][n] = qv[c] * qr;
-      sm.g[t][n] = t < nt ? MsFn<__nv_bfloat16>::exp(A * MsFn<__nv_bfloat16>::softplus(gv[c])) : 1.0f;
+    for (int c = 0; c < N4; ++c) {
+      const int n = c * 128 + 4 * lane;
+      if (n >= DP) continue;
+      auto g = [&](float raw, float b) { return t < nt ? MsFn<__nv_bfloat16>::exp(A * MsFn<__nv_bfloat16>::softplus(raw + b)) : 1.0f; };
+      *reinterpret_cast<float4*>(&sm.k[t][n]) = make_float4(kv[c].x * kr, kv[c].y * kr, kv[c].z * kr, kv[c].w * kr);
+      *reinterpret_cast<float4*>(&sm.q[t][n]) = make_float4(qv[c].x * qr, qv[c].y * qr, qv[c].z * qr, qv[c].w * qr);
+      *reinterpret_cast<float4*>(&sm.g[t][n]) = make_float4(g(gv[c].x, bias[c].x), g(gv[c].y, bias[c].y), g(gv[c].z, bias[c].z), g(gv[c].w, bias[c].w));
     }
     if (lane == 0) sm.beta[t] = t < nt ? MsFn<__nv_bfloat16>::sigmoid(a.beta[m * a.ld_beta + head]) : 0.f;
   }
   __syncthreads();
   // L_ij and M_ij, lanes over the key channels (four neighbours each); a warp takes columns j of a balanced total
   // length and walks the rows in fours, whose eight sums are brought together by a transposing reduction
-  constexpr int N4 = (DP + 127) / 128;
 #pragma unroll 1
   for (int s = 0; s < 4; ++s) {
     const int j = s == 0 ? warp : s == 1 ? 15 - warp : s == 2 ? 4 + warp : 11 - warp;
@@ -477,6 +499,10 @@ struct SsdRecord {                   // of one (chunk, head); byte offsets
   static constexpr int kG = 2 * kSmall;                // floats: e^(G_i) [16], e^(G_C - G_j) dt_j [16], e^(G_C)
   static constexpr int kBytes = kG + 4 * 36;
 };
+template <int DP>
+struct SsdTiles {                    // of one (chunk, key head): B then C, zero-padded; they follow all head records
+  static constexpr int LD = DP + 8, kMat = kC * LD * 2, kBytes = 2 * kMat;
+};
 static_assert(SsdRecord::kBytes % 16 == 0, "whole pieces");
 
 // 16 rows of `dim` columns -> [kC][LD] in shared memory by `threads` threads; rows from nt on are zero
@@ -518,6 +544,9 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(const MatrixStateArgs a) 
   cp_commit();
   cp_wait<0>();
   __syncthreads();
+  unsigned char* tiles = static_cast<unsigned char*>(a.chunk_records) + static_cast<size_t>(gridDim.z) * gridDim.x * a.heads * SsdRecord::kBytes +
+                         ((static_cast<size_t>(blockIdx.z) * gridDim.x + chunk) * a.key_heads + kh) * SsdTiles<DP>::kBytes;
+  for (int i = threadIdx.x; i < SsdTiles<DP>::kBytes / 16; i += 128) reinterpret_cast<uint4*>(tiles)[i] = reinterpret_cast<const uint4*>(tile[0])[i];
   float P[2][4] = {};                                    // C B^T [i, j]
   const uint32_t rb = smem_u32(tile[0]) + rows_as_n(lane, LD) * 2, rc = smem_u32(tile[1]) + rows_as_m(lane, LD) * 2;
 #pragma unroll
@@ -575,127 +604,135 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(const MatrixStateArgs a) 
   }
 }
 
-template <int DP>
-struct SsdStage {
-  static constexpr int LD = DP + 8;
-  __nv_bfloat16 B[kC * LD], C[kC * LD];
-  unsigned char rec[SsdRecord::kBytes];
-};
-
-// One block = (head, 16 NG columns, sequence), two warps per 16 columns.
+// One block = (head, 16 NG columns, sequence): two scan warps per 16 columns and one that fetches tiles and records.
 template <int DP, int NG>
-__global__ void __launch_bounds__(64 * NG) ssd_chunk_kernel(const MatrixStateArgs a, int chunks_max) {
-  constexpr int LD = DP + 8, NW = 2 * NG, NT = DP / 16, kThreads = 32 * NW, kStages = 4;
-  extern __shared__ __align__(16) unsigned char sd_smem[];
-  SsdStage<DP>* stage = reinterpret_cast<SsdStage<DP>*>(sd_smem);
+__global__ void __launch_bounds__(32 * (2 * NG + 1)) ssd_chunk_kernel(const MatrixStateArgs a, int chunks_max) {
+  using Tiles = SsdTiles<DP>;
+  constexpr int LD = Tiles::LD, NW = 2 * NG, NT = DP / 16, kStages = 4, kStage = Tiles::kBytes + SsdRecord::kBytes;
+  extern __shared__ __align__(128) unsigned char sd_smem[];
   __shared__ __align__(16) float4 swap[2][NW][32];
+  __shared__ __align__(8) uint64_t bars[2 * kStages];
+  __shared__ uint32_t failed;
   const int head = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const MsSpan sp = ms_span(a, blockIdx.z);
-  const int grp = warp >> 1, half = warp & 1, key0 = half * (DP / 2);
-  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NG, col = c0 + grp * 16, left = a.vdim - col;
-  const int kh = head / (a.heads / a.key_heads);
-  const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u;
-  const unsigned char* rec = static_cast<const unsigned char*>(a.chunk_records) +
-                             (static_cast<size_t>(blockIdx.z) * chunks_max * a.heads + head) * SsdRecord::kBytes;
-  const int kb = a.k0 + kh * a.dim, qb = a.q0 + kh * a.dim;
-  const bool vec = ((a.dim | kb | qb | a.ld_u) & 7) == 0;
-  if (a.dim < DP)
-    for (int i = threadIdx.x; i < kStages * static_cast<int>(sizeof(SsdStage<DP>)) / 16; i += kThreads) reinterpret_cast<uint4*>(sd_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
-  __syncthreads();
-  auto fetch = [&](int k) {
-    if (k < chunks) {
-      SsdStage<DP>& d = stage[k % kStages];
-      const int nt = min(kC, sp.n - k * kC);
-      const __nv_bfloat16* src = u + static_cast<size_t>(k) * kC * a.ld_u;
-      fetch_rows(d.B, LD, src + kb, a.ld_u, a.dim, nt, vec, threadIdx.x, kThreads);
-      fetch_rows(d.C, LD, src + qb, a.ld_u, a.dim, nt, vec, threadIdx.x, kThreads);
-      for (int i = threadIdx.x; i < SsdRecord::kBytes / 16; i += kThreads)
-        cp16(smem_u32(d.rec) + 16 * i, rec + static_cast<size_t>(k) * a.heads * SsdRecord::kBytes + 16 * i);
+  const uint32_t full = smem_u32(bars), empty = full + 8 * kStages, base = smem_u32(sd_smem);
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kStages; ++i) {
+      mbar_init(full + 8 * i, 1);
+      mbar_init(empty + 8 * i, NW);
     }
-    cp_commit();                                         // always, so that groups count chunks
-  };
-#pragma unroll
-  for (int i = 0; i < kStages - 1; ++i) fetch(i);
-  const float D = a.D[head];
-  float* state = a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim;
-  float S[NT][4];
-  load_state<NT>(a, state, key0, col, lane, sp.start > 0 && sp.n > 0, S);
-  zero_front(a, sp, blockIdx.z, head, c0, 16 * NG, kThreads);
-  const __nv_bfloat16* v = u + a.v0 + head * a.vdim + min(col, a.vdim - 1);
-  float* out = a.out + static_cast<size_t>(sp.row0) * a.ld_out + head * a.vdim + col;
-  Values vals;
-  if (chunks > 0) vals.load(v, a.ld_u, min(kC, sp.n), left, lane);
-  const int on = (rows_as_n(lane, LD) + key0) * 2, om = (rows_as_m(lane, LD) + key0) * 2, os = rows_as_n(lane, kSq) * 2;
-  for (int k = 0; k < chunks; ++k) {
-    const int nt = min(kC, sp.n - k * kC);
-    cp_wait<kStages - 2>();
-    __syncthreads();                                     // chunk k has arrived for everyone; chunk k - 1 is read
-    fetch(k + kStages - 1);
-    const SsdStage<DP>& d = stage[k % kStages];
-    const uint32_t rb = smem_u32(d.B), rc = smem_u32(d.C), rr = smem_u32(d.rec);
-    const float* fl = reinterpret_cast<const float*>(d.rec + SsdRecord::kG);
-    uint32_t x[4];
-    vals.pack(x);
-    if (k + 1 < chunks) vals.load(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, min(kC, sp.n - (k + 1) * kC), left, lane);
-    float O[2][2][4] = {};                               // S0^T C^T by the split of S0
-#pragma unroll
-    for (int ks = 0; ks < NT / 2; ++ks) {
-      uint32_t hi[4], lo[4], cn[4];
-      split_a(S[2 * ks], S[2 * ks + 1], hi, lo);
-      ldsm4(cn, rc + on + 32 * ks);
-#pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        mma(O[0][t], hi, cn + 2 * t);
-        mma(O[1][t], lo, cn + 2 * t);
-      }
-    }
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) O[0][t][e] += O[1][t][e];
-    // of the outputs this warp finishes the tile `half`; the partner gets the partial sums of the other
-    swap[k & 1][warp][lane] = half ? make_float4(O[0][0][0], O[0][0][1], O[0][0][2], O[0][0][3])
-                                   : make_float4(O[0][1][0], O[0][1][1], O[0][1][2], O[0][1][3]);
-    uint32_t uh[4], ul[4];
-#pragma unroll
-    for (int t = 0; t < 2; ++t) {
-      const float2 f = *reinterpret_cast<const float2*>(fl + 16 + 8 * t + (lane & 3) * 2);
-#pragma unroll
-      for (int h = 0; h < 2; ++h) split2(bf16_lo(x[2 * t + h]) * f.x, bf16_hi(x[2 * t + h]) * f.y, uh[2 * t + h], ul[2 * t + h]);
-    }
-    const float el = fl[32];
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      S[n][0] *= el; S[n][1] *= el; S[n][2] *= el; S[n][3] *= el;
-    }
-#pragma unroll
-    for (int p = 0; p < NT / 2; ++p) {
-      uint32_t b[4];
-      ldsm4t(b, rb + om + 32 * p);
-#pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        mma(S[2 * p + t], uh, b + 2 * t);
-        mma(S[2 * p + t], ul, b + 2 * t);
-      }
-    }
-    uint32_t mh[4], ml[4];
-    ldsm4(mh, rr + os);
-    ldsm4(ml, rr + SsdRecord::kSmall + os);
-    const float2 eg = *reinterpret_cast<const float2*>(fl + 8 * half + (lane & 3) * 2);
-    pair_sync(1 + grp);
-    const float4 po = swap[k & 1][warp ^ 1][lane];
-    const uint32_t x0 = half ? x[2] : x[0], x1 = half ? x[3] : x[1];
-    float y[4];
-    y[0] = fmaf(D, bf16_lo(x0), ((half ? O[0][1][0] : O[0][0][0]) + po.x) * eg.x);
-    y[1] = fmaf(D, bf16_hi(x0), ((half ? O[0][1][1] : O[0][0][1]) + po.y) * eg.y);
-    y[2] = fmaf(D, bf16_lo(x1), ((half ? O[0][1][2] : O[0][0][2]) + po.z) * eg.x);
-    y[3] = fmaf(D, bf16_hi(x1), ((half ? O[0][1][3] : O[0][0][3]) + po.w) * eg.y);
-    const uint32_t th[2] = {half ? mh[2] : mh[0], half ? mh[3] : mh[1]}, tl[2] = {half ? ml[2] : ml[0], half ? ml[3] : ml[1]};
-    mma(y, x, th);
-    mma(y, x, tl);
-    store_tile(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, half * 8, nt, left, lane, y);
+    mbar_fence_init();
+    failed = 0;
   }
-  if (sp.n > 0) store_state<NT>(a, state, key0, col, lane, S);
+  __syncthreads();
+  const MsSpan sp = ms_span(a, blockIdx.z);
+  const int chunks = (sp.n + kC - 1) / kC, c0 = blockIdx.y * 16 * NG;
+  if (warp == NW) {
+    if (lane == 0) {
+      const unsigned char* rec = static_cast<const unsigned char*>(a.chunk_records);
+      const unsigned char* tiles = rec + static_cast<size_t>(gridDim.z) * chunks_max * a.heads * SsdRecord::kBytes +
+                                   (static_cast<size_t>(blockIdx.z) * chunks_max * a.key_heads + head / (a.heads / a.key_heads)) * Tiles::kBytes;
+      rec += (static_cast<size_t>(blockIdx.z) * chunks_max * a.heads + head) * SsdRecord::kBytes;
+      int issued = 0;
+      for (int k = 0; k < chunks; ++k) {
+        const int s = k % kStages;
+        if (k >= kStages && !mbar_wait(empty + 8 * s, ((k / kStages) - 1) & 1)) {
+          atomicOr(&failed, 1u);
+          break;
+        }
+        mbar_expect_tx(full + 8 * s, kStage);
+        bulk_copy(base + s * kStage, tiles + static_cast<size_t>(k) * a.key_heads * Tiles::kBytes, Tiles::kBytes, full + 8 * s);
+        bulk_copy(base + s * kStage + Tiles::kBytes, rec + static_cast<size_t>(k) * a.heads * SsdRecord::kBytes, SsdRecord::kBytes, full + 8 * s);
+        issued = k + 1;
+      }
+      for (int k = max(0, issued - kStages); k < issued; ++k) mbar_wait(full + 8 * (k % kStages), (k / kStages) & 1);   // no copy outlives the block
+    }
+  } else {
+    const int grp = warp >> 1, half = warp & 1, key0 = half * (DP / 2), col = c0 + grp * 16, left = a.vdim - col;
+    const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(a.u) + static_cast<size_t>(sp.row0) * a.ld_u;
+    const float D = a.D[head];
+    float* state = a.state + (static_cast<size_t>(sp.seq) * a.heads + head) * a.dim * a.vdim;
+    float S[NT][4];
+    load_state<NT>(a, state, key0, col, lane, sp.start > 0 && sp.n > 0, S);
+    zero_front(a, sp, blockIdx.z, head, c0, 16 * NG, 32 * NW);
+    const __nv_bfloat16* v = u + a.v0 + head * a.vdim + min(col, a.vdim - 1);
+    float* out = a.out + static_cast<size_t>(sp.row0) * a.ld_out + head * a.vdim + col;
+    Values vals;
+    if (chunks > 0) vals.load(v, a.ld_u, min(kC, sp.n), left, lane);
+    const int on = (rows_as_n(lane, LD) + key0) * 2, om = (rows_as_m(lane, LD) + key0) * 2, os = rows_as_n(lane, kSq) * 2;
+    bool ok = true;                                        // a wait that runs out is remembered; the pair barriers go on
+    for (int k = 0; k < chunks; ++k) {
+      const int s = k % kStages, nt = min(kC, sp.n - k * kC);
+      if (ok) ok = mbar_wait(full + 8 * s, (k / kStages) & 1);
+      const uint32_t rb = base + s * kStage, rc = rb + Tiles::kMat, rr = rb + Tiles::kBytes;
+      const float* fl = reinterpret_cast<const float*>(sd_smem + s * kStage + Tiles::kBytes + SsdRecord::kG);
+      uint32_t x[4];
+      vals.pack(x);
+      if (k + 1 < chunks) vals.load(v + static_cast<size_t>(k + 1) * kC * a.ld_u, a.ld_u, min(kC, sp.n - (k + 1) * kC), left, lane);
+      float O[2][2][4] = {};                               // S0^T C^T by the split of S0
+#pragma unroll
+      for (int ks = 0; ks < NT / 2; ++ks) {
+        uint32_t hi[4], lo[4], cn[4];
+        split_a(S[2 * ks], S[2 * ks + 1], hi, lo);
+        ldsm4(cn, rc + on + 32 * ks);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma(O[0][t], hi, cn + 2 * t);
+          mma(O[1][t], lo, cn + 2 * t);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) O[0][t][e] += O[1][t][e];
+      // of the outputs this warp finishes the tile `half`; the partner gets the partial sums of the other
+      swap[k & 1][warp][lane] = half ? make_float4(O[0][0][0], O[0][0][1], O[0][0][2], O[0][0][3])
+                                     : make_float4(O[0][1][0], O[0][1][1], O[0][1][2], O[0][1][3]);
+      uint32_t uh[4], ul[4];
+#pragma unroll
+      for (int t = 0; t < 2; ++t) {
+        const float2 f = *reinterpret_cast<const float2*>(fl + 16 + 8 * t + (lane & 3) * 2);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) split2(bf16_lo(x[2 * t + h]) * f.x, bf16_hi(x[2 * t + h]) * f.y, uh[2 * t + h], ul[2 * t + h]);
+      }
+      const float el = fl[32];
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        S[n][0] *= el; S[n][1] *= el; S[n][2] *= el; S[n][3] *= el;
+      }
+#pragma unroll
+      for (int p = 0; p < NT / 2; ++p) {
+        uint32_t b[4];
+        ldsm4t(b, rb + om + 32 * p);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma(S[2 * p + t], uh, b + 2 * t);
+          mma(S[2 * p + t], ul, b + 2 * t);
+        }
+      }
+      uint32_t mh[4], ml[4];
+      ldsm4(mh, rr + os);
+      ldsm4(ml, rr + SsdRecord::kSmall + os);
+      const float2 eg = *reinterpret_cast<const float2*>(fl + 8 * half + (lane & 3) * 2);
+      __syncwarp();
+      if (lane == 0) arrive(empty + 8 * s);                // the stage is read
+      pair_sync(1 + grp);
+      const float4 po = swap[k & 1][warp ^ 1][lane];
+      const uint32_t x0 = half ? x[2] : x[0], x1 = half ? x[3] : x[1];
+      float y[4];
+      y[0] = fmaf(D, bf16_lo(x0), ((half ? O[0][1][0] : O[0][0][0]) + po.x) * eg.x);
+      y[1] = fmaf(D, bf16_hi(x0), ((half ? O[0][1][1] : O[0][0][1]) + po.y) * eg.y);
+      y[2] = fmaf(D, bf16_lo(x1), ((half ? O[0][1][2] : O[0][0][2]) + po.z) * eg.x);
+      y[3] = fmaf(D, bf16_hi(x1), ((half ? O[0][1][3] : O[0][0][3]) + po.w) * eg.y);
+      const uint32_t th[2] = {half ? mh[2] : mh[0], half ? mh[3] : mh[1]}, tl[2] = {half ? ml[2] : ml[0], half ? ml[3] : ml[1]};
+      mma(y, x, th);
+      mma(y, x, tl);
+      store_tile(out + static_cast<size_t>(k) * kC * a.ld_out, a.ld_out, half * 8, nt, left, lane, y);
+    }
+    if (!ok) atomicOr(&failed, 1u);
+    if (sp.n > 0 && __all_sync(0xffffffffu, ok)) store_state<NT>(a, state, key0, col, lane, S);
+  }
+  __syncthreads();
+  if (threadIdx.x == 0 && failed && a.dev_err) atomicOr(a.dev_err, kDevErrTimeout);
 }
 
 template <typename K>
@@ -731,12 +768,12 @@ cudaError_t delta(const MatrixStateArgs& a, cudaStream_t s) {
 
 template <int DP, int NG>
 cudaError_t ssd_cols(const MatrixStateArgs& a, int chunks, cudaStream_t s) {
-  constexpr int smem = 4 * static_cast<int>(sizeof(SsdStage<DP>));
-  static_assert(smem <= 200 * 1024 && sizeof(SsdStage<DP>) % 16 == 0, "shared memory");
+  constexpr int smem = 4 * (SsdTiles<DP>::kBytes + SsdRecord::kBytes);
+  static_assert(smem <= 200 * 1024 && SsdTiles<DP>::kBytes % 16 == 0, "shared memory");
   static DeviceOnce once;
   cudaError_t e = allow_smem(once, ssd_chunk_kernel<DP, NG>, smem);
   if (e != cudaSuccess) return e;
-  ssd_chunk_kernel<DP, NG><<<dim3(a.heads, (a.vdim + 16 * NG - 1) / (16 * NG), a.nseq), 64 * NG, smem, s>>>(a, chunks);
+  ssd_chunk_kernel<DP, NG><<<dim3(a.heads, (a.vdim + 16 * NG - 1) / (16 * NG), a.nseq), 32 * (2 * NG + 1), smem, s>>>(a, chunks);
   return cudaGetLastError();
 }
 
@@ -752,9 +789,10 @@ cudaError_t ssd(const MatrixStateArgs& a, cudaStream_t s) {
 
 }  // namespace
 
-int64_t matrix_chunk_record_bytes(int dim, int delta) {
-  if (!delta) return SsdRecord::kBytes;
-  return dim <= 32 ? Record<32>::kBytes : dim <= 64 ? Record<64>::kBytes : dim <= 128 ? Record<128>::kBytes : Record<256>::kBytes;
+int64_t matrix_chunk_bytes(int heads, int key_heads, int dim, int delta) {
+  const int64_t h = heads, g = key_heads;
+  if (delta) return h * (dim <= 32 ? Record<32>::kBytes : dim <= 64 ? Record<64>::kBytes : dim <= 128 ? Record<128>::kBytes : Record<256>::kBytes);
+  return h * SsdRecord::kBytes + g * (dim <= 32 ? SsdTiles<32>::kBytes : dim <= 64 ? SsdTiles<64>::kBytes : dim <= 128 ? SsdTiles<128>::kBytes : SsdTiles<256>::kBytes);
 }
 
 cudaError_t launch_matrix_chunks(const MatrixStateArgs& a, cudaStream_t s) {

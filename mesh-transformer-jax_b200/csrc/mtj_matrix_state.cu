@@ -347,13 +347,13 @@ __device__ __forceinline__ float4 mul4(const float4& x, const float4& y) { retur
 template <typename F>
 __device__ __forceinline__ float4 map4(const float4& x, F&& f) { return make_float4(f(x.x), f(x.y), f(x.z), f(x.w)); }
 
-// part_n and the row strides multiples of four, part_n up to 16 TH: four neighbouring columns a thread, loads first
-template <typename T, int TH>
+// part_n and the row strides multiples of four, part_n up to 4 TH HOLD: four neighbouring columns a thread, loads first
+template <typename T, int TH, int HOLD>
 __global__ void __launch_bounds__(256) gated_norm_vec_kernel(const GatedNormArgs a) {
   __shared__ float red[8];
   pdl_wait();
   pdl_launch_dependents();
-  constexpr int kGroups = 256 / TH, kHold = 4;
+  constexpr int kGroups = 256 / TH, kHold = HOLD;
   const int grp = threadIdx.x / TH, t = threadIdx.x % TH;
   const int64_t id = static_cast<int64_t>(blockIdx.x) * kGroups + grp;
   if (id >= static_cast<int64_t>(a.M) * a.parts) return;   // whole groups leave; with TH = 256 the grid is exact
@@ -450,8 +450,12 @@ template <typename T>
 cudaError_t gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl) {
   const int64_t n = static_cast<int64_t>(a.M) * a.parts;
   if (((a.part_n | a.ld_y | a.ld_gate | a.ld_out) & 3) == 0 && a.part_n <= 16 * 256)
-    return a.part_n <= 16 * 32 ? launch_pdl(gated_norm_vec_kernel<T, 32>, dim3(static_cast<unsigned>((n + 7) / 8)), dim3(256), 0, s, pdl, a)
-                               : launch_pdl(gated_norm_vec_kernel<T, 256>, dim3(static_cast<unsigned>(n)), dim3(256), 0, s, pdl, a);
+  {
+    const dim3 eight(static_cast<unsigned>((n + 7) / 8)), one(static_cast<unsigned>(n)), block(256);
+    if (a.part_n <= 128) return launch_pdl(gated_norm_vec_kernel<T, 32, 1>, eight, block, 0, s, pdl, a);
+    if (a.part_n <= 512) return launch_pdl(gated_norm_vec_kernel<T, 32, 4>, eight, block, 0, s, pdl, a);
+    return a.part_n <= 1024 ? launch_pdl(gated_norm_vec_kernel<T, 256, 1>, one, block, 0, s, pdl, a) : launch_pdl(gated_norm_vec_kernel<T, 256, 4>, one, block, 0, s, pdl, a);
+  }
   if (a.part_n <= 256) return launch_pdl(gated_norm_kernel<T, 32>, dim3(static_cast<unsigned>((n + 7) / 8)), dim3(256), 0, s, pdl, a);
   return launch_pdl(gated_norm_kernel<T, 256>, dim3(static_cast<unsigned>(n)), dim3(256), 0, s, pdl, a);
 }

@@ -252,7 +252,7 @@ void LayerStack::carve_workspace(Carver& c) {
       aux = std::max<int64_t>(aux, up8(l.aux));
       mix = std::max<int64_t>(mix, l.out.ld);
       if (l.dt.N) dtw = std::max<int64_t>(dtw, up8(l.dt.N));
-      rec = std::max(rec, m.heads * matrix_chunk_record_bytes(m.dim, m.mixer == MTJ_MIXER_MATRIX_STATE_DELTA));
+      rec = std::max(rec, matrix_chunk_bytes(m.heads, m.kv_heads, m.dim, m.mixer == MTJ_MIXER_MATRIX_STATE_DELTA));
       if (l.gate2.N) gate = std::max<int64_t>(gate, up8(l.gate2.N));
     } else {
       qabs = std::max<int64_t>(qabs, static_cast<int64_t>(m.heads) * l.row_ld);

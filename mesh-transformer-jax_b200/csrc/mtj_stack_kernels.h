@@ -191,7 +191,7 @@ struct MatrixStateArgs {
   float* state;                // [slots][heads][dim][vdim]
   float* out;                  // [M, ld_out]
   int ld_out;
-  void* chunk_records;         // launch_matrix_chunks: nseq * ceil(Tc / kMatrixChunk) * heads records, 16-byte aligned
+  void* chunk_records;         // launch_matrix_chunks: nseq * ceil(Tc / kMatrixChunk) * matrix_chunk_bytes, 16-byte aligned
   uint32_t* dev_err;
 };
 // row by row
@@ -202,7 +202,7 @@ bool matrix_step_ok(const MatrixStateArgs& a);      // sizes that kernel takes
 bool matrix_step_norms(const MatrixStateArgs& a);
 // ---- mtj_matrix_chunk.cu: the same over long prompts, in chunks on the tensor cores (bf16 operands)
 constexpr int kMatrixChunk = 16;
-int64_t matrix_chunk_record_bytes(int dim, int delta);
+int64_t matrix_chunk_bytes(int heads, int key_heads, int dim, int delta);     // of chunk_records, per chunk of a sequence
 cudaError_t launch_matrix_chunks(const MatrixStateArgs& a, cudaStream_t s);
 cudaError_t launch_gated_norm(const GatedNormArgs& a, cudaStream_t s, bool pdl);
 constexpr int kMatrixMaxDim = 256;
