@@ -136,6 +136,31 @@ def test_extreme_decays(cuda_device, path):
         rt.close()
 
 
+def test_many_heads_and_sequences(cuda_device):
+    """More column groups than the GPU has SMs, so that blocks of the chunked scans hold four of them: unequal prompts
+    prefilled together, then a few decoded tokens, against each alone."""
+    import torch
+    for layer in (su.delta(heads=20, kv_heads=5, dim=40, vdim=64, ff=None), su.ssd(heads=20, vdim=60, state=48, groups=4, norm_groups=5)):
+        cfg = su.bavutar([layer], eps=1e-3)
+        w = su.weights(cfg, 13)
+        lens, seq, steps = [90, 33, 70, 2], 90, 3
+        seqs = [su.ids(80 + i, n + steps, cfg["vocab"]) for i, n in enumerate(lens)]
+        want = [bo.forward(cfg, w, s)[n - 1:] for s, n in zip(seqs, lens)]
+        rt = su.runtime(cfg, w, "many_rows", seq=seq, max_batch=4, max_gen=steps + 1, max_rows=4 * seq)
+        ctx = np.zeros((4, seq), np.int32)
+        for b, n in enumerate(lens):
+            ctx[b, seq - n:] = seqs[b][:n]
+        rt.prefill(torch.tensor(ctx, device=rt.device), lens)
+        logits, errs = torch.empty((4, cfg["vocab"]), device=rt.device), []
+        for t in range(steps + 1):
+            feed = None if t == 0 else torch.tensor([s[n - 1 + t] for s, n in zip(seqs, lens)], dtype=torch.int32, device=rt.device)
+            rt.decode_step(feed, None, logits)
+            errs += [su.error(logits.cpu().numpy()[b:b + 1], want[b][t:t + 1]) for b in range(4)]
+        rt.check_device_status()
+        rt.close()
+        assert max(errs) <= 2 * su.TOL["many_rows"], (layer["type"], errs)
+
+
 @pytest.mark.parametrize("path", sorted(su.PATHS))
 def test_query_temperature_at_its_steps(cuda_device, path):
     """Queries right before and after the positions where the temperature changes, in prompts and decoded."""
